@@ -4,12 +4,14 @@
 (``-gencode arch=compute_100a,code=sm_100a -lineinfo``), one object per source in
 parallel, and links them into ``blackwell_b200/lib/libblackwell_kernels.so`` and
 the static ``libblackwell_kernels.a`` the reference's consumers link against, and builds the JSON-lines daemon
-``blackwell_b200/lib/inference_server_w4a8`` from ``daemon/``.
+``blackwell_b200/lib/inference_server_w4a8`` and the trace runner from ``daemon/``.  ``build_trace_run`` compiles only what
+the trace runner needs (``bin/trace_run`` calls it).
 No GPU is needed to build.
 """
 from __future__ import annotations
 
 import concurrent.futures as cf
+import fcntl
 import glob
 import os
 import subprocess
@@ -23,6 +25,12 @@ SO = os.path.join(LIBDIR, "libblackwell_kernels.so")
 AR = os.path.join(LIBDIR, "libblackwell_kernels.a")
 DAEMON_SRC = os.path.join(HERE, "daemon", "inference_server_w4a8.cpp")
 DAEMON = os.path.join(LIBDIR, "inference_server_w4a8")
+TRACE_RUN_SRC = os.path.join(HERE, "daemon", "trace_run.cpp")
+TRACE_RUN = os.path.join(LIBDIR, "trace_run")
+# what a program that serves config.json models alone needs (no INT4 kernels); model_registry.cu is compiled for it
+# once more with the INT4 family left out
+CONFIG_MODEL_SOURCES = ["service", "decode_glue", "decode_engine", "layered_model", "model_spec", "lm_glue", "linear_bf16",
+                        "recurrence", "latent_attention"]
 
 # IEEE division and square root are requested explicitly: the quantizers must
 # round exactly like the reference's (v / sc, roundf).
@@ -42,8 +50,8 @@ def _deps_mtime():
     return max(os.path.getmtime(h) for h in hdrs) if hdrs else 0.0
 
 
-def _compile(src: str, verbose: bool, extra: list[str]) -> str:
-    obj = os.path.join(OBJDIR, os.path.basename(src)[:-3] + ".o")
+def _compile(src: str, verbose: bool, extra: list[str], suffix: str = "") -> str:
+    obj = os.path.join(OBJDIR, os.path.basename(src)[:-3] + suffix + ".o")
     newest = max(os.path.getmtime(src), _deps_mtime())
     if os.path.exists(obj) and os.path.getmtime(obj) >= newest:
         return obj
@@ -56,6 +64,24 @@ def _compile(src: str, verbose: bool, extra: list[str]) -> str:
     if verbose and (r.stdout or r.stderr):
         print(r.stdout + r.stderr)
     return obj
+
+
+def build_trace_run(verbose: bool = False) -> str:
+    """Build (if stale) and return the path of the trace runner: host program and kernels in one executable."""
+    os.makedirs(OBJDIR, exist_ok=True)
+    with open(os.path.join(LIBDIR, "trace_run.lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)   # one build at a time
+        jobs = [(os.path.join(CSRC, n + ".cu"), [], "") for n in CONFIG_MODEL_SOURCES]
+        jobs.append((os.path.join(CSRC, "model_registry.cu"), ["-DBW_CONFIG_MODELS_ONLY"], ".config"))
+        with cf.ThreadPoolExecutor(max_workers=len(jobs)) as ex:
+            objs = list(ex.map(lambda j: _compile(j[0], verbose, j[1], j[2]), jobs))
+        newest = max([os.path.getmtime(o) for o in objs] + [os.path.getmtime(TRACE_RUN_SRC)])
+        if not os.path.exists(TRACE_RUN) or os.path.getmtime(TRACE_RUN) < newest:
+            cmd = ["nvcc", "-std=c++17", "-O2", "-Wno-deprecated-gpu-targets", "-o", TRACE_RUN, TRACE_RUN_SRC, *objs]
+            if verbose:
+                print(" ".join(cmd), flush=True)
+            subprocess.check_call(cmd, stdout=sys.stderr)
+    return TRACE_RUN
 
 
 def build(verbose: bool = False, force: bool = False, extra: list[str] | None = None) -> str:
@@ -86,6 +112,7 @@ def build(verbose: bool = False, force: bool = False, extra: list[str] | None = 
         if verbose:
             print(" ".join(cmd), flush=True)
         subprocess.check_call(cmd)
+    build_trace_run(verbose)
     return SO
 
 

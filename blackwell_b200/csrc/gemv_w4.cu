@@ -140,27 +140,6 @@ extern "C" void bw_debug_set_timeline(void* dev_ptr) { g_timeline_ptr = static_c
 void* debug_timeline_ptr() { return g_timeline_ptr; }
 #endif
 static std::atomic<int> g_tune_mma_slab{0}, g_tune_mma_min{0}, g_tune_mma_max{0}, g_tune_mma_stages{0};
-static std::atomic<long long> g_launches{0};
-
-void count_launch(int n) { g_launches.fetch_add(n, std::memory_order_relaxed); }
-static std::atomic<int> g_pdl{1};
-bool pdl_enabled() { return g_pdl.load() != 0; }
-
-// One status word per device for the whole library: kernels that give up on a bounded wait store a code here.
-static __device__ int g_status_word = 0;
-int* status_word_ptr() {
-    static int* ptr[kMaxDevices] = {nullptr};
-    static std::mutex mu;
-    std::lock_guard<std::mutex> lk(mu);
-    const int dev = current_device();
-    if (!ptr[dev]) {
-        int* p = nullptr;
-        if (cudaGetSymbolAddress(reinterpret_cast<void**>(&p), g_status_word) != cudaSuccess) return nullptr;
-        ptr[dev] = p;
-    }
-    return ptr[dev];
-}
-
 struct StreamPlan {
     bool ok = false;
     int Tg = 0, G = 0, J = 0, S = 0, T = 0, rg = 0, row_unit = 1, n_rows = 0, grid = 0, ctas_per_sm = 2;
@@ -695,20 +674,6 @@ extern "C" int bw_gemv_block_dots(int32_t* dots, const void* x, int a8, const ui
     return cudaPeekAtLastError();
 }
 
-extern "C" int bw_device_status(int* status_out) {
-    int* p = status_word_ptr();
-    if (!p) return cudaErrorInitializationError;
-    int v = 0;
-    cudaError_t e = cudaMemcpy(&v, p, sizeof(int), cudaMemcpyDeviceToHost);
-    if (e != cudaSuccess) return e;
-    if (v != 0) {
-        const int zero = 0;
-        e = cudaMemcpy(p, &zero, sizeof(int), cudaMemcpyHostToDevice);
-    }
-    if (status_out) *status_out = v;
-    return e;
-}
-
 extern "C" size_t bw_gemv_scratch_bytes(int M, int N, int K) { return tc::scratch_bytes(M, N, K); }
 extern "C" size_t bw_attention_scratch_bytes(int M, int num_q_heads, int num_kv_heads, int max_context) {
     return attn_scratch_bytes(M, num_q_heads, num_kv_heads, max_context);
@@ -729,7 +694,7 @@ extern "C" int bw_set_tuning(int key, int value) {
         case 4: g_tune_threads = value; return 0;
         case 5: g_tune_tc_min = value; return 0;
         case 6: tc::set_ksplit_override(value); return 0;
-        case 8: g_pdl = value; return 0;
+        case 8: set_pdl(value); return 0;
         case 9: set_attn_mma(value); return 0;
         case 10: peer::set_two_step_min_kb(value); return 0;
         case 11: peer::set_wait_limit_ms(value); return 0;
@@ -747,9 +712,3 @@ extern "C" int bw_set_tuning(int key, int value) {
         default: return cudaErrorInvalidValue;
     }
 }
-
-extern "C" long long bw_launch_count(int reset) {
-    return reset ? g_launches.exchange(0) : g_launches.load();
-}
-
-extern "C" int bw_version(void) { return 100; }

@@ -30,6 +30,7 @@ inline int sm_count(int dev) {
 // Launch with programmatic stream serialization: the kernel may begin before its predecessor in the stream has
 // finished and must call pdl_wait() before touching anything the predecessor produces or still reads.
 bool pdl_enabled();
+void set_pdl(int on);
 template <typename... KArgs, typename... Args>
 inline cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t st,
                               Args... args) {

@@ -1,0 +1,125 @@
+// Launchers of the latent-cache attention.
+#include <cuda_runtime.h>
+
+#include <mutex>
+
+#include "host_util.h"
+#include "latent_attention.cuh"
+
+namespace bw {
+namespace lm {
+namespace {
+
+template <typename F>
+cudaError_t allow_smem(F kern, std::once_flag (&once)[kMaxDevices]) {
+    cudaError_t e = cudaSuccess;
+    std::call_once(once[current_device()], [&] { e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem); });
+    return e;
+}
+
+template <typename A, int RB>
+cudaError_t prep(const LatentArgs& a, const Rows& r, cudaStream_t st) {
+    static std::once_flag once[kMaxDevices];
+    cudaError_t e = allow_smem(latent_prep_kernel<A, RB>, once);
+    if (e != cudaSuccess) return e;
+    const int nc = pad8(a.R) / 8, groups = std::max(1, kPrepThreads / nc);
+    const size_t smem = std::max<size_t>(128, (size_t)(RB * (pad8(a.dim) + pad8(a.rot)) + groups * RB * pad8(a.R)) * 4);
+    if (smem > kMaxDynSmem) return cudaErrorInvalidValue;
+    count_launch(1);
+    return launch_pdl(latent_prep_kernel<A, RB>, dim3(a.heads + (a.dkv ? 1 : 0), (r.T + RB - 1) / RB), dim3(kPrepThreads), smem, st, a, r);
+}
+
+template <typename A, int RB>
+cudaError_t out(const LatentArgs& a, const Rows& r, cudaStream_t st) {
+    static std::once_flag once[kMaxDevices];
+    cudaError_t e = allow_smem(latent_out_kernel<A, RB>, once);
+    if (e != cudaSuccess) return e;
+    const size_t smem = (size_t)(RB * pad8(a.R) + RB * a.splits) * 4;
+    if (smem > kMaxDynSmem) return cudaErrorInvalidValue;
+    count_launch(1);
+    return launch_pdl(latent_out_kernel<A, RB>, dim3(a.heads, (r.T + RB - 1) / RB), dim3(256), smem, st, a, r);
+}
+
+template <typename A>
+cudaError_t scalar(const LatentArgs& a, const Rows& r, cudaStream_t st) {
+    const size_t smem = (size_t)(latent_dp(a.R, a.rot) + kScalarKeys) * 4;
+    count_launch(1);
+    return launch_pdl(latent_scalar_kernel<A>, dim3(a.splits, a.heads, r.T), dim3(256), smem, st, a, r);
+}
+
+template <int NT>
+cudaError_t decode(const LatentArgs& a, const Rows& r, int nbuf, cudaStream_t st) {
+    static std::once_flag once[kMaxDevices];
+    cudaError_t e = allow_smem(latent_decode_kernel<NT>, once);
+    if (e != cudaSuccess) return e;
+    count_launch(1);
+    return launch_pdl(latent_decode_kernel<NT>, dim3(a.splits, (a.heads + 15) / 16, r.T), dim3(256), DecodeSmem(a.R, a.rot, nbuf).total,
+                      st, a, r, nbuf);
+}
+
+template <int VT>
+cudaError_t flash(const LatentArgs& a, const Rows& r, cudaStream_t st) {
+    static std::once_flag once[kMaxDevices];
+    cudaError_t e = allow_smem(latent_flash_kernel<VT>, once);
+    if (e != cudaSuccess) return e;
+    const int D = pad16(pad8(a.dim) + pad8(a.rot));
+    count_launch(1);
+    return launch_pdl(latent_flash_kernel<VT>, dim3((r.T + kFlashQ - 1) / kFlashQ, a.heads, (pad8(a.V) + VT * 8 - 1) / (VT * 8)), dim3(256),
+                      FlashSmem(D, VT).total, st, a, r);
+}
+
+int flash_vt(const LatentArgs& a) {
+    const int D = pad16(pad8(a.dim) + pad8(a.rot));
+    int vt = a.V <= 64 ? 8 : a.V <= 128 ? 16 : 32;
+    while (vt > 8 && FlashSmem(D, vt).total > kMaxDynSmem) vt /= 2;
+    return FlashSmem(D, vt).total <= kMaxDynSmem ? vt : 0;
+}
+
+}  // namespace
+
+bool latent_absorbed_supported(const LatentArgs& a) {
+    const int nc = pad8(a.R) / 8, groups = std::max(1, kPrepThreads / nc);
+    return a.R >= 1 && a.R <= 2048 && (size_t)(pad8(a.dim) + pad8(a.rot) + groups * pad8(a.R)) * 4 <= (size_t)kMaxDynSmem;
+}
+bool latent_expanded_supported(const LatentArgs& a) { return flash_vt(a) > 0; }
+
+cudaError_t latent_absorbed(const LatentArgs& a, const Rows& r, int f32, cudaStream_t st) {
+    const bool rb4 = r.T >= 8 && !f32 && a.R <= 512;
+    cudaError_t e = f32 ? prep<float, 1>(a, r, st) : rb4 ? prep<bf16, 4>(a, r, st) : prep<bf16, 1>(a, r, st);
+    if (e != cudaSuccess) return e;
+    const int nbuf = DecodeSmem(a.R, a.rot, 2).total <= kMaxDynSmem ? 2 : 1;
+    if (f32) e = scalar<float>(a, r, st);
+    else if (a.R > 1024 || DecodeSmem(a.R, a.rot, nbuf).total > kMaxDynSmem) e = scalar<bf16>(a, r, st);
+    else if (a.R <= 128) e = decode<2>(a, r, nbuf, st);
+    else if (a.R <= 256) e = decode<4>(a, r, nbuf, st);
+    else if (a.R <= 512) e = decode<8>(a, r, nbuf, st);
+    else e = decode<16>(a, r, nbuf, st);
+    if (e != cudaSuccess) return e;
+    return f32 ? out<float, 1>(a, r, st) : rb4 ? out<bf16, 4>(a, r, st) : out<bf16, 1>(a, r, st);
+}
+
+cudaError_t latent_expanded(const LatentArgs& a, const Rows& r, cudaStream_t st) {
+    if (r.row_slot) return cudaErrorInvalidValue;
+    cudaError_t e = cudaSuccess;
+    if (a.dkv) {
+        count_launch(1);
+        e = launch_pdl(latent_cache_kernel<bf16>, dim3(r.T), dim3(128), 0, st, a, r);
+        if (e != cudaSuccess) return e;
+    }
+    if (a.rot_dims >= 2) {
+        count_launch(1);
+        e = launch_pdl(latent_rotate_q_kernel, dim3((a.heads * (a.rot_dims / 2) + 127) / 128, r.T), dim3(128), 0, st, a, r);
+        if (e != cudaSuccess) return e;
+    }
+    LinearArgs x{};   // keys and values of the whole context
+    x.x = static_cast<const bf16*>(a.cache) + (long)r.slot * a.max_seq * a.ldc;
+    x.ldx = a.ldc; x.W = a.Wkv; x.ldw = a.ldw; x.T = r.pos0 + r.T; x.K = a.R;
+    x.N = a.heads * (pad8(a.dim) + pad8(a.V)); x.y = a.kv; x.ldy = x.N; x.split = x.N;
+    e = linear(x, st);
+    if (e != cudaSuccess) return e;
+    const int vt = flash_vt(a);
+    return vt == 8 ? flash<8>(a, r, st) : vt == 16 ? flash<16>(a, r, st) : vt == 32 ? flash<32>(a, r, st) : cudaErrorInvalidValue;
+}
+
+}  // namespace lm
+}  // namespace bw

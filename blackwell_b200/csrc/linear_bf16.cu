@@ -1,0 +1,147 @@
+// Host side of the bfloat16 linear kernels: routing by row count, tensor maps, launch shapes.
+#include <cuda.h>
+#include <cuda_runtime.h>
+
+#include <atomic>
+#include <mutex>
+
+#include "../../include/blackwell_b200.h"
+#include "host_util.h"
+#include "linear_bf16.cuh"
+
+namespace bw {
+namespace lm {
+namespace {
+
+typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+EncodeTiledFn encode_fn() {
+    static EncodeTiledFn fn = nullptr;
+    static std::once_flag once;
+    std::call_once(once, [] {
+        void* p = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) == cudaSuccess &&
+            q == cudaDriverEntryPointSuccess)
+            fn = reinterpret_cast<EncodeTiledFn>(p);
+    });
+    return fn;
+}
+
+// Row-major bf16 matrix [rows][cols], boxes of box_rows x 64 columns in the 128-byte swizzle.
+bool make_map(CUtensorMap* m, const void* base, int cols, int rows, long ld, int box_rows) {
+    const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+    const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {(cuuint32_t)kTcK, (cuuint32_t)box_rows}, es[2] = {1, 1};
+    return encode_fn()(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, es,
+                       CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                       CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+template <typename F>
+cudaError_t allow_smem(F kern, std::once_flag (&once)[kMaxDevices], int bytes) {
+    cudaError_t e = cudaSuccess;
+    std::call_once(once[current_device()], [&] { e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes); });
+    return e;
+}
+
+int stream_xs_stride(int ldw) {
+    const int nkb = (ldw + 31) / 32;
+    return nkb * 64 + (nkb % 2 == 0 ? 64 : 0);   // odd multiple of 64 bytes: conflict-free fragment reads
+}
+int stream_smem(int NT, int ldw) { return kStreamWarps * NT * 8 * 16 * 4 + NT * 8 * stream_xs_stride(ldw); }
+
+template <int NT>
+cudaError_t launch_stream(const LinearArgs& a, cudaStream_t st) {
+    static std::once_flag once[kMaxDevices];
+    cudaError_t e = allow_smem(linear_stream_kernel<NT>, once, kMaxDynSmem);
+    if (e != cudaSuccess) return e;
+    const int smem = stream_smem(NT, (int)a.ldw), tiles = (a.N + 15) / 16;
+    const int per_sm = smem > 110 * 1024 ? 1 : smem > 72 * 1024 ? 2 : 3;
+    const int grid = std::min(tiles, sm_count(current_device()) * per_sm);
+    e = launch_pdl(linear_stream_kernel<NT>, dim3(grid), dim3(kStreamWarps * 32), smem, st, a, stream_xs_stride((int)a.ldw));
+    count_launch(1);
+    return e;
+}
+
+template <int NT, bool SPLIT>
+cudaError_t launch_tc(const LinearArgs& a, int ksplit, cudaStream_t st) {
+    static std::once_flag once[kMaxDevices];
+    auto kern = linear_tc_kernel<NT, SPLIT>;
+    const int smem = tc_smem_bytes(NT, SPLIT);
+    static_assert(tc_smem_bytes(NT, SPLIT) <= kMaxDynSmem, "shared memory");
+    cudaError_t e = allow_smem(kern, once, smem);
+    if (e != cudaSuccess) return e;
+    if (!encode_fn()) return cudaErrorNotSupported;
+    CUtensorMap mw, mx;
+    if (!make_map(&mw, a.W, a.K, a.N, a.ldw, kTcRows) || !make_map(&mx, a.x, a.K, a.T, a.ldx, NT)) return cudaErrorInvalidValue;
+    const int tiles = ((a.N + kTcRows - 1) / kTcRows) * ((a.T + NT - 1) / NT);
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(SPLIT ? tiles * ksplit : std::min(tiles, sm_count(current_device())));
+    cfg.blockDim = dim3(kTcThreads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = ksplit;
+    attr[1].val.clusterDim.y = 1;
+    attr[1].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = SPLIT ? 2 : 1;
+    int* status = status_word_ptr();
+    e = cudaLaunchKernelEx(&cfg, kern, mw, mx, a, ksplit, status);
+    count_launch(1);
+    return e;
+}
+
+std::atomic<int> g_stream_max{32};
+
+}  // namespace
+
+void set_linear_stream_max(int rows) { g_stream_max = rows > 0 ? std::min(rows, 32) : 32; }
+
+cudaError_t linear(const LinearArgs& a, cudaStream_t st) {
+    if (a.T < 1 || a.N < 1 || a.K < 1 || a.ldw % 8 != 0 || a.ldw < a.K || (reinterpret_cast<uintptr_t>(a.W) & 15) ||
+        (reinterpret_cast<uintptr_t>(a.x) & 15) || a.ldx < a.K || (a.epi == kEpiSwiglu && a.N % 2 != 0))
+        return cudaErrorInvalidValue;
+    if (a.f32) {
+        const dim3 grid((a.N + 63) / 64, (a.T + 63) / 64);
+        cudaError_t e = launch_pdl(linear_f32_kernel, grid, dim3(256), 0, st, a);
+        count_launch(1);
+        return e;
+    }
+    if (a.ldx % 8 != 0) return cudaErrorInvalidValue;
+    const int nt = a.T <= 8 ? 1 : a.T <= 16 ? 2 : 4;
+    if (a.T <= g_stream_max && stream_smem(nt, (int)a.ldw) <= kMaxDynSmem)
+        return nt == 1 ? launch_stream<1>(a, st) : nt == 2 ? launch_stream<2>(a, st) : launch_stream<4>(a, st);
+    // enough tiles for the SMs: persistent tiles of 256 / 128 rows; otherwise the K range is split over a cluster
+    const int sms = sm_count(current_device()), rtiles = (a.N + kTcRows - 1) / kTcRows, nk = (a.K + kTcK - 1) / kTcK;
+    auto tiles = [&](int nt_) { return rtiles * ((a.T + nt_ - 1) / nt_); };
+    if (a.T > 64) {
+        if (tiles(256) >= sms) return launch_tc<256, false>(a, 1, st);
+        if (a.T > 128 || tiles(128) >= sms / 2) {
+            // fewer, larger tiles only when they fill the machine as well as the small ones do
+            const long w128 = (long)((tiles(128) + sms - 1) / sms), w64 = (long)((tiles(64) + sms - 1) / sms);
+            return 2 * w64 < 2 * w128 + 1 && w64 * 64 < w128 * 128 ? launch_tc<64, false>(a, 1, st) : launch_tc<128, false>(a, 1, st);
+        }
+    }
+    const int ntile = a.T <= 16 ? 16 : a.T <= 32 ? 32 : 64;
+    int ks = 1;
+    while (ks < 8 && 2 * ks <= nk && tiles(ntile) * 2 * ks <= sms + sms / 4) ks *= 2;
+    return ntile == 16 ? launch_tc<16, true>(a, ks, st) : ntile == 32 ? launch_tc<32, true>(a, ks, st) : launch_tc<64, true>(a, ks, st);
+}
+
+}  // namespace lm
+}  // namespace bw
+
+extern "C" int bw_linear_bf16(void* y, long ldy, const void* x, long ldx, const uint16_t* W, long ldw, int T, int N, int K,
+                              int y_f32, int x_f32, int epilogue, float softcap, void* stream) {
+    if (!y || !x || !W || epilogue < 0 || epilogue > 2) return cudaErrorInvalidValue;
+    bw::lm::LinearArgs a{};
+    a.x = x; a.ldx = ldx; a.W = reinterpret_cast<const bw::lm::bf16*>(W); a.ldw = ldw; a.T = T; a.N = N; a.K = K;
+    a.y = y; a.ldy = ldy; a.y_f32 = y_f32; a.split = N; a.epi = epilogue; a.softcap = softcap; a.f32 = x_f32;
+    return bw::lm::linear(a, static_cast<cudaStream_t>(stream));
+}

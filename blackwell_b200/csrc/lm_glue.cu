@@ -1,0 +1,208 @@
+// Element-wise and per-row kernels of the config.json models: embedding lookup, norms on the sublayer output with the
+// residual sum, gated group norm, short causal convolution with its step sizes.  fp32 arithmetic throughout; activations
+// are read and written as bf16 (serving) or fp32 (32-bit mode).
+#include <cuda_runtime.h>
+
+#include "host_util.h"
+#include "lm_device.cuh"
+#include "lm_ops.h"
+
+namespace bw {
+namespace lm {
+namespace {
+
+template <typename A>
+__global__ void __launch_bounds__(256) embed_kernel(float* x, A* xb, long ldxb, const bf16* table, long ldt, const int* tokens,
+                                                    int width, int vocab) {
+    pdl_trigger();
+    pdl_wait();
+    const int r = blockIdx.y, i = blockIdx.x * 256 + threadIdx.x;
+    if (i >= width) return;
+    int tok = tokens[r];
+    tok = tok < 0 ? 0 : tok >= vocab ? vocab - 1 : tok;
+    const float v = to_f(table[(long)tok * ldt + i]);
+    x[(long)r * width + i] = v;
+    xb[(long)r * ldxb + i] = from_f<A>(v);
+}
+
+// ADD: x += y / rms(y) * w and xb = x; otherwise xb = x / rms(x) * w for a listed row.
+template <typename A, bool ADD>
+__global__ void __launch_bounds__(512) norm_kernel(float* x, A* xb, long ldxb, const float* y, const float* w, const int* rows,
+                                                   int width, float eps) {
+    __shared__ float buf[32];
+    pdl_trigger();
+    pdl_wait();
+    const int out_row = blockIdx.x;
+    const long r = rows ? rows[out_row] : out_row;
+    const float* src = (ADD ? y : x) + r * width;
+    float ss = 0.f;
+    constexpr int kKeep = 8;   // the first values stay in registers
+    float keep[kKeep];
+#pragma unroll
+    for (int j = 0; j < kKeep; ++j) {
+        const int i = j * blockDim.x + threadIdx.x;
+        keep[j] = i < width ? src[i] : 0.f;
+        ss = fmaf(keep[j], keep[j], ss);
+    }
+    for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) ss = fmaf(src[i], src[i], ss);
+    const float rms = 1.0f / sqrtf(block_sum(ss, buf) / (float)width + eps);
+    auto emit = [&](int i, float v) {
+        v = v * rms * w[i];
+        if (ADD) {
+            v += x[r * width + i];
+            x[r * width + i] = v;
+        }
+        xb[(long)out_row * ldxb + i] = from_f<A>(v);
+    };
+#pragma unroll
+    for (int j = 0; j < kKeep; ++j) {
+        const int i = j * blockDim.x + threadIdx.x;
+        if (i < width) emit(i, keep[j]);
+    }
+    for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) emit(i, src[i]);
+}
+
+template <typename A>
+__global__ void __launch_bounds__(256) gated_norm_kernel(A* out, long ldout, const float* o, long ldo, const A* gate, long ldg,
+                                                         const float* w, int heads, int V, int groups, int gate_first,
+                                                         float eps) {
+    __shared__ float buf[32];
+    pdl_trigger();
+    pdl_wait();
+    const int grp = blockIdx.x, t = threadIdx.x;
+    const long r = blockIdx.y;
+    const int part = heads * V / groups, c0 = grp * part, V8 = pad8(V);
+    const float* orow = o + r * ldo;
+    const A* grow = gate + r * ldg;
+    float ss = 0.f;
+    for (int i = t; i < part; i += 256) {
+        const int c = c0 + i, col = (c / V) * V8 + c % V;
+        float v = orow[col];
+        if (gate_first) v *= silu_f(to_f(grow[col]));
+        ss = fmaf(v, v, ss);
+    }
+    const float rms = 1.0f / sqrtf(block_sum(ss, buf) / (float)part + eps);
+    for (int i = t; i < part; i += 256) {
+        const int c = c0 + i, h = c / V, v0 = c - h * V, col = h * V8 + v0;
+        const float v = orow[col] * silu_f(to_f(grow[col])) * rms * (w ? w[c] : 1.f);
+        out[r * ldout + col] = from_f<A>(v);
+        if (v0 == V - 1)
+            for (int z = V; z < V8; ++z) out[r * ldout + h * V8 + z] = from_f<A>(0.f);
+    }
+}
+
+// Conv channel of a padded column (counted from the start of the convolved part), -1 for padding.
+__device__ __forceinline__ int conv_channel(const ConvArgs& c, int col) {
+    const int V8 = pad8(c.V), N8 = pad8(c.N), x_cols = c.heads * V8;
+    if (col < x_cols) return col % V8 < c.V ? (col / V8) * c.V + col % V8 : -1;
+    const int b = col - x_cols;   // k groups, then q groups
+    return b % N8 < c.N ? c.heads * c.V + (b / N8) * c.N + b % N8 : -1;
+}
+__host__ __device__ __forceinline__ int conv_cols(const ConvArgs& c) { return c.heads * pad8(c.V) + 2 * c.groups * pad8(c.N); }
+
+constexpr int kConvRows = 8;   // rows per block
+
+template <typename A>
+__global__ void __launch_bounds__(128) conv_silu_kernel(const ConvArgs c, const Rows r) {
+    pdl_wait();
+    const int channels = c.heads * c.V + 2 * c.groups * c.N, cols = conv_cols(c);
+    const int col = blockIdx.x * 128 + threadIdx.x, t0 = blockIdx.y * kConvRows, t1 = min(r.T, t0 + kConvRows);
+    if (col < cols) {
+        const int ch = conv_channel(c, col);
+        if (ch < 0) {
+            for (int t = t0; t < t1; ++t) static_cast<A*>(c.out)[(long)t * c.ldo + col] = from_f<A>(0.f);
+            return;
+        }
+        const A* u = static_cast<const A*>(c.u) + c.off + col;
+        const float* ring = c.ring + (long)r.slot * c.taps * channels + ch;
+        const float bias = c.bias[ch];
+        for (int t = t0; t < t1; ++t) {
+            float y = bias;
+            for (int j = 0; j < c.taps; ++j) {
+                const int s = t - (c.taps - 1) + j, p = r.pos0 + s;
+                float v = 0.f;
+                if (s >= 0) v = to_f(u[(long)s * c.ldu]);
+                else if (p >= 0) v = ring[(long)(p % c.taps) * channels];
+                y = fmaf(c.w[ch * c.taps + j], v, y);
+            }
+            static_cast<A*>(c.out)[(long)t * c.ldo + col] = from_f<A>(silu_f(y));
+        }
+    } else if (col < cols + c.heads) {
+        const int h = col - cols;
+        const float a = -expf(c.A_log[h]), b = c.dt_bias[h];
+        for (int t = t0; t < t1; ++t) {
+            const float dt = softplus_f(c.dt_raw[(long)t * c.ld_dt + h] + b);
+            c.log_decay[(long)t * c.heads + h] = a * dt;
+            c.weight[(long)t * c.heads + h] = dt;
+        }
+    }
+}
+
+template <typename A>
+__global__ void __launch_bounds__(128) conv_ring_kernel(const ConvArgs c, const Rows r) {
+    pdl_wait();
+    const int channels = c.heads * c.V + 2 * c.groups * c.N, col = blockIdx.x * 128 + threadIdx.x;
+    const int ch = col < conv_cols(c) ? conv_channel(c, col) : -1;
+    if (ch < 0) return;
+    const A* u = static_cast<const A*>(c.u) + c.off + col;
+    float* ring = c.ring + (long)r.slot * c.taps * channels + ch;
+    for (int t = max(0, r.T - (c.taps - 1)); t < r.T; ++t) ring[(long)((r.pos0 + t) % c.taps) * channels] = to_f(u[(long)t * c.ldu]);
+}
+
+}  // namespace
+
+cudaError_t embed(float* x, void* xb, long ldxb, const bf16* table, long ldt, const int* tokens, int T, int width, int vocab,
+                  int f32, cudaStream_t st) {
+    const dim3 grid((width + 255) / 256, T), block(256);
+    count_launch(1);
+    return f32 ? launch_pdl(embed_kernel<float>, grid, block, 0, st, x, static_cast<float*>(xb), ldxb, table, ldt, tokens, width, vocab)
+               : launch_pdl(embed_kernel<bf16>, grid, block, 0, st, x, static_cast<bf16*>(xb), ldxb, table, ldt, tokens, width, vocab);
+}
+
+static int norm_threads(int width) { return width <= 256 ? 64 : width <= 1024 ? 128 : width <= 2048 ? 256 : 512; }
+
+cudaError_t norm_add(float* x, void* xb, long ldxb, const float* y, const float* w, int T, int width, float eps, int f32,
+                     cudaStream_t st) {
+    const dim3 grid(T), block(norm_threads(width));
+    const int* none = nullptr;
+    count_launch(1);
+    return f32 ? launch_pdl(norm_kernel<float, true>, grid, block, 0, st, x, static_cast<float*>(xb), ldxb, y, w, none, width, eps)
+               : launch_pdl(norm_kernel<bf16, true>, grid, block, 0, st, x, static_cast<bf16*>(xb), ldxb, y, w, none, width, eps);
+}
+
+cudaError_t norm_rows(void* xb, long ldxb, const float* x, const float* w, const int* rows, int T, int width, float eps, int f32,
+                      cudaStream_t st) {
+    const dim3 grid(T), block(norm_threads(width));
+    float* xm = const_cast<float*>(x);
+    const float* none = nullptr;
+    count_launch(1);
+    return f32 ? launch_pdl(norm_kernel<float, false>, grid, block, 0, st, xm, static_cast<float*>(xb), ldxb, none, w, rows, width, eps)
+               : launch_pdl(norm_kernel<bf16, false>, grid, block, 0, st, xm, static_cast<bf16*>(xb), ldxb, none, w, rows, width, eps);
+}
+
+cudaError_t gated_norm(void* out, long ldout, const float* o, long ldo, const void* gate, long ldg, const float* w, int T,
+                       int heads, int V, int groups, int gate_first, float eps, int f32, cudaStream_t st) {
+    if (groups < 1 || (heads * V) % groups != 0) return cudaErrorInvalidValue;
+    const dim3 grid(groups, T), block(256);
+    count_launch(1);
+    return f32 ? launch_pdl(gated_norm_kernel<float>, grid, block, 0, st, static_cast<float*>(out), ldout, o, ldo,
+                            static_cast<const float*>(gate), ldg, w, heads, V, groups, gate_first, eps)
+               : launch_pdl(gated_norm_kernel<bf16>, grid, block, 0, st, static_cast<bf16*>(out), ldout, o, ldo,
+                            static_cast<const bf16*>(gate), ldg, w, heads, V, groups, gate_first, eps);
+}
+
+cudaError_t conv_silu(const ConvArgs& c, const Rows& r, int f32, cudaStream_t st) {
+    const int n = conv_cols(c) + c.heads;
+    const dim3 grid((n + 127) / 128, (r.T + kConvRows - 1) / kConvRows), block(128);
+    count_launch(1);
+    return f32 ? launch_pdl(conv_silu_kernel<float>, grid, block, 0, st, c, r) : launch_pdl(conv_silu_kernel<bf16>, grid, block, 0, st, c, r);
+}
+
+cudaError_t conv_ring_store(const ConvArgs& c, const Rows& r, int f32, cudaStream_t st) {
+    const dim3 grid((conv_cols(c) + 127) / 128), block(128);
+    count_launch(1);
+    return f32 ? launch_pdl(conv_ring_kernel<float>, grid, block, 0, st, c, r) : launch_pdl(conv_ring_kernel<bf16>, grid, block, 0, st, c, r);
+}
+
+}  // namespace lm
+}  // namespace bw

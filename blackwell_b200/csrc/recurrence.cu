@@ -1,0 +1,59 @@
+// Launchers of the gated linear recurrence.
+#include <cuda_runtime.h>
+
+#include <mutex>
+
+#include "host_util.h"
+#include "recurrence.cuh"
+
+namespace bw {
+namespace lm {
+namespace {
+
+template <typename A, int NR, bool CONV>
+cudaError_t step_inst(const RecurrenceArgs& a, const ConvArgs& c, const Rows& r, cudaStream_t st) {
+    const dim3 grid((pad8(a.V) + kRecV - 1) / kRecV, a.heads, r.row_slot ? r.T : 1);
+    const int smem = (64 * NR + kRecV + 2 * 8 * kRecV) * 4;
+    count_launch(1);
+    return launch_pdl(recurrence_step_kernel<A, NR, CONV>, grid, dim3(kRecThreads), smem, st, a, c, r);
+}
+template <typename A, bool CONV>
+cudaError_t step_nr(const RecurrenceArgs& a, const ConvArgs& c, const Rows& r, cudaStream_t st) {
+    const int nr = (a.N + 31) / 32;
+    return nr <= 1 ? step_inst<A, 1, CONV>(a, c, r, st) : nr <= 2 ? step_inst<A, 2, CONV>(a, c, r, st)
+         : nr <= 4 ? step_inst<A, 4, CONV>(a, c, r, st) : nr <= 8 ? step_inst<A, 8, CONV>(a, c, r, st)
+         : nr <= 16 ? step_inst<A, 16, CONV>(a, c, r, st) : cudaErrorInvalidValue;
+}
+
+template <int NTW>
+cudaError_t chunk_inst(const RecurrenceArgs& a, const Rows& r, cudaStream_t st) {
+    static std::once_flag once[kMaxDevices];
+    cudaError_t e = cudaSuccess;
+    std::call_once(once[current_device()], [&] {
+        e = cudaFuncSetAttribute(recurrence_chunk_kernel<NTW>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem);
+    });
+    if (e != cudaSuccess) return e;
+    const int nbuf = ChunkSmem(a.N, 2).total <= kMaxDynSmem ? 2 : 1;
+    const dim3 grid((pad8(a.V) + kChV - 1) / kChV, a.heads);
+    count_launch(1);
+    return launch_pdl(recurrence_chunk_kernel<NTW>, grid, dim3(256), ChunkSmem(a.N, nbuf).total, st, a, r, nbuf);
+}
+
+}  // namespace
+
+cudaError_t recurrence_step(const RecurrenceArgs& a, const ConvArgs* conv, const Rows& r, int f32, cudaStream_t st) {
+    if (a.groups < 1 || a.heads % a.groups != 0 || (conv && !r.row_slot)) return cudaErrorInvalidValue;
+    const ConvArgs none{};
+    if (conv) return f32 ? step_nr<float, true>(a, *conv, r, st) : step_nr<bf16, true>(a, *conv, r, st);
+    return f32 ? step_nr<float, false>(a, none, r, st) : step_nr<bf16, false>(a, none, r, st);
+}
+
+bool recurrence_chunk_supported(const RecurrenceArgs& a) { return a.N <= 256 && ChunkSmem(a.N, 1).total <= kMaxDynSmem; }
+
+cudaError_t recurrence_chunk(const RecurrenceArgs& a, const Rows& r, cudaStream_t st) {
+    if (a.groups < 1 || a.heads % a.groups != 0 || r.row_slot || !recurrence_chunk_supported(a)) return cudaErrorInvalidValue;
+    return pad16(a.N) <= 128 ? chunk_inst<1>(a, r, st) : chunk_inst<2>(a, r, st);
+}
+
+}  // namespace lm
+}  // namespace bw

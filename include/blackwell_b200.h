@@ -357,14 +357,49 @@ typedef struct bw_decode_config {
     int act_bits;             /* 8 or 4 */
     int use_graph;            /* capture the step once and replay it */
     const char* weights_dir;  /* read during bw_decode_create only */
+    int compute_f32;          /* config.json models: 1 = 32-bit activations and products (0: bfloat16) */
+    int max_portion;          /* config.json models: most tokens of one sequence per pass (0: automatic) */
 } bw_decode_config;
 int bw_decode_create(const bw_decode_config* cfg, bw_decode** out);
+int bw_decode_get_config(const bw_decode* d, bw_decode_config* out);
 int bw_decode_begin(bw_decode* d, const int* prompt_ids, const int* prompt_len, int max_prompt, void* stream);
 int bw_decode_step(bw_decode* d, void* stream);
 int bw_decode_result(bw_decode* d, int* gen_out, void* stream);
 int bw_decode_buffers(bw_decode* d, float** logits, float** hidden, int** positions, int** sampled,
                       uint16_t** k_cache, uint16_t** v_cache);
 int bw_decode_destroy(bw_decode* d);
+
+/* Model families.  bw_decode_create looks at the weight directory: one with a config.json is a layered model whose
+ * architecture config.json names ("Vifivik": mamba2, latent-attention and retention layers; weights in
+ * model.safetensors, bfloat16) -- sizes and constants come from config.json, the corresponding fields of bw_decode_config
+ * are ignored and bw_decode_get_config returns them; any other directory is the INT4 container format above.
+ * bw_model_probe reads config.json only (no GPU) and, where it is not usable, leaves the reason in message.
+ *   Layered models take portions: bw_decode_begin runs each prompt but its last token through the prompt kernels, so
+ * that a generation of n tokens needs n steps (bw_decode_steps gives the number for either family).
+ * bw_decode_portion feeds the next n tokens of one slot at any cut -- n == 1 uses the decode step's kernels -- and
+ * returns to host memory the logits [n_want][vocab] at the places want[] (ascending, within the portion); it
+ * synchronises.  bw_decode_release gives a slot back: the next portion starts a new sequence.  bw_decode_held is the number
+ * of tokens a slot holds.  bw_decode_watch_layers: while buffer (device, [layers][rows][hidden] fp32) is not NULL,
+ * portions also store the residual stream after every layer there. */
+typedef struct bw_model_info {
+    char architecture[64];
+    int layers, width, vocab;
+    int mamba2_layers, retention_layers, latent_layers, shared_cache_layers;
+} bw_model_info;
+int bw_model_probe(const char* dir, bw_model_info* out, char* message, int message_bytes);
+int bw_decode_steps(const bw_decode* d, int longest_prompt, int new_tokens);
+int bw_decode_portion(bw_decode* d, int slot, const int* tokens, int n, const int* want, int n_want, float* logits_out,
+                      void* stream);
+int bw_decode_release(bw_decode* d, int slot);
+int bw_decode_held(const bw_decode* d, int slot);
+int bw_decode_watch_layers(bw_decode* d, float* buffer, long rows);
+
+/* y[t][n] = sum_k x[t][k] W[n][k] with bfloat16 W [N][ldw] (ldw a multiple of 8, zero beyond K): the product of the
+ * layered models.  x bfloat16 [T][ldx] (ldx a multiple of 8), or fp32 when x_f32 (32-bit FMAs); y bfloat16 or, with y_f32
+ * (or x_f32), fp32.  epilogue 0: none; 1: rows 2j / 2j+1 of W are gate / up, y[t][j] = silu(gate) * up, N / 2 columns in
+ * x's format; 2: softcap * tanh(y / softcap).  Up to 32 rows a weight-streaming kernel, beyond that tcgen05. */
+int bw_linear_bf16(void* y, long ldy, const void* x, long ldx, const uint16_t* W, long ldw, int T, int N, int K,
+                   int y_f32, int x_f32, int epilogue, float softcap, void* stream);
 
 /* ---- Tensor-parallel exchange over peer memory (no counterpart in the reference, which is single-GPU) ----
  * All-reduce of the K-split projections' partial sums across the GPUs of one box through NVLink peer loads.
