@@ -75,7 +75,7 @@ def build_trace_run(verbose: bool = False) -> str:
         jobs.append((os.path.join(CSRC, "model_registry.cu"), ["-DBW_CONFIG_MODELS_ONLY"], ".config"))
         with cf.ThreadPoolExecutor(max_workers=len(jobs)) as ex:
             objs = list(ex.map(lambda j: _compile(j[0], verbose, j[1], j[2]), jobs))
-        newest = max([os.path.getmtime(o) for o in objs] + [os.path.getmtime(TRACE_RUN_SRC)])
+        newest = max([os.path.getmtime(o) for o in objs] + [os.path.getmtime(TRACE_RUN_SRC), _deps_mtime()])
         if not os.path.exists(TRACE_RUN) or os.path.getmtime(TRACE_RUN) < newest:
             cmd = ["nvcc", "-std=c++17", "-O2", "-Wno-deprecated-gpu-targets", "-o", TRACE_RUN, TRACE_RUN_SRC, *objs]
             if verbose:
@@ -106,7 +106,7 @@ def build(verbose: bool = False, force: bool = False, extra: list[str] | None = 
             os.remove(AR)
         subprocess.check_call(["ar", "rcs", AR, *objs])
     # the JSON-lines daemon on the decode-step driver: host C++ above the C ABI, linked against the shared library
-    if not os.path.exists(DAEMON) or os.path.getmtime(DAEMON) < max(os.path.getmtime(DAEMON_SRC), os.path.getmtime(SO)):
+    if not os.path.exists(DAEMON) or os.path.getmtime(DAEMON) < max(os.path.getmtime(DAEMON_SRC), os.path.getmtime(SO), _deps_mtime()):
         cmd = ["nvcc", "-std=c++17", "-O2", "-Wno-deprecated-gpu-targets", "-o", DAEMON, DAEMON_SRC, "-L" + LIBDIR, "-lblackwell_kernels", "-cudart",
                "shared", "-Xlinker", "-rpath", "-Xlinker", "$ORIGIN"]
         if verbose:

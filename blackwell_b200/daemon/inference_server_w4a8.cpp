@@ -11,7 +11,11 @@
 // the id sampled at the last prompt position and max_tokens more -- and stops after the end-of-text id 151643.
 //
 // usage: inference_server_w4a8 [--weights DIR] [--tokenizer FILE] [--batch B] [--max-seq S] [--act-bits 4|8]
+//                              [--dtype bfloat16|float32] [--eos ID]
 // The model shape is read from the weight files (layer count, hidden size, head counts, intermediate size, vocabulary).
+// DIR may also hold a config.json and a model.safetensors (see bw_decode_create): such models need no tokenizer file --
+// without one, requests carry token ids, {"prompt_ids": [[...], ...], "max_tokens": n}, the answer has no "text", and a
+// sequence ends at --eos (default: never).  --dtype is theirs too.
 #include <cuda_runtime.h>
 #include <stdint.h>
 #include <stdio.h>
@@ -25,6 +29,7 @@
 #include <vector>
 
 #include "../../include/blackwell_b200.h"
+#include "../csrc/json.h"
 
 namespace {
 
@@ -186,6 +191,23 @@ double parse_number(const std::string& json, const char* key, double def) {
     while (p < json.size() && (json[p] == ' ' || json[p] == ':' || json[p] == '"')) ++p;
     return p < json.size() ? strtod(json.c_str() + p, nullptr) : def;
 }
+// {"prompt_ids": [[...], ...]}: false if the request has none or an id is not in [0, vocab).
+bool parse_prompt_ids(const std::string& line, int vocab, std::vector<std::vector<int>>* out) {
+    bw::Json j;
+    std::string err;
+    if (!bw::Json::parse(line.data(), line.size(), &j, &err)) return false;
+    const bw::Json* p = j.get("prompt_ids");
+    if (!p || p->type != bw::Json::kArray) return false;
+    for (const bw::Json& row : p->arr) {
+        if (row.type != bw::Json::kArray || row.arr.empty()) return false;
+        out->emplace_back();
+        for (const bw::Json& v : row.arr) {
+            if (!v.is_int() || v.num < 0 || v.num >= vocab) return false;
+            out->back().push_back((int)v.num);
+        }
+    }
+    return true;
+}
 std::string json_escape(const std::string& s) {
     std::string r;
     for (unsigned char c : s) {
@@ -206,7 +228,7 @@ constexpr int kEos = 151643;
 
 int main(int argc, char** argv) {
     std::string weights = "weights_int4_qwen3_8b", tok_path = "tokenizer_data.bin";
-    int batch = 8, max_seq = 4096, act_bits = 8, max_new_cap = 512;
+    int batch = 8, max_seq = 4096, act_bits = 8, max_new_cap = 512, eos = -2, f32 = 0;
     for (int i = 1; i + 1 < argc; i += 2) {
         const std::string k = argv[i];
         if (k == "--weights") weights = argv[i + 1];
@@ -214,33 +236,47 @@ int main(int argc, char** argv) {
         else if (k == "--batch") batch = atoi(argv[i + 1]);
         else if (k == "--max-seq") max_seq = atoi(argv[i + 1]);
         else if (k == "--act-bits") act_bits = atoi(argv[i + 1]);
+        else if (k == "--eos") eos = atoi(argv[i + 1]);
+        else if (k == "--dtype" && (!strcmp(argv[i + 1], "float32") || !strcmp(argv[i + 1], "bfloat16"))) f32 = argv[i + 1][0] == 'f';
         else { fprintf(stderr, "unknown option %s\n", k.c_str()); return 2; }
     }
+    FILE* config = fopen((weights + "/config.json").c_str(), "rb");
+    const bool layered = config != nullptr;
+    if (config) fclose(config);
     Tokenizer tok;
-    if (!tok.load(tok_path.c_str())) { fprintf(stderr, "FAIL: cannot read %s\n", tok_path.c_str()); return 1; }
+    const bool text = tok.load(tok_path.c_str());
+    if (!text && !layered) { fprintf(stderr, "FAIL: cannot read %s\n", tok_path.c_str()); return 1; }
+    if (eos == -2) eos = layered ? -1 : kEos;
 
     // model shape from the files
     bw_decode_config cfg;
     memset(&cfg, 0, sizeof cfg);
-    int K = 0, N = 0;
-    if (bw_w4_file_dims((weights + "/0_self_attn.q_proj").c_str(), &K, &N) != 0) { fprintf(stderr, "FAIL: no weights in %s\n", weights.c_str()); return 1; }
-    cfg.hidden = K; cfg.n_q_heads = N / 128;
-    if (bw_w4_file_dims((weights + "/0_self_attn.k_proj").c_str(), &K, &N) != 0) return 1;
-    cfg.n_kv_heads = N / 128;
-    if (bw_w4_file_dims((weights + "/0_mlp.gate_proj").c_str(), &K, &N) != 0) return 1;
-    cfg.inter = N;
-    if (bw_w4_file_dims((weights + "/embed_tokens").c_str(), &K, &N) != 0) return 1;
-    cfg.vocab = N;
-    int layers = 0;
-    while (bw_w4_file_dims((weights + "/" + std::to_string(layers) + "_self_attn.q_proj").c_str(), &K, &N) == 0) ++layers;
-    cfg.layers = layers; cfg.head_dim = 128; cfg.eps = 1e-6f; cfg.rope_base = 1000000.0f;
+    if (!layered) {
+        int K = 0, N = 0;
+        if (bw_w4_file_dims((weights + "/0_self_attn.q_proj").c_str(), &K, &N) != 0) { fprintf(stderr, "FAIL: no weights in %s\n", weights.c_str()); return 1; }
+        cfg.hidden = K; cfg.n_q_heads = N / 128;
+        if (bw_w4_file_dims((weights + "/0_self_attn.k_proj").c_str(), &K, &N) != 0) return 1;
+        cfg.n_kv_heads = N / 128;
+        if (bw_w4_file_dims((weights + "/0_mlp.gate_proj").c_str(), &K, &N) != 0) return 1;
+        cfg.inter = N;
+        if (bw_w4_file_dims((weights + "/embed_tokens").c_str(), &K, &N) != 0) return 1;
+        cfg.vocab = N;
+        int layers = 0;
+        while (bw_w4_file_dims((weights + "/" + std::to_string(layers) + "_self_attn.q_proj").c_str(), &K, &N) == 0) ++layers;
+        cfg.layers = layers; cfg.head_dim = 128; cfg.eps = 1e-6f; cfg.rope_base = 1000000.0f;
+    }
     cfg.batch = batch; cfg.max_seq = max_seq; cfg.max_prompt = max_seq; cfg.max_new = max_new_cap;
-    cfg.act_bits = act_bits; cfg.use_graph = 1; cfg.weights_dir = weights.c_str();
-    fprintf(stderr, "Loading %d-layer INT4 model (hidden %d, %d/%d heads, inter %d, vocab %d), batch %d, W4A%d...\n", layers,
-            cfg.hidden, cfg.n_q_heads, cfg.n_kv_heads, cfg.inter, cfg.vocab, batch, act_bits);
+    cfg.act_bits = act_bits; cfg.use_graph = 1; cfg.weights_dir = weights.c_str(); cfg.compute_f32 = layered ? f32 : 0;
+    if (!layered)
+        fprintf(stderr, "Loading %d-layer INT4 model (hidden %d, %d/%d heads, inter %d, vocab %d), batch %d, W4A%d...\n", cfg.layers,
+                cfg.hidden, cfg.n_q_heads, cfg.n_kv_heads, cfg.inter, cfg.vocab, batch, act_bits);
     bw_decode* eng = nullptr;
     const int ce = bw_decode_create(&cfg, &eng);
     if (ce != 0) { fprintf(stderr, "FAIL: bw_decode_create returned %d\n", ce); return 1; }
+    bw_decode_get_config(eng, &cfg);
+    if (layered)
+        fprintf(stderr, "Loaded %d-layer model (hidden %d, vocab %d), batch %d, %s\n", cfg.layers, cfg.hidden, cfg.vocab, batch,
+                f32 ? "float32" : "bfloat16");
     cudaStream_t st;
     if (cudaStreamCreate(&st) != cudaSuccess) return 1;
     fprintf(stderr, "Ready.\n");
@@ -254,7 +290,11 @@ int main(int argc, char** argv) {
         if (line.empty()) continue;
         const int max_tokens = std::min(std::max((int)parse_number(line, "\"max_tokens\"", 30), 1), max_new_cap - 1);
         const double temperature = parse_number(line, "\"temperature\"", 0.0);
-        const std::vector<std::string> prompts = parse_prompts(line);
+        std::vector<std::vector<int>> prompts;
+        const bool by_id = parse_prompt_ids(line, cfg.vocab, &prompts);
+        if (!by_id) prompts.clear();
+        if (!by_id && text)
+            for (const std::string& s : parse_prompts(line)) prompts.push_back(tok.encode(s));
         if (prompts.empty()) { printf("{\"error\":\"no prompts\"}\n"); fflush(stdout); continue; }
         if (temperature >= 0.01) { printf("{\"error\":\"greedy decoding only (temperature 0)\"}\n"); fflush(stdout); continue; }
         std::vector<std::vector<int>> results(prompts.size());
@@ -264,7 +304,7 @@ int main(int argc, char** argv) {
             std::vector<std::vector<int>> ids(batch, std::vector<int>(1, 0));  // idle slots run a one-token dummy
             int longest = 1;
             for (int m = 0; m < n; ++m) {
-                ids[m] = tok.encode(prompts[g0 + m]);
+                ids[m] = prompts[g0 + m];
                 if (ids[m].empty()) ids[m].push_back(0);
                 if ((int)ids[m].size() > max_seq - max_tokens - 1) ids[m].resize(std::max(1, max_seq - max_tokens - 1));
                 longest = std::max(longest, (int)ids[m].size());
@@ -275,8 +315,8 @@ int main(int argc, char** argv) {
                 std::copy(ids[m].begin(), ids[m].end(), table.begin() + (size_t)m * longest);
             }
             int e = bw_decode_begin(eng, table.data(), lens.data(), longest, st);
-            // the longest prompt needs longest + max_tokens steps for its max_tokens + 1 ids
-            for (int s = 0; e == 0 && s < longest + max_tokens; ++s) e = bw_decode_step(eng, st);
+            const int steps = bw_decode_steps(eng, longest, max_tokens + 1);   // for the longest prompt's max_tokens + 1 ids
+            for (int s = 0; e == 0 && s < steps; ++s) e = bw_decode_step(eng, st);
             std::vector<int> gen((size_t)batch * max_new_cap);
             if (e == 0) e = bw_decode_result(eng, gen.data(), st);
             int status = 0;
@@ -287,7 +327,7 @@ int main(int argc, char** argv) {
                     const int id = gen[(size_t)m * max_new_cap + j];
                     if (id < 0) break;
                     results[g0 + m].push_back(id);
-                    if (id == kEos) break;
+                    if (id == eos) break;
                 }
         }
         if (failed) { printf("{\"error\":\"decode failed\"}\n"); fflush(stdout); continue; }
@@ -297,8 +337,8 @@ int main(int argc, char** argv) {
             for (size_t i = 0; i < results[m].size(); ++i) out += (i ? "," : "") + std::to_string(results[m][i]);
             out += "]";
         }
-        out += "],\"text\":[";
-        for (size_t m = 0; m < results.size(); ++m) {
+        out += text ? "],\"text\":[" : "";
+        for (size_t m = 0; text && m < results.size(); ++m) {
             std::string text;
             for (int id : results[m]) text += tok.decode(id);
             out += std::string(m ? "," : "") + "\"" + json_escape(text) + "\"";
