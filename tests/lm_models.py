@@ -109,16 +109,24 @@ class Model:
         return plain.forward(self.cfg, self.w, tokens)
 
     def bar(self, tokens, f32):
-        """Largest error a test accepts: a few times what rounding every product's input to bfloat16 does to the logits of
-        these tokens; for the 32-bit mode the same amplification applied to fp32 roundings."""
+        """Largest error a test accepts: a few times what rounding the inputs and outputs of every product and the outputs of
+        silu to bfloat16 does to the logits of these tokens; for the 32-bit mode the same amplification applied to fp32
+        roundings."""
+        def rounded(x):
+            return to_bf16(x)[1].reshape(np.shape(x))
+
+        def product(W, x):
+            y = linear(W, rounded(x))
+            return y if len(W) == self.cfg["vocab"] else rounded(y)
+
         exact = self.plain(tokens)[0]
-        linear = plain.linear
+        linear, silu = plain.linear, plain.silu
         try:
-            plain.linear = lambda W, x: linear(W, to_bf16(x)[1].reshape(np.shape(x)))
+            plain.linear, plain.silu = product, lambda z: rounded(silu(z))
             noise = rel_error(self.plain(tokens)[0], exact).max()
         finally:
-            plain.linear = linear
-        return 4 * noise * (2.0 ** -12 if f32 else 1.0)
+            plain.linear, plain.silu = linear, silu
+        return 4 * noise * (2.0 ** -13 if f32 else 1.0)
 
     def greedy(self, prompt, n):
         seq = list(prompt)

@@ -80,7 +80,7 @@ def test_dropin_header_matches_c_header():
     assert cxx and cxx <= c, cxx - c
 
 
-@pytest.mark.skipif(not os.path.isdir(REFERENCE) or shutil.which("nvcc") is None,
+@pytest.mark.skipif(not os.path.isfile(os.path.join(REFERENCE, "include", "blackwell", "kernels.h")) or shutil.which("nvcc") is None,
                     reason="reference sources or nvcc not present on this machine")
 @pytest.mark.parametrize("consumer", ["server/inference_server_int4_batched.cu",
                                       "bench/text_generate_int4_batched.cu"])
