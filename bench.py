@@ -895,6 +895,36 @@ def run_attention_only(args):
             "us_per_launch": us, "kv_bytes": nbytes, "gbs": nbytes / us / 1e3, "device_status": k.device_status()}
 
 
+def run_layered(spec):
+    """Prefill and decode throughput of the config.json model, the roofline fraction of each of its kernels, and the same for
+    the INT4 decode model of that width (which takes prompts token by token: its decode step is its prefill)."""
+    import torch
+
+    from blackwell_b200 import bench_layered as bl
+
+    size, _, part = spec.partition(":")
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    peak, kind = measured_peak()
+    bf16 = int8_tensor_peak_tops()[0] / 2
+    sampler = ClockSampler(0)
+    sampler.start()
+    out = {"option": "layered", "size": size, "hbm_gbs": peak, "bf16_tflops": bf16, "peak_kind": kind, "data": "random weights",
+           "l2": "every timed pass reads more than L2 holds, or rotates over buffers larger than L2"}
+    if part in ("", "model"):
+        out["model"] = bl.model_records(peak, size)
+    if part in ("", "int4"):
+        shape = shapes.VIFIVIK_BENCH[size][1]
+        out["int4"] = [run_decode(shape, b, 2048, 20, dev) for b in (1, 8, 32, 64)]
+    if part in ("", "kernels"):
+        out["kernels"] = bl.linear_records(peak, bf16, size) + bl.recurrence_records(peak, bf16, size) + bl.latent_records(peak, bf16, size)
+    if part in ("", "int4kernels"):
+        out["int4_kernels"] = {"M%d" % m: per_matrix_times(dev, m) for m in (1, 8, 64)}
+        out["int4_attention"] = attention_records(dev)
+    out["clocks"] = sampler.stop()
+    return out
+
+
 def run_timeline(args):
     """Diagnostic, needs a library built with -DBW_GEMV_TIMELINE (BW_NVCC_EXTRA=-DBW_GEMV_TIMELINE python -m
     blackwell_b200._build -f): the small-batch GEMV kernel then stamps %globaltimer at its phase borders for its first,
@@ -972,6 +1002,8 @@ def main():
                     "step is timed as the mean of as many passes as that needs); 0 for profiling runs")
     ap.add_argument("--timeline", default=None, help="diagnostic: per-phase timeline of the small-batch kernel on one "
                     "matrix of the set, NAME[:f16|i8]; needs a library built with -DBW_GEMV_TIMELINE")
+    ap.add_argument("--layered", default=None, help="config.json models (Vifivik layers, random weights) beside the INT4 decode "
+                    "model of the same width: SIZE[:model|kernels|int4|int4kernels], SIZE = 2k or 4k; prints its own JSON line")
     ap.add_argument("--tune", default=None, help="profiling aid: comma list of key=value for bw_set_tuning")
     args = ap.parse_args()
     global _ONLY
@@ -986,6 +1018,9 @@ def main():
         # core (the variable is read when the oracle's OpenMP runtime starts, which has not happened yet)
         os.environ["OMP_NUM_THREADS"] = str(os.cpu_count() or 1)
         run_reference(args, rank)
+        return
+    if args.layered:
+        print(json.dumps(run_layered(args.layered)), flush=True)
         return
     if args.attn_only:
         print(json.dumps(run_attention_only(args)), flush=True)

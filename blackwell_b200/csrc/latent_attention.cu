@@ -3,6 +3,7 @@
 
 #include <mutex>
 
+#include "../../include/blackwell_b200.h"
 #include "host_util.h"
 #include "latent_attention.cuh"
 
@@ -123,3 +124,23 @@ cudaError_t latent_expanded(const LatentArgs& a, const Rows& r, cudaStream_t st)
 
 }  // namespace lm
 }  // namespace bw
+
+extern "C" int bw_latent_attention(const bw_latent_args* a, const bw_rows* rows, int expanded, int f32, void* stream) {
+    if (!a || !rows || rows->T < 1 || a->heads < 1 || a->dim < 1 || a->rot < 1 || a->V < 1 || a->R < 1 || a->rot_dims < 0 ||
+        a->rot_dims > a->rot || a->rot_dims % 2 != 0 || !a->cs || !a->cache || !a->q || !a->gate || !a->Wkv || !a->sink || !a->out ||
+        (a->dkv && !a->dkv_norm) || a->max_seq < 1 || a->ldc < bw::lm::latent_row(a->R, a->rot) || a->ldc % 8 != 0 || a->ldq % 8 != 0 ||
+        a->ldw < bw::lm::pad8(a->R) || a->ldw % 8 != 0 || a->ldout % 8 != 0 || (rows->row_slot && !rows->row_pos) ||
+        (!rows->row_slot && rows->pos0 + rows->T > a->max_seq))
+        return cudaErrorInvalidValue;
+    bw::lm::LatentArgs l{};
+    l.heads = a->heads; l.dim = a->dim; l.rot = a->rot; l.V = a->V; l.R = a->R; l.rot_dims = a->rot_dims; l.scale = a->scale; l.eps = a->eps;
+    l.cs = static_cast<const float2*>(a->cs); l.max_seq = a->max_seq; l.cache = a->cache; l.ldc = a->ldc; l.q = a->q; l.ldq = a->ldq;
+    l.dkv = a->dkv; l.gate = a->gate; l.ld32 = a->ld32; l.dkv_norm = a->dkv_norm; l.Wkv = reinterpret_cast<const bw::lm::bf16*>(a->Wkv);
+    l.ldw = a->ldw; l.sink = a->sink; l.out = a->out; l.ldout = a->ldout; l.qabs = a->qabs; l.part = a->part; l.splits = a->splits; l.kv = a->kv;
+    const bw::lm::Rows w{rows->T, rows->row_slot, rows->row_pos, rows->slot, rows->pos0};
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (expanded)
+        return f32 || !a->kv || !bw::lm::latent_expanded_supported(l) ? cudaErrorInvalidValue : bw::lm::latent_expanded(l, w, st);
+    if (!a->qabs || !a->part || a->splits < 1 || !bw::lm::latent_absorbed_supported(l)) return cudaErrorInvalidValue;
+    return bw::lm::latent_absorbed(l, w, f32, st);
+}

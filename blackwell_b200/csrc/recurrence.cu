@@ -3,6 +3,7 @@
 
 #include <mutex>
 
+#include "../../include/blackwell_b200.h"
 #include "host_util.h"
 #include "recurrence.cuh"
 
@@ -57,3 +58,18 @@ cudaError_t recurrence_chunk(const RecurrenceArgs& a, const Rows& r, cudaStream_
 
 }  // namespace lm
 }  // namespace bw
+
+extern "C" int bw_linear_recurrence(const bw_recurrence_args* a, const bw_rows* rows, int chunked, int f32, void* stream) {
+    if (!a || !rows || rows->T < 1 || !a->q || !a->k || !a->v || !a->S || !a->o || a->heads < 1 || a->N < 1 || a->V < 1 ||
+        a->groups < 1 || (a->log_decay ? !a->weight : !a->head_log_decay) || (rows->row_slot && !rows->row_pos) ||
+        a->ldq % 8 != 0 || a->ldk % 8 != 0 || a->ldv % 8 != 0 || a->ldo % 8 != 0)
+        return cudaErrorInvalidValue;
+    bw::lm::RecurrenceArgs r{};
+    r.q = a->q; r.k = a->k; r.v = a->v; r.ldq = a->ldq; r.ldk = a->ldk; r.ldv = a->ldv; r.heads = a->heads; r.N = a->N; r.V = a->V;
+    r.groups = a->groups; r.log_decay = a->log_decay; r.weight = a->weight; r.head_log_decay = a->head_log_decay;
+    r.const_weight = a->const_weight; r.D = a->D; r.S = a->S; r.o = a->o; r.ldo = a->ldo;
+    const bw::lm::Rows w{rows->T, rows->row_slot, rows->row_pos, rows->slot, rows->pos0};
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (chunked) return f32 ? cudaErrorInvalidValue : bw::lm::recurrence_chunk(r, w, st);
+    return bw::lm::recurrence_step(r, nullptr, w, f32, st);
+}

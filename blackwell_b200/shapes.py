@@ -60,3 +60,25 @@ def gemv_bytes(N: int, K: int, M: int, w_scale_bytes: int = 2, x_kind: str = "f1
     else:
         raise ValueError(x_kind)
     return w + x + M * N * 4
+
+
+def vifivik_config(width: int, ff: int, vocab: int, layers: int, head_scale: int) -> dict:
+    """A Vifivik configuration with the layer sizes of a real model (random weights, benchmark only): the pattern mamba2,
+    latent attention, latent attention on that cache, retention.  head_scale = width / 2048."""
+    mamba = {"heads": 64 * head_scale, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}
+    latent = {"heads": 16 * head_scale, "dim": 128, "rot_dim": 64, "kv_rank": 512, "vdim": 128, "scale": 192 ** -0.5,
+              "rot": {"base": 10000.0, "dims": 64}}
+    ret = {"heads": 8 * head_scale, "dim": 256, "vdim": 512, "decay": [1 - 2.0 ** -(5 + i % 8) for i in range(8 * head_scale)]}
+    out = []
+    for i in range(layers):
+        kind, mixer = [("mamba2", mamba), ("latent_attention", latent), ("latent_attention", {**latent, "kv_from": i - 1}),
+                       ("retention", ret)][i % 4]
+        out.append({"type": kind, "mixer": dict(mixer), "mlp": {"kind": "dense", "ff": ff}})
+    return {"architecture": "Vifivik", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "layers": out}
+
+
+# name -> (config.json model, the INT4 decode model of the same width, feed-forward size, layer count and vocabulary)
+VIFIVIK_BENCH = {
+    "2k": (vifivik_config(2048, 5632, 32768, 8, 1), ModelShape("int4-2k", 8, 2048, 5632, 16, 4, 128, 32768)),
+    "4k": (vifivik_config(4096, 12288, 65536, 8, 2), ModelShape("int4-4k", 8, 4096, 12288, 32, 8, 128, 65536)),
+}

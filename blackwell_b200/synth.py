@@ -74,3 +74,60 @@ def activations_f16_device(M: int, K: int, seed: int, device="cuda"):
     x = torch.empty((M, K), dtype=torch.float32, device=device)
     x.normal_(0.0, 1.0, generator=gen)
     return x.to(torch.float16)
+
+
+def write_random_model(directory: str, cfg: dict, seed: int = 0, device="cuda") -> int:
+    """A config.json model with random bfloat16 weights (values scaled by fan-in); returns the bytes of its matrices."""
+    import json
+    import os
+    import struct
+
+    import torch
+
+    W, V = cfg["width"], cfg["vocab"]
+    shapes = {"embed": (V, W), "head": (V, W), "final.norm": (W,)}
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        q, H, vd = p + "mix.", m["heads"], m["vdim"]
+        shapes[p + "norm1"] = (W,)
+        if L["type"] == "mamba2":
+            inner, gn = H * vd, m["groups"] * m["state"]
+            shapes.update({q + "in": (2 * inner + 2 * gn + H, W), q + "conv": (inner + 2 * gn, m["conv"]), q + "conv.b": (inner + 2 * gn,),
+                           q + "dt_bias": (H,), q + "A_log": (H,), q + "D": (H,), q + "norm": (inner,)})
+        elif L["type"] == "retention":
+            shapes.update({q + "q": (H * m["dim"], W), q + "k": (H * m["dim"], W), q + "v": (H * vd, W), q + "g": (H * vd, W)})
+        else:
+            R, rot = m["kv_rank"], m["rot_dim"]
+            shapes.update({q + "q": (H * (m["dim"] + rot), W), q + "uk": (H * m["dim"], R), q + "uv": (H * vd, R), q + "sink": (H,),
+                           q + "g": (H, W)})
+            if "kv_from" not in m:
+                shapes.update({q + "dkv": (R + rot, W), q + "dkv.norm": (R,)})
+        shapes[q + "o"] = (W, H * vd)
+        if L["mlp"]:
+            ff = L["mlp"]["ff"]
+            shapes.update({p + "norm2": (W,), p + "mlp.gate": (ff, W), p + "mlp.up": (ff, W), p + "mlp.down": (W, ff)})
+    header, at, matrices = {}, 0, 0
+    for name, shape in shapes.items():
+        n = 2 * int(np.prod(shape))
+        header[name] = {"dtype": "BF16", "shape": list(shape), "data_offsets": [at, at + n]}
+        at += n
+        if len(shape) == 2 and not name.endswith(".conv") and name != "embed":
+            matrices += n
+    gen = torch.Generator(device=device).manual_seed(seed)
+    os.makedirs(directory, exist_ok=True)
+    with open(os.path.join(directory, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    head = json.dumps(header).encode()
+    head += b" " * (-len(head) % 8)
+    with open(os.path.join(directory, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(head)) + head)
+        for name, shape in shapes.items():
+            t = torch.randn(shape, generator=gen, device=device)
+            if len(shape) == 2 and name != "embed":
+                t *= shape[1] ** -0.5
+            elif name.endswith(("norm", "norm1", "norm2")):
+                t = 1.0 + 0.1 * t
+            elif name.endswith("dt_bias"):
+                t = t - 4.0
+            f.write(t.to(torch.bfloat16).view(torch.int16).cpu().numpy().tobytes())
+    return matrices

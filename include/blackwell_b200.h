@@ -401,6 +401,62 @@ int bw_decode_watch_layers(bw_decode* d, float* buffer, long rows);
 int bw_linear_bf16(void* y, long ldy, const void* x, long ldx, const uint16_t* W, long ldw, int T, int N, int K,
                    int y_f32, int x_f32, int epilogue, float softcap, void* stream);
 
+/* Rows of a call: one token each of T sequences (row_slot / row_pos on the device), or -- row_slot NULL -- T consecutive
+ * tokens of the sequence in `slot`, at pos0, pos0 + 1, ...  Per-head blocks of every operand below are padded to multiples
+ * of 8 columns (P8); padding is zero.  Element type: bfloat16, or fp32 with f32 != 0. */
+typedef struct bw_rows {
+    int T;
+    const int *row_slot, *row_pos;
+    int slot, pos0;
+} bw_rows;
+/* Gated linear recurrence with an fp32 state per head, S [slot][heads][N][P8(V)]:
+ *   S_t = exp(log_decay) S_(t-1) + weight k_t v_t^T,  o_t = S_t^T q_t + D v_t;  a sequence's state is zero before position 0.
+ * q, k: head h at column (h / (heads / groups)) * P8(N); v, o: at h * P8(V).  log_decay / weight [T][heads] fp32, or NULL:
+ * head_log_decay [heads] and const_weight.  N <= 512.  chunked: 64 tokens at a time on the tensor cores (bfloat16, rows of
+ * one sequence, N <= 256); otherwise token by token. */
+typedef struct bw_recurrence_args {
+    const void *q, *k, *v;
+    long ldq, ldk, ldv;
+    int heads, N, V, groups;
+    const float *log_decay, *weight, *head_log_decay;
+    float const_weight;
+    const float* D;
+    float* S;
+    float* o;
+    long ldo;
+} bw_recurrence_args;
+int bw_linear_recurrence(const bw_recurrence_args* a, const bw_rows* rows, int chunked, int f32, void* stream);
+/* Latent attention: a position is cached as [latent (R) | rotated key part (rot)], blocks padded to P8, one vector for all
+ * heads.  q [T][heads * (P8(dim) + P8(rot))] (the expanded form rotates it in place), dkv [T][ld32] the latent before its
+ * norm and the key part before rotation (NULL: the rows are in the cache already), gate [T][ld32] one logit per head,
+ * Wkv rows uk (head h at h * P8(dim)) then uv, cs cos / sin [max_seq][rot_dims / 2], sink [heads];
+ * out [T][heads * P8(V)] = sigmoid(gate) * softmax-with-sink attention.  Scratch: absorbed form qabs
+ * (4 * T * heads * P16(P8(R) + P8(rot)) bytes) and part (T * heads * splits * (R + 2) floats); expanded form kv
+ * (max_seq * heads * (P8(dim) + P8(V)) elements; bfloat16, rows of one sequence only). */
+typedef struct bw_latent_args {
+    int heads, dim, rot, V, R, rot_dims;
+    float scale, eps;
+    const void* cs;
+    int max_seq;
+    void* cache;
+    long ldc;
+    void* q;
+    long ldq;
+    const float *dkv, *gate;
+    long ld32;
+    const float* dkv_norm;
+    const uint16_t* Wkv;
+    long ldw;
+    const float* sink;
+    void* out;
+    long ldout;
+    void* qabs;
+    float* part;
+    int splits;
+    void* kv;
+} bw_latent_args;
+int bw_latent_attention(const bw_latent_args* a, const bw_rows* rows, int expanded, int f32, void* stream);
+
 /* ---- Tensor-parallel exchange over peer memory (no counterpart in the reference, which is single-GPU) ----
  * All-reduce of the K-split projections' partial sums across the GPUs of one box through NVLink peer loads.
  * bw_peer_comm_create allocates this rank's region on the current device (two slots of slot_bytes; the GEMV writes
