@@ -157,10 +157,10 @@ def latent_records(peak, bf16_peak, size):
         nw, sink, cs = torch.ones(R, device="cuda"), torch.zeros(H, device="cuda"), torch.ones((ctx, rot // 2, 2), device="cuda") * 0.7
         wkv = torch.randn((H * (dim + V), R), device="cuda", dtype=torch.bfloat16) * R ** -0.5
         o = torch.empty((M, H * V), device="cuda", dtype=torch.bfloat16)
-        splits = max(1, min(64, ctx // 128, 148 // (M * -(-H // 16))))
+        splits = max(1, min(64, ctx // 64, 148 // (M * -(-H // 16))))
         rows = M if not expanded else 1
         qabs = torch.empty((rows * H * 2 * D,), device="cuda", dtype=torch.bfloat16)
-        part = torch.empty((rows * H * splits * (R + 2),), device="cuda")
+        part = torch.empty((rows * H * splits * (R + 4),), device="cuda")
         kv = torch.empty((ctx if expanded else 1, H * (dim + V)), device="cuda", dtype=torch.bfloat16)
         ids = torch.arange(slots, device="cuda", dtype=torch.int32)
         pos = torch.full((slots,), ctx - 1, device="cuda", dtype=torch.int32)

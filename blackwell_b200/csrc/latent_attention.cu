@@ -23,22 +23,22 @@ cudaError_t prep(const LatentArgs& a, const Rows& r, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
     cudaError_t e = allow_smem(latent_prep_kernel<A, RB>, once);
     if (e != cudaSuccess) return e;
-    const int nc = pad8(a.R) / 8, groups = std::max(1, kPrepThreads / nc);
-    const size_t smem = std::max<size_t>(128, (size_t)(RB * (pad8(a.dim) + pad8(a.rot)) + groups * RB * pad8(a.R)) * 4);
+    const int cblocks = (pad8(a.R) + kPrepCols - 1) / kPrepCols;
+    const size_t smem = (size_t)(RB * (pad8(a.dim) + pad8(a.rot)) + 8 * RB * kPrepCols) * 4;
     if (smem > kMaxDynSmem) return cudaErrorInvalidValue;
     count_launch(1);
-    return launch_pdl(latent_prep_kernel<A, RB>, dim3(a.heads + (a.dkv ? 1 : 0), (r.T + RB - 1) / RB), dim3(kPrepThreads), smem, st, a, r);
+    return launch_pdl(latent_prep_kernel<A, RB>, dim3(a.heads * cblocks + (a.dkv ? RB : 0), (r.T + RB - 1) / RB), dim3(kPrepThreads), smem, st, a, r);
 }
 
 template <typename A, int RB>
-cudaError_t out(const LatentArgs& a, const Rows& r, cudaStream_t st) {
+cudaError_t out(const LatentArgs& a, const Rows& r, int keys, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
     cudaError_t e = allow_smem(latent_out_kernel<A, RB>, once);
     if (e != cudaSuccess) return e;
-    const size_t smem = (size_t)(RB * pad8(a.R) + RB * a.splits) * 4;
+    const size_t smem = (size_t)(2 * RB * pad8(a.R) + ((RB * a.splits + 3) & ~3)) * 4;
     if (smem > kMaxDynSmem) return cudaErrorInvalidValue;
     count_launch(1);
-    return launch_pdl(latent_out_kernel<A, RB>, dim3(a.heads, (r.T + RB - 1) / RB), dim3(256), smem, st, a, r);
+    return launch_pdl(latent_out_kernel<A, RB>, dim3(a.heads * ((pad8(a.V) + kOutV - 1) / kOutV), (r.T + RB - 1) / RB), dim3(256), smem, st, a, r, keys);
 }
 
 template <typename A>
@@ -58,45 +58,48 @@ cudaError_t decode(const LatentArgs& a, const Rows& r, int nbuf, cudaStream_t st
                       st, a, r, nbuf);
 }
 
-template <int VT>
+template <int VT, int MT>
 cudaError_t flash(const LatentArgs& a, const Rows& r, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
-    cudaError_t e = allow_smem(latent_flash_kernel<VT>, once);
+    auto kern = latent_flash_kernel<VT, MT>;
+    cudaError_t e = allow_smem(kern, once);
     if (e != cudaSuccess) return e;
     const int D = pad16(pad8(a.dim) + pad8(a.rot));
     count_launch(1);
-    return launch_pdl(latent_flash_kernel<VT>, dim3((r.T + kFlashQ - 1) / kFlashQ, a.heads, (pad8(a.V) + VT * 8 - 1) / (VT * 8)), dim3(256),
-                      FlashSmem(D, VT).total, st, a, r);
+    return launch_pdl(kern, dim3((r.T + 128 * MT - 1) / (128 * MT), a.heads, (pad8(a.V) + VT * 8 - 1) / (VT * 8)), dim3(256),
+                      FlashSmem(D, VT, MT).total, st, a, r);
 }
 
+// value columns / 8 per block, 0 if no form fits shared memory
 int flash_vt(const LatentArgs& a) {
     const int D = pad16(pad8(a.dim) + pad8(a.rot));
     int vt = a.V <= 64 ? 8 : a.V <= 128 ? 16 : 32;
-    while (vt > 8 && FlashSmem(D, vt).total > kMaxDynSmem) vt /= 2;
-    return FlashSmem(D, vt).total <= kMaxDynSmem ? vt : 0;
+    while (vt > 8 && FlashSmem(D, vt, 1).total > kMaxDynSmem) vt /= 2;
+    return FlashSmem(D, vt, 1).total <= kMaxDynSmem ? vt : 0;
 }
 
 }  // namespace
 
 bool latent_absorbed_supported(const LatentArgs& a) {
-    const int nc = pad8(a.R) / 8, groups = std::max(1, kPrepThreads / nc);
-    return a.R >= 1 && a.R <= 2048 && (size_t)(pad8(a.dim) + pad8(a.rot) + groups * pad8(a.R)) * 4 <= (size_t)kMaxDynSmem;
+    return a.R >= 1 && a.R <= 2048 && (size_t)(pad8(a.dim) + pad8(a.rot) + 8 * kPrepCols) * 4 <= (size_t)kMaxDynSmem;
 }
 bool latent_expanded_supported(const LatentArgs& a) { return flash_vt(a) > 0; }
 
 cudaError_t latent_absorbed(const LatentArgs& a, const Rows& r, int f32, cudaStream_t st) {
-    const bool rb4 = r.T >= 8 && !f32 && a.R <= 512;
+    const bool rb4 = r.T >= 8 && !f32 && a.R <= 1024 && (pad8(a.dim) + pad8(a.rot)) <= 1024;
     cudaError_t e = f32 ? prep<float, 1>(a, r, st) : rb4 ? prep<bf16, 4>(a, r, st) : prep<bf16, 1>(a, r, st);
     if (e != cudaSuccess) return e;
     const int nbuf = DecodeSmem(a.R, a.rot, 2).total <= kMaxDynSmem ? 2 : 1;
+    const bool by_scalar = f32 || a.R > 1024 || DecodeSmem(a.R, a.rot, nbuf).total > kMaxDynSmem;
+    const int keys = by_scalar ? kScalarKeys : kDecKeys;
     if (f32) e = scalar<float>(a, r, st);
-    else if (a.R > 1024 || DecodeSmem(a.R, a.rot, nbuf).total > kMaxDynSmem) e = scalar<bf16>(a, r, st);
+    else if (by_scalar) e = scalar<bf16>(a, r, st);
     else if (a.R <= 128) e = decode<2>(a, r, nbuf, st);
     else if (a.R <= 256) e = decode<4>(a, r, nbuf, st);
     else if (a.R <= 512) e = decode<8>(a, r, nbuf, st);
     else e = decode<16>(a, r, nbuf, st);
     if (e != cudaSuccess) return e;
-    return f32 ? out<float, 1>(a, r, st) : rb4 ? out<bf16, 4>(a, r, st) : out<bf16, 1>(a, r, st);
+    return f32 ? out<float, 1>(a, r, keys, st) : rb4 ? out<bf16, 4>(a, r, keys, st) : out<bf16, 1>(a, r, keys, st);
 }
 
 cudaError_t latent_expanded(const LatentArgs& a, const Rows& r, cudaStream_t st) {
@@ -119,7 +122,11 @@ cudaError_t latent_expanded(const LatentArgs& a, const Rows& r, cudaStream_t st)
     e = linear(x, st);
     if (e != cudaSuccess) return e;
     const int vt = flash_vt(a);
-    return vt == 8 ? flash<8>(a, r, st) : vt == 16 ? flash<16>(a, r, st) : vt == 32 ? flash<32>(a, r, st) : cudaErrorInvalidValue;
+    // 256 query rows per block where that still gives every SM a block
+    const bool tall = vt <= 16 && FlashSmem(pad16(pad8(a.dim) + pad8(a.rot)), vt, 2).total <= kMaxDynSmem &&
+                      (r.T + 255) / 256 * a.heads >= sm_count(current_device());
+    if (tall) return vt == 8 ? flash<8, 2>(a, r, st) : flash<16, 2>(a, r, st);
+    return vt == 8 ? flash<8, 1>(a, r, st) : vt == 16 ? flash<16, 1>(a, r, st) : vt == 32 ? flash<32, 1>(a, r, st) : cudaErrorInvalidValue;
 }
 
 }  // namespace lm

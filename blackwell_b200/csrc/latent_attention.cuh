@@ -69,22 +69,34 @@ __global__ void __launch_bounds__(128) latent_rotate_q_kernel(const LatentArgs a
 
 // ------------------------------------------------------------------------------------------ absorbed form
 constexpr int kPrepThreads = 256;
+constexpr int kPrepCols = 64;    // latent columns per block
 
-// Block (head, group of RB rows): q_abs = W_uk^T q and the rotated part.  One more block per row group writes the cache.
+// Block (head, 64 latent columns; RB rows): q_abs = W_uk^T q, and from the first column block the rotated part.  RB more
+// blocks per row group write the cache entries.  8 threads cover the columns, 32 groups of threads the query dimensions;
+// the weights are fetched before the kernel waits for its predecessor.
 template <typename A, int RB>
 __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentArgs a, const Rows r) {
     extern __shared__ float sm[];
-    const int h = blockIdx.x, row0 = blockIdx.y * RB, t = threadIdx.x;
+    const int dim8 = pad8(a.dim), rot8 = pad8(a.rot), R8 = pad8(a.R), Dp = latent_dp(a.R, a.rot);
+    const int cblocks = (R8 + kPrepCols - 1) / kPrepCols, t = threadIdx.x, warp = t >> 5, lane = t & 31;
+    const int h = blockIdx.x / cblocks, cb = blockIdx.x - h * cblocks, row0 = blockIdx.y * RB;
     pdl_trigger();
-    pdl_wait();
-    if (h == a.heads) {
-        for (int b = 0; b < RB; ++b)
-            if (row0 + b < r.T) write_entry<A>(a, r, row0 + b, sm);
+    if (h >= a.heads) {
+        pdl_wait();
+        const int row = row0 + (int)blockIdx.x - a.heads * cblocks;
+        if (row < r.T) write_entry<A>(a, r, row, sm);
         return;
     }
-    const int dim8 = pad8(a.dim), rot8 = pad8(a.rot), R8 = pad8(a.R), Dp = latent_dp(a.R, a.rot), nc = R8 / 8;
-    float* qs = sm;                         // [RB][dim8 + rot8]
-    float* red = qs + RB * (dim8 + rot8);   // [groups][RB][R8]
+    constexpr int kPre = 4;
+    const int col = cb * kPrepCols + (lane & 7) * 8, grp = warp * 4 + (lane >> 3);
+    const bf16* W = a.Wkv + (long)h * dim8 * a.ldw + col;
+    uint4 pre[kPre];
+#pragma unroll
+    for (int i = 0; i < kPre; ++i)
+        pre[i] = col < R8 && grp + 32 * i < a.dim ? __ldg(reinterpret_cast<const uint4*>(W + (long)(grp + 32 * i) * a.ldw)) : make_uint4(0, 0, 0, 0);
+    pdl_wait();
+    float* qs = sm;                                   // [RB][dim8 + rot8]
+    float* red = qs + RB * (dim8 + rot8);             // [8 warps][RB][kPrepCols]
     for (int i = t; i < RB * (dim8 + rot8); i += kPrepThreads) {
         const int b = i / (dim8 + rot8), d = i - b * (dim8 + rot8);
         float v = 0.f;
@@ -100,43 +112,41 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentA
         qs[i] = v;
     }
     __syncthreads();
-    const int groups = max(1, kPrepThreads / nc), grp = t / nc;
-    if (grp < groups || nc > kPrepThreads) {
-        for (int c = nc > kPrepThreads ? t : t % nc; c < nc; c += nc > kPrepThreads ? kPrepThreads : nc) {
-            float acc[RB][8] = {};
-            const bf16* W = a.Wkv + (long)h * dim8 * a.ldw + c * 8;
-#pragma unroll 8
-            for (int d = nc > kPrepThreads ? 0 : grp; d < a.dim; d += groups) {
-                const uint4 w = __ldg(reinterpret_cast<const uint4*>(W + (long)d * a.ldw));
-                const uint32_t ww[4] = {w.x, w.y, w.z, w.w};
+    float acc[RB][8] = {};
+    auto add = [&](const uint4& w, int d) {
+        const uint32_t ww[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
-                for (int b = 0; b < RB; ++b) {
-                    const float q = qs[b * (dim8 + rot8) + d];
+        for (int b = 0; b < RB; ++b) {
+            const float q = qs[b * (dim8 + rot8) + d];
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) {
-                        acc[b][2 * j] = fmaf(q, __uint_as_float(ww[j] << 16), acc[b][2 * j]);
-                        acc[b][2 * j + 1] = fmaf(q, __uint_as_float(ww[j] & 0xFFFF0000u), acc[b][2 * j + 1]);
-                    }
-                }
+            for (int j = 0; j < 4; ++j) {
+                acc[b][2 * j] = fmaf(q, __uint_as_float(ww[j] << 16), acc[b][2 * j]);
+                acc[b][2 * j + 1] = fmaf(q, __uint_as_float(ww[j] & 0xFFFF0000u), acc[b][2 * j + 1]);
             }
+        }
+    };
 #pragma unroll
-            for (int b = 0; b < RB; ++b) {
-                float* o = red + ((long)(nc > kPrepThreads ? 0 : grp) * RB + b) * R8 + c * 8;
-                *reinterpret_cast<float4*>(o) = make_float4(acc[b][0], acc[b][1], acc[b][2], acc[b][3]);
-                *reinterpret_cast<float4*>(o + 4) = make_float4(acc[b][4], acc[b][5], acc[b][6], acc[b][7]);
-            }
+    for (int i = 0; i < kPre; ++i)
+        if (grp + 32 * i < a.dim) add(pre[i], grp + 32 * i);
+    if (col < R8)
+        for (int d = grp + 32 * kPre; d < a.dim; d += 32) add(__ldg(reinterpret_cast<const uint4*>(W + (long)d * a.ldw)), d);
+#pragma unroll
+    for (int b = 0; b < RB; ++b)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            acc[b][j] += __shfl_xor_sync(0xffffffffu, acc[b][j], 8);
+            acc[b][j] += __shfl_xor_sync(0xffffffffu, acc[b][j], 16);
+        }
+    if (lane < 8) {
+#pragma unroll
+        for (int b = 0; b < RB; ++b) {
+            float* o = red + (warp * RB + b) * kPrepCols + lane * 8;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) o[j] = acc[b][j];
         }
     }
     __syncthreads();
-    for (int i = t; i < RB * Dp; i += kPrepThreads) {
-        const int b = i / Dp, d = i - b * Dp;
-        if (row0 + b >= r.T) break;
-        float v = 0.f;
-        if (d < R8) {
-            for (int g = 0; g < groups; ++g) v += red[((long)g * RB + b) * R8 + d];
-        } else if (d < R8 + rot8) {
-            v = qs[b * (dim8 + rot8) + dim8 + (d - R8)];
-        }
+    auto put = [&](int b, int d, float v) {
         const long base = ((long)(row0 + b) * a.heads + h);
         if (sizeof(A) == 4) {
             static_cast<float*>(a.qabs)[base * Dp + d] = v;
@@ -146,12 +156,30 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentA
             o[0] = hi;
             o[Dp] = __float2bfloat16_rn(v - __bfloat162float(hi));
         }
+    };
+    for (int i = t; i < RB * kPrepCols; i += kPrepThreads) {
+        const int b = i / kPrepCols, c = i - b * kPrepCols;
+        if (row0 + b >= r.T || cb * kPrepCols + c >= R8) continue;
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) v += red[(w * RB + b) * kPrepCols + c];
+        put(b, cb * kPrepCols + c, v);
     }
+    if (cb == 0)
+        for (int i = t; i < RB * (Dp - R8); i += kPrepThreads) {
+            const int b = i / (Dp - R8), e = i - b * (Dp - R8);
+            if (row0 + b < r.T) put(b, R8 + e, e < rot8 ? qs[b * (dim8 + rot8) + dim8 + e] : 0.f);
+        }
 }
 
-// One partial result per (row, head, split): R un-normalised outputs, then the running maximum and the sum.
+// One partial result per (row, head, split): pad8(R) un-normalised outputs, then the running maximum and the sum.
 __device__ __forceinline__ float* part_ptr(const LatentArgs& a, int row, int h, int split) {
-    return a.part + (((long)row * a.heads + h) * a.splits + split) * (a.R + 2);
+    return a.part + (((long)row * a.heads + h) * a.splits + split) * (pad8(a.R) + kPartStats);
+}
+// Splits of a context of `len` positions that hold any (tiles of `keys` are dealt out in runs of equal length).
+__device__ __forceinline__ int used_splits(int len, int keys, int splits) {
+    const int tiles = (len + keys - 1) / keys, per = (tiles + splits - 1) / splits;
+    return (tiles + per - 1) / per;
 }
 
 // Scalar kernel (32-bit mode; latent sizes the tensor-core kernel does not take): block (split, head, row).
@@ -168,12 +196,10 @@ __global__ void __launch_bounds__(256) latent_scalar_kernel(const LatentArgs a, 
     pdl_wait();
     const int slot = r.slot_of(row), len = min(r.pos_of(row) + 1, a.max_seq);
     float* out = part_ptr(a, row, h, split);
+    float* stats = out + R8;
     const int tiles = (len + kScalarKeys - 1) / kScalarKeys, per = (tiles + a.splits - 1) / a.splits;
     const int k0 = min(split * per * kScalarKeys, len), k1 = min((split + 1) * per * kScalarKeys, len);
-    if (slot < 0 || k0 >= k1) {
-        if (t == 0) { out[a.R] = -INFINITY; out[a.R + 1] = 0.f; }
-        return;
-    }
+    if (slot < 0 || k0 >= k1) return;   // the merge reads the splits that hold positions
     const long base = (long)row * a.heads + h;
     for (int i = t; i < Dp; i += 256)
         q[i] = sizeof(A) == 4 ? static_cast<const float*>(a.qabs)[base * Dp + i]
@@ -205,14 +231,14 @@ __global__ void __launch_bounds__(256) latent_scalar_kernel(const LatentArgs a, 
             const A* e = cache + (long)(kt + j) * a.ldc;
 #pragma unroll
             for (int c = 0; c < kCols; ++c)
-                if (c * 256 + t < a.R) acc[c] = fmaf(p, to_f(e[c * 256 + t]), acc[c]);
+                if (c * 256 + t < R8) acc[c] = fmaf(p, to_f(e[c * 256 + t]), acc[c]);
         }
         m = mn;
     }
 #pragma unroll
     for (int c = 0; c < kCols; ++c)
-        if (c * 256 + t < a.R) out[c * 256 + t] = acc[c];
-    if (t == 0) { out[a.R] = m; out[a.R + 1] = l; }
+        if (c * 256 + t < R8) out[c * 256 + t] = acc[c];
+    if (t == 0) { stats[0] = m; stats[1] = l; }
 }
 
 constexpr int kDecKeys = 64;
@@ -247,14 +273,7 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
     const int slot = r.slot_of(row), len = min(r.pos_of(row) + 1, a.max_seq);
     const int tiles = (len + kDecKeys - 1) / kDecKeys, per = (tiles + a.splits - 1) / a.splits;
     const int t0 = split * per, t1 = min(tiles, t0 + per);
-    if (slot < 0 || t0 >= t1) {
-        if (t < 16 && h0 + t < a.heads) {
-            float* out = part_ptr(a, row, h0 + t, split);
-            out[a.R] = -INFINITY;
-            out[a.R + 1] = 0.f;
-        }
-        return;
-    }
+    if (slot < 0 || t0 >= t1) return;   // the merge reads the splits that hold positions
     const bf16* cache = static_cast<const bf16*>(a.cache) + (long)slot * a.max_seq * a.ldc;
     const int nc = Dp / 8;
     auto issue = [&](int tile, int buf) {
@@ -280,19 +299,36 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
         cp_async_wait<0>();
         __syncthreads();
         if (nbuf == 2 && tile + 1 < t1) issue(tile + 1, buf ^ 1);
-        float s[4] = {}, sl[4] = {};
-        for (int k0 = 0; k0 < Dp; k0 += 16) {
+        float s[4] = {}, sl[4] = {}, s2[4] = {}, sl2[4] = {};   // four independent chains
+        const uint32_t qa = sb + L.q_off + (lane & 15) * L.row + (lane >> 4) * 16;
+        const uint32_t ka = kb + (8 * warp + (lane & 7)) * L.row + (lane >> 3) * 16;
+        int k0 = 0;
+#pragma unroll 4
+        for (; k0 + 32 <= Dp; k0 += 32) {
+            uint32_t ah[4], al[4], bh[4], bl[4], b[4];
+            ldsm4(ka + k0 * 2, b);
+            ldsm4(qa + k0 * 2, ah);
+            ldsm4(qa + 16 * L.row + k0 * 2, al);
+            ldsm4(qa + k0 * 2 + 32, bh);
+            ldsm4(qa + 16 * L.row + k0 * 2 + 32, bl);
+            mma_bf16(s, ah[0], ah[1], ah[2], ah[3], b[0], b[1]);
+            mma_bf16(sl, al[0], al[1], al[2], al[3], b[0], b[1]);
+            mma_bf16(s2, bh[0], bh[1], bh[2], bh[3], b[2], b[3]);
+            mma_bf16(sl2, bl[0], bl[1], bl[2], bl[3], b[2], b[3]);
+        }
+        if (k0 < Dp) {
             uint32_t ah[4], al[4], b[2];
-            const uint32_t qa = sb + L.q_off + (lane & 15) * L.row + (k0 + (lane >> 4) * 8) * 2;
-            ldsm4(qa, ah);
-            ldsm4(qa + 16 * L.row, al);
+            ldsm4(qa + k0 * 2, ah);
+            ldsm4(qa + 16 * L.row + k0 * 2, al);
             ldsm2(kb + (8 * warp + (lane & 7)) * L.row + (k0 + ((lane >> 3) & 1) * 8) * 2, b);
             mma_bf16(s, ah[0], ah[1], ah[2], ah[3], b[0], b[1]);
             mma_bf16(sl, al[0], al[1], al[2], al[3], b[0], b[1]);
         }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s[i] = (s[i] + s2[i]) + (sl[i] + sl2[i]);
         const int key = tile * kDecKeys + 8 * warp + 2 * q4;
 #pragma unroll
-        for (int i = 0; i < 4; ++i) s[i] = key + (i & 1) < len ? (s[i] + sl[i]) * a.scale : -INFINITY;
+        for (int i = 0; i < 4; ++i) s[i] = key + (i & 1) < len ? s[i] * a.scale : -INFINITY;
         float x0 = fmaxf(s[0], s[1]), x1 = fmaxf(s[2], s[3]);
 #pragma unroll
         for (int o = 1; o <= 2; o <<= 1) {
@@ -362,122 +398,159 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
             const int col = (warp * NT + j) * 8 + 2 * q4;
-            if (col < a.R) out[col] = O[j][2 * p];
-            if (col + 1 < a.R) out[col + 1] = O[j][2 * p + 1];
+            if (col < R8) *reinterpret_cast<float2*>(out + col) = make_float2(O[j][2 * p], O[j][2 * p + 1]);
         }
         if (warp == 0 && q4 == 0) {
-            out[a.R] = p ? m1 : m0;
-            out[a.R + 1] = p ? l1 : l0;
+            out[R8] = p ? m1 : m0;
+            out[R8 + 1] = p ? l1 : l0;
         }
     }
 }
 
-// Block (head, group of RB rows): merges the splits, adds the sink to the denominator, applies W_uv and the gate.
+constexpr int kOutV = 32;   // value columns per block
+
+// Block (head and 32 value columns, RB rows): merges the splits, adds the sink to the denominator, applies W_uv and the gate.
+// A warp has four value columns; their first weights are fetched before the kernel waits for its predecessor.
 template <typename A, int RB>
-__global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, const Rows r) {
+__global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, const Rows r, int keys) {
     extern __shared__ float sm[];
-    const int R8 = pad8(a.R), dim8 = pad8(a.dim), V8 = pad8(a.V);
+    const int R8 = pad8(a.R), dim8 = pad8(a.dim), V8 = pad8(a.V), nq = R8 / 4;
     float* lat = sm;                     // [RB][R8]
     float* wsp = lat + RB * R8;          // [RB][splits] weights of the splits
-    const int h = blockIdx.x, row0 = blockIdx.y * RB, t = threadIdx.x, warp = t >> 5, lane = t & 31;
+    float* red = wsp + ((RB * a.splits + 3) & ~3);   // [RB][R8], second half of the splits
+    const int vblocks = (V8 + kOutV - 1) / kOutV;
+    const int h = blockIdx.x / vblocks, v0 = (blockIdx.x - h * vblocks) * kOutV, row0 = blockIdx.y * RB;
+    const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
+    const bf16* W = a.Wkv + ((long)a.heads * dim8 + (long)h * V8) * a.ldw;
     pdl_trigger();
+    constexpr int kVs = kOutV / 8, kPre = 2;
+    uint4 pre[kVs][kPre];
+#pragma unroll
+    for (int i = 0; i < kVs; ++i)
+#pragma unroll
+        for (int j = 0; j < kPre; ++j) {
+            const int v = v0 + warp + 8 * i, c = lane * 8 + 256 * j;
+            pre[i][j] = v < a.V && c < R8 ? __ldg(reinterpret_cast<const uint4*>(W + (long)v * a.ldw + c)) : make_uint4(0, 0, 0, 0);
+        }
     pdl_wait();
     if (warp < RB && row0 + warp < r.T) {
-        const int row = row0 + warp;
+        const int row = row0 + warp, ns = r.slot_of(row) < 0 ? 0 : used_splits(min(r.pos_of(row) + 1, a.max_seq), keys, a.splits);
         const float sink = a.sink[h];
         float m = sink;
-        for (int s = lane; s < a.splits; s += 32) m = fmaxf(m, part_ptr(a, row, h, s)[a.R]);
+        for (int s = lane; s < ns; s += 32) m = fmaxf(m, part_ptr(a, row, h, s)[R8]);
         m = warp_max(m);
         float l = 0.f;
-        for (int s = lane; s < a.splits; s += 32) {
-            const float* p = part_ptr(a, row, h, s);
-            const float w = p[a.R + 1] > 0.f ? expf(p[a.R] - m) : 0.f;
+        for (int s = lane; s < ns; s += 32) {
+            const float* p = part_ptr(a, row, h, s) + R8;
+            const float w = expf(p[0] - m);
             wsp[warp * a.splits + s] = w;
-            l += w > 0.f ? w * p[a.R + 1] : 0.f;
+            l = fmaf(w, p[1], l);
         }
         l = warp_sum(l) + expf(sink - m);
         __syncwarp();
-        for (int s = lane; s < a.splits; s += 32) wsp[warp * a.splits + s] /= l;
+        for (int s = lane; s < ns; s += 32) wsp[warp * a.splits + s] /= l;
     }
     __syncthreads();
-    for (int i = t; i < RB * R8; i += 256) {
-        const int b = i / R8, c = i - b * R8;
-        float v = 0.f;
-        if (row0 + b < r.T && c < a.R)
-            for (int s = 0; s < a.splits; ++s) {
+    const int halves = nq <= 128 ? 2 : 1, part = halves == 2 ? t >> 7 : 0;
+    for (int i = halves == 2 ? t & 127 : t; i < RB * nq; i += 256 / halves) {
+        const int b = i / nq, c = (i - b * nq) * 4, row = row0 + b;
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (row < r.T) {
+            const int ns = r.slot_of(row) < 0 ? 0 : used_splits(min(r.pos_of(row) + 1, a.max_seq), keys, a.splits);
+            const float* p = part_ptr(a, row, h, 0) + c;
+            const long step = R8 + kPartStats;
+#pragma unroll 8
+            for (int s = part; s < ns; s += halves) {
                 const float w = wsp[b * a.splits + s];
-                if (w > 0.f) v = fmaf(w, part_ptr(a, row0 + b, h, s)[c], v);
-            }
-        lat[i] = v;
-    }
-    __syncthreads();
-    float gate[RB];
-#pragma unroll
-    for (int b = 0; b < RB; ++b) gate[b] = row0 + b < r.T ? sigmoid_f(a.gate[(long)(row0 + b) * a.ld32 + h]) : 0.f;
-    const bf16* W = a.Wkv + ((long)a.heads * dim8 + (long)h * V8) * a.ldw;
-#pragma unroll 2
-    for (int v = warp; v < V8; v += 8) {
-        float acc[RB] = {};
-        if (v < a.V) {
-#pragma unroll 2
-            for (int c = lane * 8; c < R8; c += 256) {
-                const uint4 w = __ldg(reinterpret_cast<const uint4*>(W + (long)v * a.ldw + c));
-                const uint32_t ww[4] = {w.x, w.y, w.z, w.w};
-#pragma unroll
-                for (int b = 0; b < RB; ++b) {
-                    const float4 x0 = *reinterpret_cast<const float4*>(lat + b * R8 + c);
-                    const float4 x1 = *reinterpret_cast<const float4*>(lat + b * R8 + c + 4);
-                    acc[b] = fmaf(x0.x, __uint_as_float(ww[0] << 16), acc[b]);
-                    acc[b] = fmaf(x0.y, __uint_as_float(ww[0] & 0xFFFF0000u), acc[b]);
-                    acc[b] = fmaf(x0.z, __uint_as_float(ww[1] << 16), acc[b]);
-                    acc[b] = fmaf(x0.w, __uint_as_float(ww[1] & 0xFFFF0000u), acc[b]);
-                    acc[b] = fmaf(x1.x, __uint_as_float(ww[2] << 16), acc[b]);
-                    acc[b] = fmaf(x1.y, __uint_as_float(ww[2] & 0xFFFF0000u), acc[b]);
-                    acc[b] = fmaf(x1.z, __uint_as_float(ww[3] << 16), acc[b]);
-                    acc[b] = fmaf(x1.w, __uint_as_float(ww[3] & 0xFFFF0000u), acc[b]);
-                }
+                const float4 x = *reinterpret_cast<const float4*>(p + s * step);
+                acc.x = fmaf(w, x.x, acc.x);
+                acc.y = fmaf(w, x.y, acc.y);
+                acc.z = fmaf(w, x.z, acc.z);
+                acc.w = fmaf(w, x.w, acc.w);
             }
         }
+        *reinterpret_cast<float4*>((part ? red : lat) + b * R8 + c) = acc;
+    }
+    __syncthreads();
+    if (halves == 2) {
+        for (int i = t; i < RB * R8; i += 256) lat[i] += red[i];
+        __syncthreads();
+    }
+    float acc[kVs][RB] = {};
+    auto add = [&](const uint4& w, int c, int i) {
+        const uint32_t ww[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
         for (int b = 0; b < RB; ++b) {
-            const float s = warp_sum(acc[b]);
-            if (lane == 0 && row0 + b < r.T)
-                static_cast<A*>(a.out)[(long)(row0 + b) * a.ldout + h * V8 + v] = from_f<A>(s * gate[b]);
+            const float4 x0 = *reinterpret_cast<const float4*>(lat + b * R8 + c);
+            const float4 x1 = *reinterpret_cast<const float4*>(lat + b * R8 + c + 4);
+            float s = acc[i][b];
+            s = fmaf(x0.x, __uint_as_float(ww[0] << 16), s);
+            s = fmaf(x0.y, __uint_as_float(ww[0] & 0xFFFF0000u), s);
+            s = fmaf(x0.z, __uint_as_float(ww[1] << 16), s);
+            s = fmaf(x0.w, __uint_as_float(ww[1] & 0xFFFF0000u), s);
+            s = fmaf(x1.x, __uint_as_float(ww[2] << 16), s);
+            s = fmaf(x1.y, __uint_as_float(ww[2] & 0xFFFF0000u), s);
+            s = fmaf(x1.z, __uint_as_float(ww[3] << 16), s);
+            s = fmaf(x1.w, __uint_as_float(ww[3] & 0xFFFF0000u), s);
+            acc[i][b] = s;
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < kVs; ++i) {
+        const int v = v0 + warp + 8 * i;
+#pragma unroll
+        for (int j = 0; j < kPre; ++j)
+            if (lane * 8 + 256 * j < R8) add(pre[i][j], lane * 8 + 256 * j, i);
+        if (v < a.V)
+            for (int c = lane * 8 + 256 * kPre; c < R8; c += 256) add(__ldg(reinterpret_cast<const uint4*>(W + (long)v * a.ldw + c)), c, i);
+    }
+#pragma unroll
+    for (int i = 0; i < kVs; ++i) {
+        const int v = v0 + warp + 8 * i;
+#pragma unroll
+        for (int b = 0; b < RB; ++b) {
+            const float s = warp_sum(acc[i][b]);
+            if (lane == 0 && v < V8 && row0 + b < r.T)
+                static_cast<A*>(a.out)[(long)(row0 + b) * a.ldout + h * V8 + v] =
+                    from_f<A>(v < a.V ? s * sigmoid_f(a.gate[(long)(row0 + b) * a.ld32 + h]) : 0.f);
         }
     }
 }
 
 // ------------------------------------------------------------------------------------------ expanded form
-constexpr int kFlashQ = 128, kFlashK = 64;
+constexpr int kFlashK = 64;   // keys per shared-memory tile
 struct FlashSmem {
     int row, vrow, k_off, kbuf, total;
-    __host__ __device__ FlashSmem(int D, int VT) {
+    __host__ __device__ FlashSmem(int D, int VT, int MT) {
         row = D * 2 + 16;
         vrow = VT * 16 + 16;
-        k_off = kFlashQ * row;
+        k_off = 128 * MT * row;
         kbuf = kFlashK * (row + vrow);
         total = k_off + 2 * kbuf;
     }
 };
 
-// Block (128 query rows, head, slice of VT * 8 value columns); warp w has rows 16 w .. 16 w + 15.
-template <int VT>
+// Block (128 * MT query rows, head, slice of VT * 8 value columns); a warp has MT tiles of 16 rows, so that every key and
+// value fragment it reads from shared memory serves MT products.  MT == 2 takes the 64 keys of a tile in two halves.
+template <int VT, int MT>
 __global__ void __launch_bounds__(256, 1) latent_flash_kernel(const LatentArgs a, const Rows r) {
     extern __shared__ __align__(16) unsigned char smem[];
+    constexpr int kQ = 128 * MT, KT = MT == 1 ? 8 : 4;     // KT: 8-key tiles per softmax step
     const int dim8 = pad8(a.dim), rot8 = pad8(a.rot), D8 = dim8 + rot8, D = pad16(D8), V8 = pad8(a.V), R8 = pad8(a.R);
-    const FlashSmem L(D, VT);
+    const FlashSmem L(D, VT, MT);
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, q4 = lane & 3;
-    const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kFlashQ, h = blockIdx.y, v0 = blockIdx.z * VT * 8;
+    const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kQ, h = blockIdx.y, v0 = blockIdx.z * VT * 8;
     const uint32_t sb = smem_u32(smem);
     const bf16* kv = static_cast<const bf16*>(a.kv);
     const long ldkv = (long)a.heads * (dim8 + V8);
     const bf16* kr = static_cast<const bf16*>(a.cache) + (long)r.slot * a.max_seq * a.ldc + R8;
-    const int last = min(r.T, q0 + kFlashQ) - 1;           // last real query row of the block
+    const int last = min(r.T, q0 + kQ) - 1;                // last real query row of the block
     const int nkeys = r.pos0 + last + 1, tiles = (nkeys + kFlashK - 1) / kFlashK;
+    pdl_trigger();
     pdl_wait();
+    const int nc = D / 8;
     auto issue = [&](int tile, int buf) {
         const uint32_t kb = sb + L.k_off + buf * L.kbuf, vb = kb + kFlashK * L.row;
-        const int nc = D / 8;
         for (int i = t; i < kFlashK * nc; i += 256) {
             const int k = i / nc, c = (i - k * nc) * 8, key = tile * kFlashK + k;
             const bool ok = key < nkeys && c < D8;
@@ -491,19 +564,18 @@ __global__ void __launch_bounds__(256, 1) latent_flash_kernel(const LatentArgs a
         }
         cp_async_commit();
     };
-    {
-        const int nc = D / 8;
-        for (int i = t; i < kFlashQ * nc; i += 256) {
-            const int q = i / nc, c = (i - q * nc) * 8;
-            const bool ok = q0 + q < r.T && c < D8;
-            const bf16* src = static_cast<const bf16*>(a.q);
-            cp_async16z(sb + q * L.row + c * 2, ok ? src + (long)(q0 + q) * a.ldq + h * D8 + c : src, ok);
-        }
+    for (int i = t; i < kQ * nc; i += 256) {
+        const int q = i / nc, c = (i - q * nc) * 8;
+        const bool ok = q0 + q < r.T && c < D8;
+        const bf16* src = static_cast<const bf16*>(a.q);
+        cp_async16z(sb + q * L.row + c * 2, ok ? src + (long)(q0 + q) * a.ldq + h * D8 + c : src, ok);
     }
     issue(0, 0);
-    float O[VT][4] = {};
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-    const int wrow = q0 + 16 * warp;                       // first query row of the warp
+    float O[MT][VT][4] = {};
+    float m[MT][2], l[MT][2];
+#pragma unroll
+    for (int i = 0; i < MT; ++i) { m[i][0] = m[i][1] = -INFINITY; l[i][0] = l[i][1] = 0.f; }
+    const int wrow = q0 + 16 * MT * warp;                  // first query row of the warp
     const float sl2 = a.scale * 1.4426950408889634f;       // softmax in base 2
     for (int tile = 0; tile < tiles; ++tile) {
         const int buf = tile & 1;
@@ -511,85 +583,107 @@ __global__ void __launch_bounds__(256, 1) latent_flash_kernel(const LatentArgs a
         cp_async_wait<0>();
         __syncthreads();
         if (tile + 1 < tiles) issue(tile + 1, buf ^ 1);
-        if (tile * kFlashK > r.pos0 + wrow + 15) continue;  // nothing of this tile is visible to the warp
-        float s[8][4] = {};
-        for (int k0 = 0; k0 < D; k0 += 16) {
-            uint32_t fa[4];
-            ldsm4(sb + (16 * warp + (lane & 15)) * L.row + (k0 + (lane >> 4) * 8) * 2, fa);
+#pragma unroll 1
+        for (int sub = 0; sub < kFlashK; sub += 8 * KT) {
+            const int key0 = tile * kFlashK + sub;
+            if (key0 > r.pos0 + wrow + 16 * MT - 1) break;  // nothing more of this tile is visible to the warp
+            float s[MT][KT][4] = {};
+#pragma unroll 2
+            for (int k0 = 0; k0 < D; k0 += 16) {
+                uint32_t fa[MT][4];
 #pragma unroll
-            for (int jj = 0; jj < 4; ++jj) {
-                uint32_t fb[4];
-                ldsm4(kb + (16 * jj + (lane & 7) + (lane >> 4) * 8) * L.row + (k0 + ((lane >> 3) & 1) * 8) * 2, fb);
-                mma_bf16(s[2 * jj], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
-                mma_bf16(s[2 * jj + 1], fa[0], fa[1], fa[2], fa[3], fb[2], fb[3]);
+                for (int i = 0; i < MT; ++i)
+                    ldsm4(sb + (16 * (MT * warp + i) + (lane & 15)) * L.row + (k0 + (lane >> 4) * 8) * 2, fa[i]);
+#pragma unroll
+                for (int jj = 0; jj < KT / 2; ++jj) {
+                    uint32_t fb[4];
+                    ldsm4(kb + (sub + 16 * jj + (lane & 7) + (lane >> 4) * 8) * L.row + (k0 + ((lane >> 3) & 1) * 8) * 2, fb);
+#pragma unroll
+                    for (int i = 0; i < MT; ++i) {
+                        mma_bf16(s[i][2 * jj], fa[i][0], fa[i][1], fa[i][2], fa[i][3], fb[0], fb[1]);
+                        mma_bf16(s[i][2 * jj + 1], fa[i][0], fa[i][1], fa[i][2], fa[i][3], fb[2], fb[3]);
+                    }
+                }
             }
-        }
-        const bool edge = tile * kFlashK + kFlashK - 1 > r.pos0 + wrow;
+            const bool edge = key0 + 8 * KT - 1 > r.pos0 + wrow;
 #pragma unroll
-        for (int p = 0; p < 2; ++p) {
-            const int pos = r.pos0 + wrow + g + 8 * p;
-            float mx = m[p];
+            for (int i = 0; i < MT; ++i)
 #pragma unroll
-            for (int j = 0; j < 8; ++j)
+                for (int p = 0; p < 2; ++p) {
+                    const int pos = r.pos0 + wrow + 16 * i + g + 8 * p;
+                    float mx = m[i][p];
 #pragma unroll
-                for (int i = 0; i < 2; ++i) {
-                    float& x = s[j][2 * p + i];
-                    x *= sl2;
-                    if (edge && tile * kFlashK + 8 * j + 2 * q4 + i > pos) x = -INFINITY;
-                    mx = fmaxf(mx, x);
+                    for (int j = 0; j < KT; ++j)
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) {
+                            float& x = s[i][j][2 * p + e];
+                            x *= sl2;
+                            if (edge && key0 + 8 * j + 2 * q4 + e > pos) x = -INFINITY;
+                            mx = fmaxf(mx, x);
+                        }
+                    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+                    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+                    const float base = mx == -INFINITY ? 0.f : mx, alpha = exp2f(m[i][p] - base);
+                    m[i][p] = mx;
+                    float sum = 0.f;
+#pragma unroll
+                    for (int j = 0; j < KT; ++j)
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) {
+                            float& x = s[i][j][2 * p + e];
+                            x = exp2f(x - base);
+                            sum += x;
+                        }
+                    l[i][p] = l[i][p] * alpha + sum;
+                    if (__any_sync(0xffffffffu, alpha != 1.f)) {
+#pragma unroll
+                        for (int j = 0; j < VT; ++j) { O[i][j][2 * p] *= alpha; O[i][j][2 * p + 1] *= alpha; }
+                    }
                 }
-            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-            const float base = mx == -INFINITY ? 0.f : mx, alpha = exp2f(m[p] - base);
-            m[p] = mx;
-            float sum = 0.f;
 #pragma unroll
-            for (int j = 0; j < 8; ++j)
+            for (int kk = 0; kk < KT / 2; ++kk) {   // 16 keys: the score fragments are the A operand
+                uint32_t ph[MT][4], pl[MT][4];
 #pragma unroll
-                for (int i = 0; i < 2; ++i) {
-                    float& x = s[j][2 * p + i];
-                    x = exp2f(x - base);
-                    sum += x;
+                for (int i = 0; i < MT; ++i) {
+                    split_bf16(s[i][2 * kk][0], s[i][2 * kk][1], ph[i][0], pl[i][0]);
+                    split_bf16(s[i][2 * kk][2], s[i][2 * kk][3], ph[i][1], pl[i][1]);
+                    split_bf16(s[i][2 * kk + 1][0], s[i][2 * kk + 1][1], ph[i][2], pl[i][2]);
+                    split_bf16(s[i][2 * kk + 1][2], s[i][2 * kk + 1][3], ph[i][3], pl[i][3]);
                 }
-            l[p] = l[p] * alpha + sum;
 #pragma unroll
-            for (int j = 0; j < VT; ++j) { O[j][2 * p] *= alpha; O[j][2 * p + 1] *= alpha; }
-        }
+                for (int j = 0; j < VT; j += 2) {
+                    uint32_t v[4];
+                    ldsm4t(vb + (sub + 16 * kk + (lane & 15)) * L.vrow + (8 * j + (lane >> 4) * 8) * 2, v);
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk) {   // 16 keys: the score fragments are the A operand
-            uint32_t ph[4], pl[4];
-            split_bf16(s[2 * kk][0], s[2 * kk][1], ph[0], pl[0]);
-            split_bf16(s[2 * kk][2], s[2 * kk][3], ph[1], pl[1]);
-            split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], ph[2], pl[2]);
-            split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], ph[3], pl[3]);
-#pragma unroll
-            for (int j = 0; j < VT; j += 2) {
-                uint32_t v[4];
-                ldsm4t(vb + (16 * kk + (lane & 15)) * L.vrow + (8 * j + (lane >> 4) * 8) * 2, v);
-                mma_bf16(O[j], ph[0], ph[1], ph[2], ph[3], v[0], v[1]);
-                mma_bf16(O[j + 1], ph[0], ph[1], ph[2], ph[3], v[2], v[3]);
-                mma_bf16(O[j], pl[0], pl[1], pl[2], pl[3], v[0], v[1]);
-                mma_bf16(O[j + 1], pl[0], pl[1], pl[2], pl[3], v[2], v[3]);
+                    for (int i = 0; i < MT; ++i) {
+                        mma_bf16(O[i][j], ph[i][0], ph[i][1], ph[i][2], ph[i][3], v[0], v[1]);
+                        mma_bf16(O[i][j + 1], ph[i][0], ph[i][1], ph[i][2], ph[i][3], v[2], v[3]);
+                        mma_bf16(O[i][j], pl[i][0], pl[i][1], pl[i][2], pl[i][3], v[0], v[1]);
+                        mma_bf16(O[i][j + 1], pl[i][0], pl[i][1], pl[i][2], pl[i][3], v[2], v[3]);
+                    }
+                }
             }
         }
     }
     const float sink = a.sink[h] * 1.4426950408889634f;
 #pragma unroll
-    for (int p = 0; p < 2; ++p) {
-        const int q = wrow + g + 8 * p;
-        float tot = l[p];
-        tot += __shfl_xor_sync(0xffffffffu, tot, 1);
-        tot += __shfl_xor_sync(0xffffffffu, tot, 2);
-        if (q >= r.T) continue;
-        const float mm = fmaxf(m[p], sink), sc = exp2f(m[p] - mm);
-        const float f = sc / (tot * sc + exp2f(sink - mm)) * sigmoid_f(a.gate[(long)q * a.ld32 + h]);
-        bf16* out = static_cast<bf16*>(a.out) + (long)q * a.ldout + h * V8 + v0;
+    for (int i = 0; i < MT; ++i)
 #pragma unroll
-        for (int j = 0; j < VT; ++j) {
-            const int col = 8 * j + 2 * q4;
-            if (v0 + col < V8) *reinterpret_cast<uint32_t*>(out + col) = pack_bf16(O[j][2 * p] * f, O[j][2 * p + 1] * f);
+        for (int p = 0; p < 2; ++p) {
+            const int q = wrow + 16 * i + g + 8 * p;
+            float tot = l[i][p];
+            tot += __shfl_xor_sync(0xffffffffu, tot, 1);
+            tot += __shfl_xor_sync(0xffffffffu, tot, 2);
+            if (q >= r.T) continue;
+            const float mm = fmaxf(m[i][p], sink), sc = exp2f(m[i][p] - mm);
+            const float f = sc / (tot * sc + exp2f(sink - mm)) * sigmoid_f(a.gate[(long)q * a.ld32 + h]);
+            bf16* out = static_cast<bf16*>(a.out) + (long)q * a.ldout + h * V8 + v0;
+#pragma unroll
+            for (int j = 0; j < VT; ++j) {
+                const int col = 8 * j + 2 * q4;
+                if (v0 + col < V8) *reinterpret_cast<uint32_t*>(out + col) = pack_bf16(O[i][j][2 * p] * f, O[i][j][2 * p + 1] * f);
+            }
         }
-    }
 }
 
 }  // namespace lm

@@ -305,7 +305,7 @@ public:
         w->proj32 = std::max(w->proj32, (long)in_.N - split_);
         w->mixed = std::max(w->mixed, (long)mixed_ld());
         w->absorbed_bytes = std::max(w->absorbed_bytes, 4L * rows * s_.heads * lm::latent_dp(s_.kv_rank, s_.rot_dim));
-        for (int T = 1; T <= rows; ++T) w->part = std::max(w->part, (long)T * s_.heads * splits(e, T) * (s_.kv_rank + 2));
+        for (int T = 1; T <= rows; ++T) w->part = std::max(w->part, (long)T * s_.heads * splits(e, T) * (pad8(s_.kv_rank) + lm::kPartStats));
         if (expanded_) w->kv = std::max(w->kv, (long)e.max_seq * s_.heads * (pad8(s_.dim) + pad8(s_.vdim)));
         if (owner_) return 0;
         char* c = nullptr;
@@ -331,10 +331,10 @@ public:
 
 private:
     int q8() const { return pad8(s_.dim) + pad8(s_.rot_dim); }
-    // context splits of an absorbed call with T rows: fills the SMs, at least two 64-key tiles each at full length
+    // context splits of an absorbed call with T rows: one CTA per SM, at least one 64-key tile each at full length
     int splits(const Env& e, int T) const {
         const int blocks = T * (e.f32 ? s_.heads : (s_.heads + 15) / 16);
-        return std::max(1, std::min({64, (e.max_seq + 127) / 128, e.sms / blocks}));
+        return std::max(1, std::min({64, (e.max_seq + 63) / 64, e.sms / blocks}));
     }
     lm::LatentArgs base(const Env& e) const {
         lm::LatentArgs a{};

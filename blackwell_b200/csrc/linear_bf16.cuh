@@ -193,7 +193,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearArgs a) {
 // ---------------------------------------------------------------------------------------------- tcgen05
 constexpr int kTcRows = 128;      // weight rows per tile (MMA M)
 constexpr int kTcK = 64;          // k per stage: one 128-byte swizzle atom of bf16
-constexpr int kTcThreads = 256;   // warp 0 copies, warp 1 MMAs, warps 4-7 epilogue
+constexpr int kTcThreads = 384;   // warp 0 copies, warp 1 MMAs, warps 4-11 epilogue (two per TMEM lane quarter)
 
 __host__ __device__ constexpr int tc_stage_bytes(int NT) { return kTcRows * 128 + NT * 128; }
 __host__ __device__ constexpr int tc_stages(int NT) { return NT >= 256 ? 4 : NT >= 128 ? 6 : 8; }
@@ -255,7 +255,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
     };
     if (t == 0) {
         for (int i = 0; i < S; ++i) { mbar_init(full(i), 1); mbar_init(empty(i), 1); }
-        for (int i = 0; i < 2; ++i) { mbar_init(dfull(i), 1); mbar_init(dempty(i), 4); }
+        for (int i = 0; i < 2; ++i) { mbar_init(dfull(i), 1); mbar_init(dempty(i), 8); }
         *abort_flag = 0;
         mbar_fence_init();
     }
@@ -331,7 +331,9 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             }
         }
     } else if (warp >= 4) {
-        const int quarter = warp & 3;
+        const int quarter = warp & 3, half = (warp - 4) >> 2;
+        constexpr int CW = NT >= 64 ? 32 : 16;               // columns per read
+        constexpr int HC = NT >= 32 ? NT / 2 : NT;           // columns per warp
         int w = 0;
         for (int tile = first; tile < tiles; tile += stride, ++w) {
             const int d = w % NACC;
@@ -339,27 +341,53 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             tc::tc_fence_after();
             const int row = (tile % rtiles) * kTcRows + quarter * 32 + lane, tok0 = (tile / rtiles) * NT;
             const uint32_t src = tmem + d * NT + ((uint32_t)(quarter * 32) << 16);
+            const int g0 = row - lane;                       // the warp's 32 rows
+            const bool whole = g0 + 32 <= a.N && (g0 + 32 <= a.split || g0 >= a.split);
+            const bool to32 = g0 >= a.split || a.y_f32;
+            const bool packed = whole && !to32 && a.epi == kEpiNone && a.ldy % 2 == 0 && (reinterpret_cast<uintptr_t>(a.y) & 3) == 0;
 #pragma unroll 1
-            for (int c0 = 0; c0 < NT; c0 += 16) {
+            for (int c0 = half * HC; c0 < half * HC + HC && c0 < NT; c0 += CW) {
                 if (!SPLIT && tok0 + c0 >= a.T) break;
-                uint32_t v[16];
-                tc::tmem_ld16(src + c0, v);
+                uint32_t v[CW / 16][16];
+#pragma unroll
+                for (int i = 0; i < CW / 16; ++i) tc::tmem_ld16(src + c0 + 16 * i, v[i]);
                 tc::tmem_wait_ld();
+                const int left = a.T - tok0 - c0;            // columns with a row of x
                 if (SPLIT) {
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) part[(c0 + i) * kTcRows + quarter * 32 + lane] = __uint_as_float(v[i]);
+                    for (int i = 0; i < CW; ++i) part[(c0 + i) * kTcRows + quarter * 32 + lane] = __uint_as_float(v[i / 16][i % 16]);
                 } else if (a.epi == kEpiSwiglu) {
+                    // even lanes hold gates, odd lanes the ups beside them: a pair of lanes exchanges one value each and
+                    // finishes two columns
+                    bf16* y = static_cast<bf16*>(a.y) + (long)(tok0 + c0 + (lane & 1)) * a.ldy + (row >> 1);
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) {
-                        const float mine = __uint_as_float(v[i]);
-                        const float up = __shfl_down_sync(0xffffffffu, mine, 1);
-                        if (!(lane & 1) && row < a.N && tok0 + c0 + i < a.T)
-                            static_cast<bf16*>(a.y)[(long)(tok0 + c0 + i) * a.ldy + (row >> 1)] = __float2bfloat16_rn(silu_f(mine) * up);
+                    for (int i = 0; i < CW; i += 2) {
+                        const float x0 = __uint_as_float(v[i / 16][i % 16]), x1 = __uint_as_float(v[i / 16][i % 16 + 1]);
+                        const float got = __shfl_xor_sync(0xffffffffu, (lane & 1) ? x0 : x1, 1);
+                        const float gate = (lane & 1) ? got : x0, up = (lane & 1) ? x1 : got;
+                        if (row < a.N && i + (lane & 1) < left)
+                            y[(long)i * a.ldy] = __float2bfloat16_rn(__fdividef(gate, 1.0f + __expf(-gate)) * up);
                     }
+                } else if (packed) {   // two rows of one column per lane
+                    bf16* y = static_cast<bf16*>(a.y) + (long)(tok0 + c0 + (lane & 1)) * a.ldy + (row & ~1);
+#pragma unroll
+                    for (int i = 0; i < CW; i += 2) {
+                        const float x0 = __uint_as_float(v[i / 16][i % 16]), x1 = __uint_as_float(v[i / 16][i % 16 + 1]);
+                        const float got = __shfl_xor_sync(0xffffffffu, (lane & 1) ? x0 : x1, 1);
+                        if (i + (lane & 1) < left)
+                            *reinterpret_cast<uint32_t*>(y + (long)i * a.ldy) = (lane & 1) ? pack_bf16(got, x1) : pack_bf16(x0, got);
+                    }
+                } else if (whole && to32 && a.epi == kEpiNone) {
+                    const bool second = g0 >= a.split;
+                    const long ld = second ? a.ldy32 : a.ldy;
+                    float* y = (second ? a.y32 - a.split : static_cast<float*>(a.y)) + (long)(tok0 + c0) * ld + row;
+#pragma unroll
+                    for (int i = 0; i < CW; ++i)
+                        if (i < left) y[(long)i * ld] = __uint_as_float(v[i / 16][i % 16]);
                 } else if (row < a.N) {
 #pragma unroll
-                    for (int i = 0; i < 16; ++i)
-                        if (tok0 + c0 + i < a.T) store_out<false>(a, tok0 + c0 + i, row, __uint_as_float(v[i]));
+                    for (int i = 0; i < CW; ++i)
+                        if (i < left) store_out<false>(a, tok0 + c0 + i, row, __uint_as_float(v[i / 16][i % 16]));
                 }
             }
             tc::tc_fence_before();

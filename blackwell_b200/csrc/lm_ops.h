@@ -99,6 +99,7 @@ bool recurrence_chunk_supported(const RecurrenceArgs& a);
 cudaError_t recurrence_chunk(const RecurrenceArgs& a, const Rows& r, cudaStream_t st);   // bf16, rows of one sequence
 
 // ---------------------------------------------------------------- latent attention
+constexpr int kPartStats = 4;   // floats after a split's outputs: running maximum, sum, padding
 struct LatentArgs {
     int heads, dim, rot, V, R;        // per head: unrotated / rotated query size, value size; latent size
     int rot_dims;                     // rotated part of the `rot` dimensions
@@ -120,7 +121,7 @@ struct LatentArgs {
     long ldout;
     // scratch
     void* qabs;                       // [T][heads][2][Dp] bf16 (high, remainder) or [T][heads][Dp] fp32
-    float* part;                      // [T][heads][splits][R + 2]
+    float* part;                      // [T][heads][splits][pad8(R) + kPartStats]
     int splits;
     void* kv;                         // expanded keys and values [max_seq][heads * (pad8(dim) + pad8(V))]
 };

@@ -26,18 +26,18 @@ cudaError_t step_nr(const RecurrenceArgs& a, const ConvArgs& c, const Rows& r, c
          : nr <= 16 ? step_inst<A, 16, CONV>(a, c, r, st) : cudaErrorInvalidValue;
 }
 
-template <int NTW>
+template <int NTW, int VT>
 cudaError_t chunk_inst(const RecurrenceArgs& a, const Rows& r, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
+    auto kern = recurrence_chunk_kernel<NTW, VT>;
     cudaError_t e = cudaSuccess;
     std::call_once(once[current_device()], [&] {
-        e = cudaFuncSetAttribute(recurrence_chunk_kernel<NTW>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem);
+        e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxDynSmem);
     });
     if (e != cudaSuccess) return e;
-    const int nbuf = ChunkSmem(a.N, 2).total <= kMaxDynSmem ? 2 : 1;
-    const dim3 grid((pad8(a.V) + kChV - 1) / kChV, a.heads);
+    const int nbuf = ChunkSmem(a.N, VT, 2).total <= kMaxDynSmem ? 2 : 1;
     count_launch(1);
-    return launch_pdl(recurrence_chunk_kernel<NTW>, grid, dim3(256), ChunkSmem(a.N, nbuf).total, st, a, r, nbuf);
+    return launch_pdl(kern, dim3((pad8(a.V) + VT - 1) / VT, a.heads), dim3(256), ChunkSmem(a.N, VT, nbuf).total, st, a, r, nbuf);
 }
 
 }  // namespace
@@ -49,11 +49,15 @@ cudaError_t recurrence_step(const RecurrenceArgs& a, const ConvArgs* conv, const
     return f32 ? step_nr<float, false>(a, none, r, st) : step_nr<bf16, false>(a, none, r, st);
 }
 
-bool recurrence_chunk_supported(const RecurrenceArgs& a) { return a.N <= 256 && ChunkSmem(a.N, 1).total <= kMaxDynSmem; }
+bool recurrence_chunk_supported(const RecurrenceArgs& a) { return a.N <= 256 && ChunkSmem(a.N, 32, 1).total <= kMaxDynSmem; }
 
 cudaError_t recurrence_chunk(const RecurrenceArgs& a, const Rows& r, cudaStream_t st) {
     if (a.groups < 1 || a.heads % a.groups != 0 || r.row_slot || !recurrence_chunk_supported(a)) return cudaErrorInvalidValue;
-    return pad16(a.N) <= 128 ? chunk_inst<1>(a, r, st) : chunk_inst<2>(a, r, st);
+    // narrow state tiles while the wide ones leave SMs idle, and where only they fit shared memory twice
+    const int wide = (pad8(a.V) + 63) / 64 * a.heads;
+    const bool narrow = a.V <= 32 || wide <= sm_count(current_device()) / 2 || ChunkSmem(a.N, 64, 1).total > kMaxDynSmem;
+    if (pad16(a.N) <= 128) return narrow ? chunk_inst<1, 32>(a, r, st) : chunk_inst<1, 64>(a, r, st);
+    return narrow ? chunk_inst<2, 32>(a, r, st) : chunk_inst<2, 64>(a, r, st);
 }
 
 }  // namespace lm

@@ -140,14 +140,13 @@ __global__ void __launch_bounds__(kRecThreads) recurrence_step_kernel(const Recu
 
 // ---------------------------------------------------------------------------------------------- chunks of 64 tokens
 constexpr int kChunk = 64;
-constexpr int kChV = 64;                 // state columns per CTA
-constexpr int kVRow = kChV * 2 + 16;     // bytes of a 64-column bf16 row in shared memory (odd multiple of 16)
-constexpr int kPRow = kChunk * 2 + 16;
+constexpr int kPRow = kChunk * 2 + 16;   // bytes of a row of scores in shared memory (odd multiple of 16)
+constexpr float kLog2e = 1.4426950408889634f;
 
 struct ChunkSmem {
     int qrow, k_off, v_off, buf, vw_off, s_off, p_off, f_off, total;
-    __host__ __device__ ChunkSmem(int N, int nbuf) {
-        const int NP = pad16(N);
+    __host__ __device__ ChunkSmem(int N, int VT, int nbuf) {   // VT: state columns per CTA
+        const int NP = pad16(N), kVRow = VT * 2 + 16;
         qrow = NP * 2 + 16;
         k_off = kChunk * qrow;
         v_off = 2 * kChunk * qrow;
@@ -156,21 +155,21 @@ struct ChunkSmem {
         s_off = vw_off + 2 * kChunk * kVRow;       // state, high and remainder
         p_off = s_off + 2 * NP * kVRow;            // decayed scores, high and remainder
         f_off = p_off + 2 * kChunk * kPRow;        // cumulative log decay, weights
-        total = f_off + 2 * kChunk * 4 + 16;
+        total = f_off + 2 * 2 * kChunk * 4;
     }
 };
 
-// NTW: 16-row state tiles per warp.
-template <int NTW>
+// NTW: 16-row state tiles per warp; VT: state columns per CTA (64 or 32).
+template <int NTW, int VT>
 __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceArgs a, const Rows r, int nbuf) {
     extern __shared__ __align__(16) unsigned char smem[];
-    const ChunkSmem L(a.N, nbuf);
+    constexpr int kVRow = VT * 2 + 16, NJ = VT / 16;   // NJ: 8-column output tiles per warp
+    const ChunkSmem L(a.N, VT, nbuf);
     const int NP = pad16(a.N), N8 = pad8(a.N), V8 = pad8(a.V);
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, q4 = lane & 3;
-    const int h = blockIdx.y, v0 = blockIdx.x * kChV, grp = h / (a.heads / a.groups);
+    const int h = blockIdx.y, v0 = blockIdx.x * VT, grp = h / (a.heads / a.groups);
     const uint32_t sb = smem_u32(smem);
-    float* cum = reinterpret_cast<float*>(smem + L.f_off);
-    float* wt = cum + kChunk;
+    float* dec = reinterpret_cast<float*>(smem + L.f_off);   // [2][cumulative log2 decay, weight][chunk]
     const int nchunks = (r.T + kChunk - 1) / kChunk;
     const bf16* qg = static_cast<const bf16*>(a.q) + grp * N8;
     const bf16* kg = static_cast<const bf16*>(a.k) + grp * N8;
@@ -186,8 +185,8 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
             cp_async16z(base + row * L.qrow + col * 2, ok ? qg + (long)tok * a.ldq + col : qg, ok);
             cp_async16z(base + L.k_off + row * L.qrow + col * 2, ok ? kg + (long)tok * a.ldk + col : kg, ok);
         }
-        for (int i = t; i < kChunk * (kChV / 8); i += 256) {
-            const int row = i >> 3, col = (i & 7) * 8, tok = ch * kChunk + row;
+        for (int i = t; i < kChunk * (VT / 8); i += 256) {
+            const int row = i / (VT / 8), col = (i % (VT / 8)) * 8, tok = ch * kChunk + row;
             const bool ok = tok < r.T && v0 + col < V8;
             cp_async16z(base + L.v_off + row * kVRow + col * 2, ok ? vg + (long)tok * a.ldv + col : vg, ok);
         }
@@ -195,7 +194,7 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
     };
 
     // state fragments: rows 16 * (i * 8 + warp) .., columns 8 * j ..
-    float S[NTW][8][4];
+    float S[NTW][VT / 8][4];
     float* Sg = a.S + (((long)r.slot * a.heads + h) * a.N) * V8 + v0;
     auto state_to_smem = [&] {
 #pragma unroll
@@ -203,7 +202,7 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
             const int n0 = 16 * (i * 8 + warp);
             if (n0 >= NP) continue;
 #pragma unroll
-            for (int j = 0; j < 8; ++j)
+            for (int j = 0; j < VT / 8; ++j)
 #pragma unroll
                 for (int p = 0; p < 2; ++p) {
                     uint32_t hi, lo;
@@ -214,11 +213,40 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
                 }
         }
     };
+    // warp 0 keeps the decays one chunk ahead: the loads of the next chunk are in flight during this one
+    float l[2], w[2];
+    auto load_decay = [&](int ch) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int tok = ch * kChunk + 2 * lane + i;
+            const bool ok = tok < r.T;   // rows past the end: no decay, no weight
+            l[i] = !ok ? 0.f : a.log_decay ? a.log_decay[(long)tok * a.heads + h] : a.head_log_decay[h];
+            w[i] = !ok ? 0.f : a.log_decay ? a.weight[(long)tok * a.heads + h] : a.const_weight;
+        }
+    };
+    auto store_decay = [&](int buf) {
+        const float l0 = l[0] * kLog2e, pair = l0 + l[1] * kLog2e;
+        float s = pair;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float up = __shfl_up_sync(0xffffffffu, s, o);
+            if (lane >= o) s += up;
+        }
+        float* cum = dec + buf * 2 * kChunk;
+        cum[2 * lane] = (s - pair) + l0;
+        cum[2 * lane + 1] = s;
+        cum[kChunk + 2 * lane] = w[0];
+        cum[kChunk + 2 * lane + 1] = w[1];
+    };
     issue(0, 0);
+    if (warp == 0) {
+        load_decay(0);
+        store_decay(0);
+    }
 #pragma unroll
     for (int i = 0; i < NTW; ++i)
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
+        for (int j = 0; j < VT / 8; ++j)
 #pragma unroll
             for (int p = 0; p < 2; ++p) {
                 const int n = 16 * (i * 8 + warp) + g + 8 * p, v = 8 * j + 2 * q4;
@@ -232,66 +260,50 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
     for (int ch = 0; ch < nchunks; ++ch) {
         const int buf = nbuf == 2 ? ch & 1 : 0;
         const uint32_t qb = sb + buf * L.buf, kb = qb + L.k_off, vb = qb + L.v_off;
-        if (warp == 0) {   // cumulative log decay of the chunk (rows past the end: no decay, no weight)
-            float l[2], w[2];
-#pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                const int tok = ch * kChunk + 2 * lane + i;
-                const bool ok = tok < r.T;
-                l[i] = !ok ? 0.f : a.log_decay ? a.log_decay[(long)tok * a.heads + h] : a.head_log_decay[h];
-                w[i] = !ok ? 0.f : a.log_decay ? a.weight[(long)tok * a.heads + h] : a.const_weight;
-            }
-            const float pair = l[0] + l[1];
-            float s = pair;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float up = __shfl_up_sync(0xffffffffu, s, o);
-                if (lane >= o) s += up;
-            }
-            const float before = s - pair;
-            cum[2 * lane] = before + l[0];
-            cum[2 * lane + 1] = s;
-            wt[2 * lane] = w[0];
-            wt[2 * lane + 1] = w[1];
-        }
         cp_async_wait<0>();
         __syncthreads();   // operands, state copy and decays are in shared memory
         if (nbuf == 2 && ch + 1 < nchunks) issue(ch + 1, buf ^ 1);
+        if (warp == 0) load_decay(ch + 1);
+        const float *cum = dec + (ch & 1) * 2 * kChunk, *wt = cum + kChunk;
         const float total = cum[kChunk - 1];
-        const int r0 = 16 * (warp & 3), c0 = 32 * (warp >> 2);
+        const int r0 = 16 * (warp & 3), c0 = 32 * (warp >> 2);   // score columns; output columns start at
+        const int o0 = (VT / 2) * (warp >> 2);
         const float cg0 = cum[r0 + g], cg1 = cum[r0 + g + 8];
 
         // scores q k^T and inter-chunk part q S, both over the N dimension
-        float sc[4][4] = {}, out[4][4] = {};
+        float sc[4][4] = {}, out[NJ][4] = {};
+#pragma unroll 2
         for (int k0 = 0; k0 < NP; k0 += 16) {
             uint32_t fa[4];
             ldsm4(qb + (r0 + (lane & 15)) * L.qrow + (k0 + (lane >> 4) * 8) * 2, fa);
 #pragma unroll
             for (int jj = 0; jj < 2; ++jj) {
-                uint32_t fb[4];   // two 8-token tiles of k rows: (k low, k high) each
-                ldsm4(kb + (c0 + 16 * jj + (lane & 7) + (lane >> 4) * 8) * L.qrow + (k0 + ((lane >> 3) & 1) * 8) * 2, fb);
                 if (c0 + 16 * jj <= r0 + 15) {
+                    uint32_t fb[4];   // two 8-token tiles of k rows: (k low, k high) each
+                    ldsm4(kb + (c0 + 16 * jj + (lane & 7) + (lane >> 4) * 8) * L.qrow + (k0 + ((lane >> 3) & 1) * 8) * 2, fb);
                     mma_bf16(sc[2 * jj], fa[0], fa[1], fa[2], fa[3], fb[0], fb[1]);
                     mma_bf16(sc[2 * jj + 1], fa[0], fa[1], fa[2], fa[3], fb[2], fb[3]);
                 }
+            }
+#pragma unroll
+            for (int jj = 0; jj < NJ / 2; ++jj)
 #pragma unroll
                 for (int part = 0; part < 2; ++part) {
                     uint32_t fs[4];
-                    ldsm4t(sb + L.s_off + part * NP * kVRow + (k0 + (lane & 15)) * kVRow + (c0 + 16 * jj + (lane >> 4) * 8) * 2, fs);
+                    ldsm4t(sb + L.s_off + part * NP * kVRow + (k0 + (lane & 15)) * kVRow + (o0 + 16 * jj + (lane >> 4) * 8) * 2, fs);
                     mma_bf16(out[2 * jj], fa[0], fa[1], fa[2], fa[3], fs[0], fs[1]);
                     mma_bf16(out[2 * jj + 1], fa[0], fa[1], fa[2], fa[3], fs[2], fs[3]);
                 }
-            }
         }
-        const float e0 = expf(cg0), e1 = expf(cg1);
+        const float e0 = exp2f(cg0), e1 = exp2f(cg1);
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) { out[j][0] *= e0; out[j][1] *= e0; out[j][2] *= e1; out[j][3] *= e1; }
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-            out[j][0] *= e0; out[j][1] *= e0; out[j][2] *= e1; out[j][3] *= e1;
-            const int col = c0 + 8 * j + 2 * q4;
+            const int col = c0 + 8 * j + 2 * q4, ra = r0 + g, rb = ra + 8;
             const float cc0 = cum[col], cc1 = cum[col + 1], w0 = wt[col], w1 = wt[col + 1];
-            const int ra = r0 + g, rb = ra + 8;
-            const float p0 = col <= ra ? sc[j][0] * expf(cg0 - cc0) * w0 : 0.f, p1 = col + 1 <= ra ? sc[j][1] * expf(cg0 - cc1) * w1 : 0.f;
-            const float p2 = col <= rb ? sc[j][2] * expf(cg1 - cc0) * w0 : 0.f, p3 = col + 1 <= rb ? sc[j][3] * expf(cg1 - cc1) * w1 : 0.f;
+            const float p0 = col <= ra ? sc[j][0] * exp2f(cg0 - cc0) * w0 : 0.f, p1 = col + 1 <= ra ? sc[j][1] * exp2f(cg0 - cc1) * w1 : 0.f;
+            const float p2 = col <= rb ? sc[j][2] * exp2f(cg1 - cc0) * w0 : 0.f, p3 = col + 1 <= rb ? sc[j][3] * exp2f(cg1 - cc1) * w1 : 0.f;
             uint32_t hi, lo;
             unsigned char* pd = smem + L.p_off + ra * kPRow + col * 2;
             split_bf16(p0, p1, hi, lo);
@@ -302,15 +314,16 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
             *reinterpret_cast<uint32_t*>(pd + 8 * kPRow + kChunk * kPRow) = lo;
         }
         // values weighted by what is left of them at the end of the chunk
-        for (int i = t; i < kChunk * kChV / 2; i += 256) {
-            const int row = i >> 5, col = (i & 31) * 2;
+        for (int i = t; i < kChunk * VT / 2; i += 256) {
+            const int row = i / (VT / 2), col = (i % (VT / 2)) * 2;
             const uint32_t vv = *reinterpret_cast<const uint32_t*>(smem + buf * L.buf + L.v_off + row * kVRow + col * 2);
-            const float f = expf(total - cum[row]) * wt[row];
+            const float f = exp2f(total - cum[row]) * wt[row];
             uint32_t hi, lo;
             split_bf16(__uint_as_float(vv << 16) * f, __uint_as_float(vv & 0xFFFF0000u) * f, hi, lo);
             *reinterpret_cast<uint32_t*>(smem + L.vw_off + row * kVRow + col * 2) = hi;
             *reinterpret_cast<uint32_t*>(smem + L.vw_off + (kChunk + row) * kVRow + col * 2) = lo;
         }
+        if (warp == 0) store_decay((ch + 1) & 1);
         __syncthreads();   // scores and weighted values written, old state copy read
 
         // within the chunk: out += P v
@@ -320,9 +333,9 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
             ldsm4(pa, ph);
             ldsm4(pa + kChunk * kPRow, pl);
 #pragma unroll
-            for (int jj = 0; jj < 2; ++jj) {
+            for (int jj = 0; jj < NJ / 2; ++jj) {
                 uint32_t fv[4];
-                ldsm4t(vb + (k0 + (lane & 15)) * kVRow + (c0 + 16 * jj + (lane >> 4) * 8) * 2, fv);
+                ldsm4t(vb + (k0 + (lane & 15)) * kVRow + (o0 + 16 * jj + (lane >> 4) * 8) * 2, fv);
                 mma_bf16(out[2 * jj], ph[0], ph[1], ph[2], ph[3], fv[0], fv[1]);
                 mma_bf16(out[2 * jj], pl[0], pl[1], pl[2], pl[3], fv[0], fv[1]);
                 mma_bf16(out[2 * jj + 1], ph[0], ph[1], ph[2], ph[3], fv[2], fv[3]);
@@ -331,10 +344,10 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
         }
         const float Dh = a.D ? a.D[h] : 0.f;
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
+        for (int j = 0; j < NJ; ++j)
 #pragma unroll
             for (int p = 0; p < 2; ++p) {
-                const int row = r0 + g + 8 * p, col = c0 + 8 * j + 2 * q4, tok = ch * kChunk + row;
+                const int row = r0 + g + 8 * p, col = o0 + 8 * j + 2 * q4, tok = ch * kChunk + row;
                 if (tok < r.T && v0 + col < V8) {
                     float2 o2 = make_float2(out[j][2 * p], out[j][2 * p + 1]);
                     if (a.D) {
@@ -346,13 +359,13 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
                 }
             }
         // state: S = exp(total) S + k^T (weighted v)
-        const float et = expf(total);
+        const float et = exp2f(total);
 #pragma unroll
         for (int i = 0; i < NTW; ++i) {
             const int n0 = 16 * (i * 8 + warp);
             if (n0 >= NP) continue;
 #pragma unroll
-            for (int j = 0; j < 8; ++j)
+            for (int j = 0; j < VT / 8; ++j)
 #pragma unroll
                 for (int p = 0; p < 4; ++p) S[i][j][p] *= et;
 #pragma unroll
@@ -360,7 +373,7 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
                 uint32_t fk[4];   // k^T: row n, column token
                 ldsm4t(kb + (k0 + (lane & 7) + (lane >> 4) * 8) * L.qrow + (n0 + ((lane >> 3) & 1) * 8) * 2, fk);
 #pragma unroll
-                for (int jj = 0; jj < 4; ++jj)
+                for (int jj = 0; jj < VT / 16; ++jj)
 #pragma unroll
                     for (int part = 0; part < 2; ++part) {
                         uint32_t fv[4];
@@ -371,14 +384,15 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
             }
         }
         state_to_smem();
-        if (nbuf == 1 || ch + 1 == nchunks) __syncthreads();
-        if (nbuf == 1 && ch + 1 < nchunks) issue(ch + 1, 0);
-        if (nbuf == 2) __syncthreads();   // cum / wt may be overwritten
+        if (nbuf == 1) {
+            __syncthreads();
+            if (ch + 1 < nchunks) issue(ch + 1, 0);
+        }
     }
 #pragma unroll
     for (int i = 0; i < NTW; ++i)
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
+        for (int j = 0; j < VT / 8; ++j)
 #pragma unroll
             for (int p = 0; p < 2; ++p) {
                 const int n = 16 * (i * 8 + warp) + g + 8 * p, v = 8 * j + 2 * q4;

@@ -150,6 +150,8 @@ SINGLE = {   # one mixer each, sizes that are not multiples of anything
     "mamba2_wide_state": lambda: config(64, 70, [mamba2(2, 72, 200, 1, 3, 4)], [None]),
     "retention": lambda: config(44, 71, [retention(3, 20, 36, [0.9, 0.99, 0.999])], [None]),
     "retention_edges": lambda: config(48, 64, [retention(4, 136, 8, [0.0, 1.0, 0.5, 0.96875])], [28]),
+    "mamba2_many_heads": lambda: config(48, 64, [mamba2(76, 40, 136, 4, 4, 19)], [None]),
+    "retention_many_heads": lambda: config(48, 64, [retention(80, 20, 40, list(np.linspace(0.5, 1.0, 80)))], [None]),
     "latent": lambda: config(56, 79, [latent(3, 12, 6, 36, 20, 0.25)], [None]),
     "latent_many_heads": lambda: config(72, 90, [latent(21, 8, 4, 24, 12, 0.3, base=500.0)], [40]),
     "latent_wide_values": lambda: config(64, 64, [latent(2, 40, 24, 264, 150, 0.12)], [None]),

@@ -107,6 +107,20 @@ def test_mechanism_alone(cuda, tmp_path, name, f32):
     d.close()
 
 
+@pytest.mark.parametrize("vdim", [40, 100])
+def test_long_prompt_many_heads(cuda, tmp_path, vdim):
+    """Prompts long enough for the attention kernel's tall blocks, cut in unequal parts and whole."""
+    m = lm.Model(tmp_path, lm.config(40, 50, [lm.latent(40, 12, 6, 24, vdim, 0.3)], [None]), 4)
+    tok = tokens_for(m, 1100)
+    want, bar = m.plain(tok)[0], m.bar(tok, False)
+    d = driver(m, False, max_seq=1100)
+    for cuts in ([1100], [37, 1063], [1030, 17, 1]):
+        d.release(0)
+        err = lm.rel_error(run(d, 0, tok, cuts), want)
+        assert err.max() < bar, (cuts, int(err.argmax()), err.max(), bar)
+    d.close()
+
+
 @both
 def test_layers_one_by_one(cuda, tmp_path, f32):
     m = lm.Model(tmp_path, lm.mixed(), 6)
