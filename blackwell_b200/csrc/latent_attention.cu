@@ -18,16 +18,17 @@ cudaError_t allow_smem(F kern, std::once_flag (&once)[kMaxDevices]) {
     return e;
 }
 
-template <typename A, int RB>
+template <typename A, int RB, int COLS>
 cudaError_t prep(const LatentArgs& a, const Rows& r, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
-    cudaError_t e = allow_smem(latent_prep_kernel<A, RB>, once);
+    auto kern = latent_prep_kernel<A, RB, COLS>;
+    cudaError_t e = allow_smem(kern, once);
     if (e != cudaSuccess) return e;
-    const int cblocks = (pad8(a.R) + kPrepCols - 1) / kPrepCols;
-    const size_t smem = (size_t)(RB * (pad8(a.dim) + pad8(a.rot)) + 8 * RB * kPrepCols) * 4;
+    const int cblocks = (pad8(a.R) + COLS - 1) / COLS;
+    const size_t smem = (size_t)(RB * (pad8(a.dim) + pad8(a.rot)) + 8 * RB * kPrepThreads) * 4;
     if (smem > kMaxDynSmem) return cudaErrorInvalidValue;
     count_launch(1);
-    return launch_pdl(latent_prep_kernel<A, RB>, dim3(a.heads * cblocks + (a.dkv ? RB : 0), (r.T + RB - 1) / RB), dim3(kPrepThreads), smem, st, a, r);
+    return launch_pdl(kern, dim3(a.heads * cblocks + (a.dkv ? RB : 0), (r.T + RB - 1) / RB), dim3(kPrepThreads), smem, st, a, r);
 }
 
 template <typename A, int RB>
@@ -35,7 +36,7 @@ cudaError_t out(const LatentArgs& a, const Rows& r, int keys, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
     cudaError_t e = allow_smem(latent_out_kernel<A, RB>, once);
     if (e != cudaSuccess) return e;
-    const size_t smem = (size_t)(2 * RB * pad8(a.R) + ((RB * a.splits + 3) & ~3)) * 4;
+    const size_t smem = (size_t)(3 * RB * pad8(a.R) + ((RB * a.splits + 3) & ~3)) * 4;
     if (smem > kMaxDynSmem) return cudaErrorInvalidValue;
     count_launch(1);
     return launch_pdl(latent_out_kernel<A, RB>, dim3(a.heads * ((pad8(a.V) + kOutV - 1) / kOutV), (r.T + RB - 1) / RB), dim3(256), smem, st, a, r, keys);
@@ -66,7 +67,7 @@ cudaError_t flash(const LatentArgs& a, const Rows& r, cudaStream_t st) {
     if (e != cudaSuccess) return e;
     const int D = pad16(pad8(a.dim) + pad8(a.rot));
     count_launch(1);
-    return launch_pdl(kern, dim3((r.T + 128 * MT - 1) / (128 * MT), a.heads, (pad8(a.V) + VT * 8 - 1) / (VT * 8)), dim3(256),
+    return launch_pdl(kern, dim3(a.heads, (r.T + 128 * MT - 1) / (128 * MT), (pad8(a.V) + VT * 8 - 1) / (VT * 8)), dim3(256),
                       FlashSmem(D, VT, MT).total, st, a, r);
 }
 
@@ -81,13 +82,13 @@ int flash_vt(const LatentArgs& a) {
 }  // namespace
 
 bool latent_absorbed_supported(const LatentArgs& a) {
-    return a.R >= 1 && a.R <= 2048 && (size_t)(pad8(a.dim) + pad8(a.rot) + 8 * kPrepCols) * 4 <= (size_t)kMaxDynSmem;
+    return a.R >= 1 && a.R <= 2048 && (size_t)(pad8(a.dim) + pad8(a.rot) + 8 * kPrepThreads) * 4 <= (size_t)kMaxDynSmem;
 }
 bool latent_expanded_supported(const LatentArgs& a) { return flash_vt(a) > 0; }
 
 cudaError_t latent_absorbed(const LatentArgs& a, const Rows& r, int f32, cudaStream_t st) {
     const bool rb4 = r.T >= 8 && !f32 && a.R <= 1024 && (pad8(a.dim) + pad8(a.rot)) <= 1024;
-    cudaError_t e = f32 ? prep<float, 1>(a, r, st) : rb4 ? prep<bf16, 4>(a, r, st) : prep<bf16, 1>(a, r, st);
+    cudaError_t e = f32 ? prep<float, 1, 64>(a, r, st) : rb4 ? prep<bf16, 4, 256>(a, r, st) : prep<bf16, 1, 64>(a, r, st);
     if (e != cudaSuccess) return e;
     const int nbuf = DecodeSmem(a.R, a.rot, 2).total <= kMaxDynSmem ? 2 : 1;
     const bool by_scalar = f32 || a.R > 1024 || DecodeSmem(a.R, a.rot, nbuf).total > kMaxDynSmem;

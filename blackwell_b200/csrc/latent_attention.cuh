@@ -69,16 +69,15 @@ __global__ void __launch_bounds__(128) latent_rotate_q_kernel(const LatentArgs a
 
 // ------------------------------------------------------------------------------------------ absorbed form
 constexpr int kPrepThreads = 256;
-constexpr int kPrepCols = 64;    // latent columns per block
 
-// Block (head, 64 latent columns; RB rows): q_abs = W_uk^T q, and from the first column block the rotated part.  RB more
-// blocks per row group write the cache entries.  8 threads cover the columns, 32 groups of threads the query dimensions;
-// the weights are fetched before the kernel waits for its predecessor.
-template <typename A, int RB>
+// Block (head, COLS latent columns; RB rows): q_abs = W_uk^T q, and from the first column block the rotated part.  RB more
+// blocks per row group write the cache entries.  COLS / 8 threads cover the columns, the others split the query
+// dimensions; the first weights are fetched before the kernel waits for its predecessor.
+template <typename A, int RB, int COLS>
 __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentArgs a, const Rows r) {
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     const int dim8 = pad8(a.dim), rot8 = pad8(a.rot), R8 = pad8(a.R), Dp = latent_dp(a.R, a.rot);
-    const int cblocks = (R8 + kPrepCols - 1) / kPrepCols, t = threadIdx.x, warp = t >> 5, lane = t & 31;
+    const int cblocks = (R8 + COLS - 1) / COLS, t = threadIdx.x;
     const int h = blockIdx.x / cblocks, cb = blockIdx.x - h * cblocks, row0 = blockIdx.y * RB;
     pdl_trigger();
     if (h >= a.heads) {
@@ -87,16 +86,17 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentA
         if (row < r.T) write_entry<A>(a, r, row, sm);
         return;
     }
-    constexpr int kPre = 4;
-    const int col = cb * kPrepCols + (lane & 7) * 8, grp = warp * 4 + (lane >> 3);
+    constexpr int TC = COLS / 8, GR = kPrepThreads / TC;   // threads across the columns, groups over the dimensions
+    constexpr int kPre = RB > 1 ? 8 : 4;
+    const int col = cb * COLS + (t % TC) * 8, grp = t / TC;
     const bf16* W = a.Wkv + (long)h * dim8 * a.ldw + col;
     uint4 pre[kPre];
 #pragma unroll
     for (int i = 0; i < kPre; ++i)
-        pre[i] = col < R8 && grp + 32 * i < a.dim ? __ldg(reinterpret_cast<const uint4*>(W + (long)(grp + 32 * i) * a.ldw)) : make_uint4(0, 0, 0, 0);
+        pre[i] = col < R8 && grp + GR * i < a.dim ? __ldg(reinterpret_cast<const uint4*>(W + (long)(grp + GR * i) * a.ldw)) : make_uint4(0, 0, 0, 0);
     pdl_wait();
-    float* qs = sm;                                   // [RB][dim8 + rot8]
-    float* red = qs + RB * (dim8 + rot8);             // [8 warps][RB][kPrepCols]
+    float* qs = sm;                                   // [dim8 + rot8][RB]
+    float* red = qs + RB * (dim8 + rot8);             // [GR][RB][COLS]
     for (int i = t; i < RB * (dim8 + rot8); i += kPrepThreads) {
         const int b = i / (dim8 + rot8), d = i - b * (dim8 + rot8);
         float v = 0.f;
@@ -109,41 +109,36 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentA
                 v = rot_elem(a.cs + (long)max(p, 0) * (a.rot_dims / 2), e, v, to_f(q[d ^ 1]));
             }
         }
-        qs[i] = v;
+        qs[d * RB + b] = v;
     }
     __syncthreads();
     float acc[RB][8] = {};
     auto add = [&](const uint4& w, int d) {
         const uint32_t ww[4] = {w.x, w.y, w.z, w.w};
+        float q[RB];
+        if (RB == 4) *reinterpret_cast<float4*>(q) = *reinterpret_cast<const float4*>(qs + d * RB);
+        else
 #pragma unroll
-        for (int b = 0; b < RB; ++b) {
-            const float q = qs[b * (dim8 + rot8) + d];
+            for (int b = 0; b < RB; ++b) q[b] = qs[d * RB + b];
+#pragma unroll
+        for (int b = 0; b < RB; ++b)
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                acc[b][2 * j] = fmaf(q, __uint_as_float(ww[j] << 16), acc[b][2 * j]);
-                acc[b][2 * j + 1] = fmaf(q, __uint_as_float(ww[j] & 0xFFFF0000u), acc[b][2 * j + 1]);
+                acc[b][2 * j] = fmaf(q[b], __uint_as_float(ww[j] << 16), acc[b][2 * j]);
+                acc[b][2 * j + 1] = fmaf(q[b], __uint_as_float(ww[j] & 0xFFFF0000u), acc[b][2 * j + 1]);
             }
-        }
     };
 #pragma unroll
     for (int i = 0; i < kPre; ++i)
-        if (grp + 32 * i < a.dim) add(pre[i], grp + 32 * i);
+        if (grp + GR * i < a.dim) add(pre[i], grp + GR * i);
     if (col < R8)
-        for (int d = grp + 32 * kPre; d < a.dim; d += 32) add(__ldg(reinterpret_cast<const uint4*>(W + (long)d * a.ldw)), d);
+#pragma unroll 4
+        for (int d = grp + GR * kPre; d < a.dim; d += GR) add(__ldg(reinterpret_cast<const uint4*>(W + (long)d * a.ldw)), d);
 #pragma unroll
-    for (int b = 0; b < RB; ++b)
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            acc[b][j] += __shfl_xor_sync(0xffffffffu, acc[b][j], 8);
-            acc[b][j] += __shfl_xor_sync(0xffffffffu, acc[b][j], 16);
-        }
-    if (lane < 8) {
-#pragma unroll
-        for (int b = 0; b < RB; ++b) {
-            float* o = red + (warp * RB + b) * kPrepCols + lane * 8;
-#pragma unroll
-            for (int j = 0; j < 8; ++j) o[j] = acc[b][j];
-        }
+    for (int b = 0; b < RB; ++b) {
+        float* o = red + (grp * RB + b) * COLS + (t % TC) * 8;
+        *reinterpret_cast<float4*>(o) = make_float4(acc[b][0], acc[b][1], acc[b][2], acc[b][3]);
+        *reinterpret_cast<float4*>(o + 4) = make_float4(acc[b][4], acc[b][5], acc[b][6], acc[b][7]);
     }
     __syncthreads();
     auto put = [&](int b, int d, float v) {
@@ -157,18 +152,18 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentA
             o[Dp] = __float2bfloat16_rn(v - __bfloat162float(hi));
         }
     };
-    for (int i = t; i < RB * kPrepCols; i += kPrepThreads) {
-        const int b = i / kPrepCols, c = i - b * kPrepCols;
-        if (row0 + b >= r.T || cb * kPrepCols + c >= R8) continue;
+    for (int i = t; i < RB * COLS; i += kPrepThreads) {
+        const int b = i / COLS, c = i % COLS;
+        if (row0 + b >= r.T || cb * COLS + c >= R8) continue;
         float v = 0.f;
 #pragma unroll
-        for (int w = 0; w < 8; ++w) v += red[(w * RB + b) * kPrepCols + c];
-        put(b, cb * kPrepCols + c, v);
+        for (int w = 0; w < GR; ++w) v += red[(w * RB + b) * COLS + c];
+        put(b, cb * COLS + c, v);
     }
     if (cb == 0)
         for (int i = t; i < RB * (Dp - R8); i += kPrepThreads) {
             const int b = i / (Dp - R8), e = i - b * (Dp - R8);
-            if (row0 + b < r.T) put(b, R8 + e, e < rot8 ? qs[b * (dim8 + rot8) + dim8 + e] : 0.f);
+            if (row0 + b < r.T) put(b, R8 + e, e < rot8 ? qs[(dim8 + e) * RB + b] : 0.f);
         }
 }
 
@@ -243,21 +238,24 @@ __global__ void __launch_bounds__(256) latent_scalar_kernel(const LatentArgs a, 
 
 constexpr int kDecKeys = 64;
 constexpr int kDecP = kDecKeys * 2 + 16;   // bytes of a row of softmax weights
+constexpr int kDecS = kDecKeys + 4;        // floats of a row of partial scores
 struct DecodeSmem {
-    int row, q_off, k_off, kbuf, p_off, f_off, total;
+    int row, q_off, k_off, kbuf, p_off, s_off, f_off, total;
     __host__ __device__ DecodeSmem(int R, int rot, int nbuf) {
         row = latent_dp(R, rot) * 2 + 16;
         q_off = 0;
         k_off = 2 * 16 * row;
         kbuf = kDecKeys * row;
         p_off = k_off + nbuf * kbuf;
-        f_off = p_off + 2 * 16 * kDecP;
-        total = f_off + 2 * 8 * 16 * 4;
+        s_off = p_off + 2 * 16 * kDecP;
+        f_off = s_off + 8 * 16 * kDecS * 4;
+        total = f_off + 16 * 4;
     }
 };
 
-// Block (split, 16 heads, row); 8 warps: warp w scores keys 8w .. 8w+7 of a 64-key tile and accumulates latent columns
-// [w * NT * 8, (w + 1) * NT * 8).
+// Block (split, 16 heads, row); 8 warps.  Scores: a warp takes every eighth 16-wide step of the query / key dimension for
+// all 64 keys of a tile, and the partial scores meet in shared memory, where 16 neighbouring threads own one head's row
+// (softmax without further exchange).  Output: a warp accumulates latent columns [w * NT * 8, (w + 1) * NT * 8).
 template <int NT>
 __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, const Rows r, int nbuf) {
     extern __shared__ __align__(16) unsigned char smem[];
@@ -266,8 +264,8 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, q4 = lane & 3;
     const int split = blockIdx.x, h0 = blockIdx.y * 16, row = blockIdx.z;
     const uint32_t sb = smem_u32(smem);
-    float* redm = reinterpret_cast<float*>(smem + L.f_off);   // [8][16]
-    float* redl = redm + 8 * 16;
+    float* part = reinterpret_cast<float*>(smem + L.s_off);    // [8][16][kDecS]
+    float* alphas = reinterpret_cast<float*>(smem + L.f_off);  // [16]
     pdl_trigger();
     pdl_wait();
     const int slot = r.slot_of(row), len = min(r.pos_of(row) + 1, a.max_seq);
@@ -276,94 +274,87 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
     if (slot < 0 || t0 >= t1) return;   // the merge reads the splits that hold positions
     const bf16* cache = static_cast<const bf16*>(a.cache) + (long)slot * a.max_seq * a.ldc;
     const int nc = Dp / 8;
+    const RowWalk walk(t, 256, nc);
     auto issue = [&](int tile, int buf) {
-        for (int i = t; i < kDecKeys * nc; i += 256) {
-            const int k = i / nc, c = (i - k * nc) * 8, key = tile * kDecKeys + k;
-            const bool ok = key < len && c < D8;
-            cp_async16z(sb + L.k_off + buf * L.kbuf + k * L.row + c * 2, ok ? cache + (long)key * a.ldc + c : cache, ok);
+        const uint32_t dst = sb + L.k_off + buf * L.kbuf;
+        for (RowWalk w = walk; w.row < kDecKeys; w.next()) {
+            const int key = tile * kDecKeys + w.row;
+            const bool ok = key < len && w.col * 8 < D8;
+            cp_async16z(dst + w.row * L.row + w.col * 16, ok ? cache + (long)key * a.ldc + w.col * 8 : cache, ok);
         }
         cp_async_commit();
     };
-    for (int i = t; i < 2 * 16 * nc; i += 256) {
-        const int part = i / (16 * nc), rem = i - part * 16 * nc, hh = rem / nc, c = (rem - hh * nc) * 8;
+    for (RowWalk w = walk; w.row < 32; w.next()) {   // 16 heads' high parts, then their remainders
+        const int hh = w.row & 15, lo = w.row >> 4;
         const bool ok = h0 + hh < a.heads;
         const bf16* q = static_cast<const bf16*>(a.qabs);
-        cp_async16z(sb + L.q_off + (part * 16 + hh) * L.row + c * 2, ok ? q + (((long)row * a.heads + h0 + hh) * 2 + part) * Dp + c : q, ok);
+        cp_async16z(sb + L.q_off + w.row * L.row + w.col * 16, ok ? q + (((long)row * a.heads + h0 + hh) * 2 + lo) * Dp + w.col * 8 : q, ok);
     }
     issue(t0, 0);
     float O[NT][4] = {};
-    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+    const int srow = t >> 4, skey = (t & 15) * 4;     // this thread's head row and keys in the softmax
+    float m = -INFINITY, l = 0.f;
     for (int tile = t0; tile < t1; ++tile) {
         const int buf = nbuf == 2 ? (tile - t0) & 1 : 0;
         const uint32_t kb = sb + L.k_off + buf * L.kbuf;
         cp_async_wait<0>();
         __syncthreads();
         if (nbuf == 2 && tile + 1 < t1) issue(tile + 1, buf ^ 1);
-        float s[4] = {}, sl[4] = {}, s2[4] = {}, sl2[4] = {};   // four independent chains
-        const uint32_t qa = sb + L.q_off + (lane & 15) * L.row + (lane >> 4) * 16;
-        const uint32_t ka = kb + (8 * warp + (lane & 7)) * L.row + (lane >> 3) * 16;
-        int k0 = 0;
-#pragma unroll 4
-        for (; k0 + 32 <= Dp; k0 += 32) {
-            uint32_t ah[4], al[4], bh[4], bl[4], b[4];
-            ldsm4(ka + k0 * 2, b);
-            ldsm4(qa + k0 * 2, ah);
-            ldsm4(qa + 16 * L.row + k0 * 2, al);
-            ldsm4(qa + k0 * 2 + 32, bh);
-            ldsm4(qa + 16 * L.row + k0 * 2 + 32, bl);
-            mma_bf16(s, ah[0], ah[1], ah[2], ah[3], b[0], b[1]);
-            mma_bf16(sl, al[0], al[1], al[2], al[3], b[0], b[1]);
-            mma_bf16(s2, bh[0], bh[1], bh[2], bh[3], b[2], b[3]);
-            mma_bf16(sl2, bl[0], bl[1], bl[2], bl[3], b[2], b[3]);
-        }
-        if (k0 < Dp) {
-            uint32_t ah[4], al[4], b[2];
-            ldsm4(qa + k0 * 2, ah);
-            ldsm4(qa + 16 * L.row + k0 * 2, al);
-            ldsm2(kb + (8 * warp + (lane & 7)) * L.row + (k0 + ((lane >> 3) & 1) * 8) * 2, b);
-            mma_bf16(s, ah[0], ah[1], ah[2], ah[3], b[0], b[1]);
-            mma_bf16(sl, al[0], al[1], al[2], al[3], b[0], b[1]);
+        float s[8][4] = {};
+        for (int k0 = warp * 16; k0 < Dp; k0 += 128) {
+            uint32_t ah[4], al[4];
+            const uint32_t qa = sb + L.q_off + (lane & 15) * L.row + (k0 + (lane >> 4) * 8) * 2;
+            ldsm4(qa, ah);
+            ldsm4(qa + 16 * L.row, al);
+            const uint32_t ka = kb + ((lane & 7) + (lane >> 4) * 8) * L.row + (k0 + ((lane >> 3) & 1) * 8) * 2;
+            uint32_t b[4][4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) ldsm4(ka + 16 * j * L.row, b[j]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                mma_bf16(s[2 * j], ah[0], ah[1], ah[2], ah[3], b[j][0], b[j][1]);
+                mma_bf16(s[2 * j + 1], ah[0], ah[1], ah[2], ah[3], b[j][2], b[j][3]);
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                mma_bf16(s[2 * j], al[0], al[1], al[2], al[3], b[j][0], b[j][1]);
+                mma_bf16(s[2 * j + 1], al[0], al[1], al[2], al[3], b[j][2], b[j][3]);
+            }
         }
 #pragma unroll
-        for (int i = 0; i < 4; ++i) s[i] = (s[i] + s2[i]) + (sl[i] + sl2[i]);
-        const int key = tile * kDecKeys + 8 * warp + 2 * q4;
-#pragma unroll
-        for (int i = 0; i < 4; ++i) s[i] = key + (i & 1) < len ? s[i] * a.scale : -INFINITY;
-        float x0 = fmaxf(s[0], s[1]), x1 = fmaxf(s[2], s[3]);
-#pragma unroll
-        for (int o = 1; o <= 2; o <<= 1) {
-            x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, o));
-            x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, o));
+        for (int j = 0; j < 8; ++j) {
+            float* p = part + (warp * 16 + g) * kDecS + 8 * j + 2 * q4;
+            *reinterpret_cast<float2*>(p) = make_float2(s[j][0], s[j][1]);
+            *reinterpret_cast<float2*>(p + 8 * kDecS) = make_float2(s[j][2], s[j][3]);
         }
-        if (q4 == 0) { redm[warp * 16 + g] = x0; redm[warp * 16 + g + 8] = x1; }
         __syncthreads();
-        float n0 = m0, n1 = m1;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-        for (int w = 0; w < 8; ++w) { n0 = fmaxf(n0, redm[w * 16 + g]); n1 = fmaxf(n1, redm[w * 16 + g + 8]); }
-        const float al0 = expf(m0 - n0), al1 = expf(m1 - n1);   // the tile's first key is always visible: n is finite
-        m0 = n0;
-        m1 = n1;
-        const float p0 = expf(s[0] - n0), p1 = expf(s[1] - n0), p2 = expf(s[2] - n1), p3 = expf(s[3] - n1);
-        uint32_t hi, lo;
-        unsigned char* pd = smem + L.p_off + g * kDecP + (8 * warp + 2 * q4) * 2;
-        split_bf16(p0, p1, hi, lo);
-        *reinterpret_cast<uint32_t*>(pd) = hi;
-        *reinterpret_cast<uint32_t*>(pd + 16 * kDecP) = lo;
-        split_bf16(p2, p3, hi, lo);
-        *reinterpret_cast<uint32_t*>(pd + 8 * kDecP) = hi;
-        *reinterpret_cast<uint32_t*>(pd + 24 * kDecP) = lo;
-        float y0 = p0 + p1, y1 = p2 + p3;
-#pragma unroll
-        for (int o = 1; o <= 2; o <<= 1) {
-            y0 += __shfl_xor_sync(0xffffffffu, y0, o);
-            y1 += __shfl_xor_sync(0xffffffffu, y1, o);
+        for (int w = 0; w < 8; ++w) {
+            const float4 y = *reinterpret_cast<const float4*>(part + (w * 16 + srow) * kDecS + skey);
+            x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
         }
-        if (q4 == 0) { redl[warp * 16 + g] = y0; redl[warp * 16 + g + 8] = y1; }
-        __syncthreads();
-        l0 *= al0;
-        l1 *= al1;
+        const int key = tile * kDecKeys + skey;
+        x.x = key < len ? x.x * a.scale : -INFINITY;
+        x.y = key + 1 < len ? x.y * a.scale : -INFINITY;
+        x.z = key + 2 < len ? x.z * a.scale : -INFINITY;
+        x.w = key + 3 < len ? x.w * a.scale : -INFINITY;
+        float mx = fmaxf(fmaxf(x.x, x.y), fmaxf(x.z, x.w));
 #pragma unroll
-        for (int w = 0; w < 8; ++w) { l0 += redl[w * 16 + g]; l1 += redl[w * 16 + g + 8]; }
+        for (int o = 1; o < 16; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        mx = fmaxf(mx, m);                           // finite: the first key of a tile is always visible
+        const float alpha = expf(m - mx);
+        m = mx;
+        x.x = expf(x.x - mx); x.y = expf(x.y - mx); x.z = expf(x.z - mx); x.w = expf(x.w - mx);
+        l = l * alpha + ((x.x + x.y) + (x.z + x.w));
+        uint2 hi, lo;
+        split_bf16(x.x, x.y, hi.x, lo.x);
+        split_bf16(x.z, x.w, hi.y, lo.y);
+        *reinterpret_cast<uint2*>(smem + L.p_off + srow * kDecP + skey * 2) = hi;
+        *reinterpret_cast<uint2*>(smem + L.p_off + (16 + srow) * kDecP + skey * 2) = lo;
+        if ((t & 15) == 0) alphas[srow] = alpha;
+        __syncthreads();
+        const float al0 = alphas[g], al1 = alphas[g + 8];
 #pragma unroll
         for (int j = 0; j < NT; ++j) { O[j][0] *= al0; O[j][1] *= al0; O[j][2] *= al1; O[j][3] *= al1; }
 #pragma unroll
@@ -400,10 +391,13 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
             const int col = (warp * NT + j) * 8 + 2 * q4;
             if (col < R8) *reinterpret_cast<float2*>(out + col) = make_float2(O[j][2 * p], O[j][2 * p + 1]);
         }
-        if (warp == 0 && q4 == 0) {
-            out[R8] = p ? m1 : m0;
-            out[R8 + 1] = p ? l1 : l0;
-        }
+    }
+#pragma unroll
+    for (int o = 1; o < 16; o <<= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+    if ((t & 15) == 0 && h0 + srow < a.heads) {
+        float* stats = part_ptr(a, row, h0 + srow, split) + R8;
+        stats[0] = m;
+        stats[1] = l;
     }
 }
 
@@ -472,49 +466,57 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, con
         *reinterpret_cast<float4*>((part ? red : lat) + b * R8 + c) = acc;
     }
     __syncthreads();
-    if (halves == 2) {
-        for (int i = t; i < RB * R8; i += 256) lat[i] += red[i];
-        __syncthreads();
+    // sum of the halves, stored as [row][4-column half][8-column block][4]: neighbouring lanes read neighbouring words
+    float* lat2 = red + RB * R8;
+    for (int i = t; i < RB * R8; i += 256) {
+        const int b = i / R8, c = i - b * R8;
+        lat2[b * R8 + ((c >> 2) & 1) * (R8 / 2) + (c >> 3) * 4 + (c & 3)] = halves == 2 ? lat[i] + red[i] : lat[i];
     }
-    float acc[kVs][RB] = {};
-    auto add = [&](const uint4& w, int c, int i) {
-        const uint32_t ww[4] = {w.x, w.y, w.z, w.w};
+    __syncthreads();
+    float acc[kVs * RB] = {};
+    auto add = [&](const uint4 (&w)[kVs], int c) {
 #pragma unroll
         for (int b = 0; b < RB; ++b) {
-            const float4 x0 = *reinterpret_cast<const float4*>(lat + b * R8 + c);
-            const float4 x1 = *reinterpret_cast<const float4*>(lat + b * R8 + c + 4);
-            float s = acc[i][b];
-            s = fmaf(x0.x, __uint_as_float(ww[0] << 16), s);
-            s = fmaf(x0.y, __uint_as_float(ww[0] & 0xFFFF0000u), s);
-            s = fmaf(x0.z, __uint_as_float(ww[1] << 16), s);
-            s = fmaf(x0.w, __uint_as_float(ww[1] & 0xFFFF0000u), s);
-            s = fmaf(x1.x, __uint_as_float(ww[2] << 16), s);
-            s = fmaf(x1.y, __uint_as_float(ww[2] & 0xFFFF0000u), s);
-            s = fmaf(x1.z, __uint_as_float(ww[3] << 16), s);
-            s = fmaf(x1.w, __uint_as_float(ww[3] & 0xFFFF0000u), s);
-            acc[i][b] = s;
+            const float4 x0 = *reinterpret_cast<const float4*>(lat2 + b * R8 + (c >> 1));
+            const float4 x1 = *reinterpret_cast<const float4*>(lat2 + b * R8 + R8 / 2 + (c >> 1));
+#pragma unroll
+            for (int i = 0; i < kVs; ++i) {
+                float s = acc[i * RB + b];
+                s = fmaf(x0.x, __uint_as_float(w[i].x << 16), s);
+                s = fmaf(x0.y, __uint_as_float(w[i].x & 0xFFFF0000u), s);
+                s = fmaf(x0.z, __uint_as_float(w[i].y << 16), s);
+                s = fmaf(x0.w, __uint_as_float(w[i].y & 0xFFFF0000u), s);
+                s = fmaf(x1.x, __uint_as_float(w[i].z << 16), s);
+                s = fmaf(x1.y, __uint_as_float(w[i].z & 0xFFFF0000u), s);
+                s = fmaf(x1.z, __uint_as_float(w[i].w << 16), s);
+                s = fmaf(x1.w, __uint_as_float(w[i].w & 0xFFFF0000u), s);
+                acc[i * RB + b] = s;
+            }
         }
     };
 #pragma unroll
-    for (int i = 0; i < kVs; ++i) {
-        const int v = v0 + warp + 8 * i;
+    for (int j = 0; j < kPre; ++j)
+        if (lane * 8 + 256 * j < R8) {
+            uint4 w[kVs];
 #pragma unroll
-        for (int j = 0; j < kPre; ++j)
-            if (lane * 8 + 256 * j < R8) add(pre[i][j], lane * 8 + 256 * j, i);
-        if (v < a.V)
-            for (int c = lane * 8 + 256 * kPre; c < R8; c += 256) add(__ldg(reinterpret_cast<const uint4*>(W + (long)v * a.ldw + c)), c, i);
-    }
-#pragma unroll
-    for (int i = 0; i < kVs; ++i) {
-        const int v = v0 + warp + 8 * i;
-#pragma unroll
-        for (int b = 0; b < RB; ++b) {
-            const float s = warp_sum(acc[i][b]);
-            if (lane == 0 && v < V8 && row0 + b < r.T)
-                static_cast<A*>(a.out)[(long)(row0 + b) * a.ldout + h * V8 + v] =
-                    from_f<A>(v < a.V ? s * sigmoid_f(a.gate[(long)(row0 + b) * a.ld32 + h]) : 0.f);
+            for (int i = 0; i < kVs; ++i) w[i] = pre[i][j];
+            add(w, lane * 8 + 256 * j);
         }
+    for (int c = lane * 8 + 256 * kPre; c < R8; c += 256) {
+        uint4 w[kVs];
+#pragma unroll
+        for (int i = 0; i < kVs; ++i) {
+            const int v = v0 + warp + 8 * i;
+            w[i] = v < a.V ? __ldg(reinterpret_cast<const uint4*>(W + (long)v * a.ldw + c)) : make_uint4(0, 0, 0, 0);
+        }
+        add(w, c);
     }
+    const float s = warp_sum_many<kVs * RB>(acc, lane);   // lane -> one (value column, row)
+    const int idx = warp_sum_many_index<kVs * RB>(lane), v = v0 + warp + 8 * (idx / RB), row = row0 + idx % RB;
+    constexpr int kSpread = 32 / (kVs * RB);              // lanes that hold the same sum
+    if (lane % kSpread == 0 && v < V8 && row < r.T)
+        static_cast<A*>(a.out)[(long)row * a.ldout + h * V8 + v] =
+            from_f<A>(v < a.V ? s * sigmoid_f(a.gate[(long)row * a.ld32 + h]) : 0.f);
 }
 
 // ------------------------------------------------------------------------------------------ expanded form
@@ -539,7 +541,8 @@ __global__ void __launch_bounds__(256, 1) latent_flash_kernel(const LatentArgs a
     const int dim8 = pad8(a.dim), rot8 = pad8(a.rot), D8 = dim8 + rot8, D = pad16(D8), V8 = pad8(a.V), R8 = pad8(a.R);
     const FlashSmem L(D, VT, MT);
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, q4 = lane & 3;
-    const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kQ, h = blockIdx.y, v0 = blockIdx.z * VT * 8;
+    // heads fastest, longest rows first
+    const int q0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * kQ, h = blockIdx.x, v0 = blockIdx.z * VT * 8;
     const uint32_t sb = smem_u32(smem);
     const bf16* kv = static_cast<const bf16*>(a.kv);
     const long ldkv = (long)a.heads * (dim8 + V8);
@@ -549,26 +552,30 @@ __global__ void __launch_bounds__(256, 1) latent_flash_kernel(const LatentArgs a
     pdl_trigger();
     pdl_wait();
     const int nc = D / 8;
+    const RowWalk kwalk(t, 256, nc);
     auto issue = [&](int tile, int buf) {
         const uint32_t kb = sb + L.k_off + buf * L.kbuf, vb = kb + kFlashK * L.row;
-        for (int i = t; i < kFlashK * nc; i += 256) {
-            const int k = i / nc, c = (i - k * nc) * 8, key = tile * kFlashK + k;
+        for (RowWalk w = kwalk; w.row < kFlashK; w.next()) {
+            const int c = w.col * 8, key = tile * kFlashK + w.row;
             const bool ok = key < nkeys && c < D8;
             const bf16* src = c < dim8 ? kv + (long)key * ldkv + h * dim8 + c : kr + (long)key * a.ldc + (c - dim8);
-            cp_async16z(kb + k * L.row + c * 2, ok ? src : kv, ok);
+            cp_async16z(kb + w.row * L.row + c * 2, ok ? src : kv, ok);
         }
-        for (int i = t; i < kFlashK * VT; i += 256) {
-            const int k = i / VT, c = (i - k * VT) * 8, key = tile * kFlashK + k;
-            const bool ok = key < nkeys && v0 + c < V8;
-            cp_async16z(vb + k * L.vrow + c * 2, ok ? kv + (long)key * ldkv + a.heads * dim8 + h * V8 + v0 + c : kv, ok);
+        const int vc = (t % VT) * 8;                       // 256 is a multiple of VT: the column stays
+        const bool vok = v0 + vc < V8;
+        const bf16* vsrc = kv + a.heads * dim8 + h * V8 + v0 + vc;
+#pragma unroll
+        for (int k = t / VT; k < kFlashK; k += 256 / VT) {
+            const int key = tile * kFlashK + k;
+            const bool ok = vok && key < nkeys;
+            cp_async16z(vb + k * L.vrow + vc * 2, ok ? vsrc + (long)key * ldkv : kv, ok);
         }
         cp_async_commit();
     };
-    for (int i = t; i < kQ * nc; i += 256) {
-        const int q = i / nc, c = (i - q * nc) * 8;
-        const bool ok = q0 + q < r.T && c < D8;
+    for (RowWalk w = kwalk; w.row < kQ; w.next()) {
+        const bool ok = q0 + w.row < r.T && w.col * 8 < D8;
         const bf16* src = static_cast<const bf16*>(a.q);
-        cp_async16z(sb + q * L.row + c * 2, ok ? src + (long)(q0 + q) * a.ldq + h * D8 + c : src, ok);
+        cp_async16z(sb + w.row * L.row + w.col * 16, ok ? src + (long)(q0 + w.row) * a.ldq + h * D8 + w.col * 8 : src, ok);
     }
     issue(0, 0);
     float O[MT][VT][4] = {};
@@ -623,7 +630,7 @@ __global__ void __launch_bounds__(256, 1) latent_flash_kernel(const LatentArgs a
                         }
                     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
                     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-                    const float base = mx == -INFINITY ? 0.f : mx, alpha = exp2f(m[i][p] - base);
+                    const float base = mx == -INFINITY ? 0.f : mx, alpha = exp2_fast(m[i][p] - base);
                     m[i][p] = mx;
                     float sum = 0.f;
 #pragma unroll
@@ -631,7 +638,7 @@ __global__ void __launch_bounds__(256, 1) latent_flash_kernel(const LatentArgs a
 #pragma unroll
                         for (int e = 0; e < 2; ++e) {
                             float& x = s[i][j][2 * p + e];
-                            x = exp2f(x - base);
+                            x = exp2_fast(x - base);
                             sum += x;
                         }
                     l[i][p] = l[i][p] * alpha + sum;

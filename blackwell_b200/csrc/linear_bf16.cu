@@ -50,14 +50,14 @@ int stream_xs_stride(int ldw) {
     const int nkb = (ldw + 31) / 32;
     return nkb * 64 + (nkb % 2 == 0 ? 64 : 0);   // odd multiple of 64 bytes: conflict-free fragment reads
 }
-int stream_smem(int NT, int ldw) { return kStreamWarps * NT * 8 * 16 * 4 + NT * 8 * stream_xs_stride(ldw); }
+int stream_smem(int T, int NT, int ldw) { return kStreamWarps * NT * 8 * 16 * 4 + T * stream_xs_stride(ldw); }
 
 template <int NT>
 cudaError_t launch_stream(const LinearArgs& a, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
     cudaError_t e = allow_smem(linear_stream_kernel<NT>, once, kMaxDynSmem);
     if (e != cudaSuccess) return e;
-    const int smem = stream_smem(NT, (int)a.ldw), tiles = (a.N + 15) / 16;
+    const int smem = stream_smem(a.T, NT, (int)a.ldw), tiles = (a.N + 15) / 16;
     const int per_sm = smem > 110 * 1024 ? 1 : smem > 72 * 1024 ? 2 : 3;
     const int grid = std::min(tiles, sm_count(current_device()) * per_sm);
     e = launch_pdl(linear_stream_kernel<NT>, dim3(grid), dim3(kStreamWarps * 32), smem, st, a, stream_xs_stride((int)a.ldw));
@@ -115,7 +115,7 @@ cudaError_t linear(const LinearArgs& a, cudaStream_t st) {
     }
     if (a.ldx % 8 != 0) return cudaErrorInvalidValue;
     const int nt = a.T <= 8 ? 1 : a.T <= 16 ? 2 : 4;
-    if (a.T <= g_stream_max && stream_smem(nt, (int)a.ldw) <= kMaxDynSmem)
+    if (a.T <= g_stream_max && stream_smem(a.T, nt, (int)a.ldw) <= kMaxDynSmem)
         return nt == 1 ? launch_stream<1>(a, st) : nt == 2 ? launch_stream<2>(a, st) : launch_stream<4>(a, st);
     // enough tiles for the SMs: persistent tiles of 256 / 128 rows; otherwise the K range is split over a cluster
     const int sms = sm_count(current_device()), rtiles = (a.N + kTcRows - 1) / kTcRows, nk = (a.K + kTcK - 1) / kTcK;

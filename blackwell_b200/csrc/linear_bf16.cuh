@@ -40,7 +40,7 @@ template <int NT>  // 8-row tiles of the activations
 __global__ void __launch_bounds__(kStreamWarps * 32) linear_stream_kernel(const LinearArgs a, int xs_stride) {
     extern __shared__ __align__(16) unsigned char smem[];
     float* red = reinterpret_cast<float*>(smem);                         // [warps][NT * 8][16]
-    unsigned char* xs = smem + kStreamWarps * NT * 8 * 16 * 4;           // [NT * 8][xs_stride] bytes
+    unsigned char* xs = smem + kStreamWarps * NT * 8 * 16 * 4;           // [T][xs_stride] bytes
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, q = lane & 3;
     const int tiles = (a.N + 15) / 16, kw = (int)a.ldw;
     const int nkb = (kw + 31) / 32;
@@ -61,14 +61,14 @@ __global__ void __launch_bounds__(kStreamWarps * 32) linear_stream_kernel(const 
     if (tile < tiles) load(cur, tile, 0);
     pdl_trigger();
     pdl_wait();
-    // activations: rows >= T and columns >= K are zero
+    // activations: columns >= K are zero; rows >= T are not stored (their fragments are zero registers)
     const int kpad = nkb * 32;
-    for (int i = t; i < NT * 8 * (kpad / 8); i += kStreamWarps * 32) {
-        const int r = i / (kpad / 8), c = (i - r * (kpad / 8)) * 8;
+    const RowWalk walk(t, kStreamWarps * 32, kpad / 8);
+    for (RowWalk w = walk; w.row < a.T; w.next()) {
+        const int c = w.col * 8;
         uint4 v = zero4;
-        if (r < a.T && c < a.K) {
-            const bf16* src = static_cast<const bf16*>(a.x) + (long)r * a.ldx + c;
-            v = *reinterpret_cast<const uint4*>(src);
+        if (c < a.K) {
+            v = *reinterpret_cast<const uint4*>(static_cast<const bf16*>(a.x) + (long)w.row * a.ldx + c);
             if (c + 8 > a.K) {   // ragged end: keep only the real columns
                 uint32_t* e = reinterpret_cast<uint32_t*>(&v);
 #pragma unroll
@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(kStreamWarps * 32) linear_stream_kernel(const 
                 }
             }
         }
-        *reinterpret_cast<uint4*>(xs + (long)r * xs_stride + c * 2) = v;
+        *reinterpret_cast<uint4*>(xs + (long)w.row * xs_stride + c * 2) = v;
     }
     __syncthreads();
 
@@ -98,7 +98,8 @@ __global__ void __launch_bounds__(kStreamWarps * 32) linear_stream_kernel(const 
             if (kb < nkb) {
 #pragma unroll
                 for (int j = 0; j < NT; ++j) {
-                    const uint4 b = *reinterpret_cast<const uint4*>(xs + (long)(j * 8 + g) * xs_stride + (kb * 32 + q * 8) * 2);
+                    uint4 b = zero4;
+                    if (j * 8 + g < a.T) b = *reinterpret_cast<const uint4*>(xs + (j * 8 + g) * xs_stride + (kb * 32 + q * 8) * 2);
                     mma_bf16(acc[j], cur[u][0].x, cur[u][1].x, cur[u][0].y, cur[u][1].y, b.x, b.y);
                     mma_bf16(acc[j], cur[u][0].z, cur[u][1].z, cur[u][0].w, cur[u][1].w, b.z, b.w);
                 }

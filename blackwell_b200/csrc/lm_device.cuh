@@ -68,6 +68,25 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
         : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
+// 2^x by the hardware instruction (subnormal results become zero).
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// Walks the elements t, t + threads, t + 2 * threads, ... of a [rows][cols] array without a division per step.
+struct RowWalk {
+    int row, col, drow, dcol, cols;
+    __device__ __forceinline__ RowWalk(int t, int threads, int cols_)
+        : row(t / cols_), col(t % cols_), drow(threads / cols_), dcol(threads % cols_), cols(cols_) {}
+    __device__ __forceinline__ void next() {
+        row += drow;
+        col += dcol;
+        if (col >= cols) { col -= cols; ++row; }
+    }
+};
+
 // Sum over a block of up to 1024 threads; every thread gets the total.  `buf`: 32 floats of shared memory.
 __device__ __forceinline__ float block_sum(float v, float* buf) {
     v = warp_sum(v);

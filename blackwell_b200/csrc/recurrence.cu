@@ -53,9 +53,10 @@ bool recurrence_chunk_supported(const RecurrenceArgs& a) { return a.N <= 256 && 
 
 cudaError_t recurrence_chunk(const RecurrenceArgs& a, const Rows& r, cudaStream_t st) {
     if (a.groups < 1 || a.heads % a.groups != 0 || r.row_slot || !recurrence_chunk_supported(a)) return cudaErrorInvalidValue;
-    // narrow state tiles while the wide ones leave SMs idle, and where only they fit shared memory twice
-    const int wide = (pad8(a.V) + 63) / 64 * a.heads;
-    const bool narrow = a.V <= 32 || wide <= sm_count(current_device()) / 2 || ChunkSmem(a.N, 64, 1).total > kMaxDynSmem;
+    // narrow state tiles while the wide ones leave SMs idle or two narrow CTAs share an SM
+    const int wide = (pad8(a.V) + 63) / 64 * a.heads, sms = sm_count(current_device());
+    const bool pairs = ChunkSmem(a.N, 32, 2).total <= 112 * 1024;
+    const bool narrow = a.V <= 32 || wide <= (pairs ? sms : sms / 2) || ChunkSmem(a.N, 64, 1).total > kMaxDynSmem;
     if (pad16(a.N) <= 128) return narrow ? chunk_inst<1, 32>(a, r, st) : chunk_inst<1, 64>(a, r, st);
     return narrow ? chunk_inst<2, 32>(a, r, st) : chunk_inst<2, 64>(a, r, st);
 }

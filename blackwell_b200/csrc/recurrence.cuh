@@ -155,7 +155,7 @@ struct ChunkSmem {
         s_off = vw_off + 2 * kChunk * kVRow;       // state, high and remainder
         p_off = s_off + 2 * NP * kVRow;            // decayed scores, high and remainder
         f_off = p_off + 2 * kChunk * kPRow;        // cumulative log decay, weights
-        total = f_off + 2 * 2 * kChunk * 4;
+        total = f_off + 2 * 3 * kChunk * 4;
     }
 };
 
@@ -169,21 +169,21 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, q4 = lane & 3;
     const int h = blockIdx.y, v0 = blockIdx.x * VT, grp = h / (a.heads / a.groups);
     const uint32_t sb = smem_u32(smem);
-    float* dec = reinterpret_cast<float*>(smem + L.f_off);   // [2][cumulative log2 decay, weight][chunk]
+    float* dec = reinterpret_cast<float*>(smem + L.f_off);   // [2][cumulative log2 decay, weight, weight left at the end][chunk]
     const int nchunks = (r.T + kChunk - 1) / kChunk;
     const bf16* qg = static_cast<const bf16*>(a.q) + grp * N8;
     const bf16* kg = static_cast<const bf16*>(a.k) + grp * N8;
     const bf16* vg = static_cast<const bf16*>(a.v) + h * V8 + v0;
     pdl_wait();
 
+    const RowWalk walk(t, 256, NP / 8);
     auto issue = [&](int ch, int buf) {
         const uint32_t base = sb + buf * L.buf;
-        const int nc = NP / 8;
-        for (int i = t; i < kChunk * nc; i += 256) {
-            const int row = i / nc, col = (i - row * nc) * 8, tok = ch * kChunk + row;
+        for (RowWalk w = walk; w.row < kChunk; w.next()) {
+            const int col = w.col * 8, tok = ch * kChunk + w.row;
             const bool ok = tok < r.T && col < N8;
-            cp_async16z(base + row * L.qrow + col * 2, ok ? qg + (long)tok * a.ldq + col : qg, ok);
-            cp_async16z(base + L.k_off + row * L.qrow + col * 2, ok ? kg + (long)tok * a.ldk + col : kg, ok);
+            cp_async16z(base + w.row * L.qrow + col * 2, ok ? qg + (long)tok * a.ldq + col : qg, ok);
+            cp_async16z(base + L.k_off + w.row * L.qrow + col * 2, ok ? kg + (long)tok * a.ldk + col : kg, ok);
         }
         for (int i = t; i < kChunk * (VT / 8); i += 256) {
             const int row = i / (VT / 8), col = (i % (VT / 8)) * 8, tok = ch * kChunk + row;
@@ -232,11 +232,11 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
             const float up = __shfl_up_sync(0xffffffffu, s, o);
             if (lane >= o) s += up;
         }
-        float* cum = dec + buf * 2 * kChunk;
-        cum[2 * lane] = (s - pair) + l0;
-        cum[2 * lane + 1] = s;
-        cum[kChunk + 2 * lane] = w[0];
-        cum[kChunk + 2 * lane + 1] = w[1];
+        const float first = (s - pair) + l0, total = __shfl_sync(0xffffffffu, s, 31);
+        float* cum = dec + buf * 3 * kChunk;
+        *reinterpret_cast<float2*>(cum + 2 * lane) = make_float2(first, s);
+        *reinterpret_cast<float2*>(cum + kChunk + 2 * lane) = make_float2(w[0], w[1]);
+        *reinterpret_cast<float2*>(cum + 2 * kChunk + 2 * lane) = make_float2(exp2_fast(total - first) * w[0], exp2_fast(total - s) * w[1]);
     };
     issue(0, 0);
     if (warp == 0) {
@@ -264,7 +264,7 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
         __syncthreads();   // operands, state copy and decays are in shared memory
         if (nbuf == 2 && ch + 1 < nchunks) issue(ch + 1, buf ^ 1);
         if (warp == 0) load_decay(ch + 1);
-        const float *cum = dec + (ch & 1) * 2 * kChunk, *wt = cum + kChunk;
+        const float *cum = dec + (ch & 1) * 3 * kChunk, *wt = cum + kChunk, *left = wt + kChunk;
         const float total = cum[kChunk - 1];
         const int r0 = 16 * (warp & 3), c0 = 32 * (warp >> 2);   // score columns; output columns start at
         const int o0 = (VT / 2) * (warp >> 2);
@@ -295,15 +295,15 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
                     mma_bf16(out[2 * jj + 1], fa[0], fa[1], fa[2], fa[3], fs[2], fs[3]);
                 }
         }
-        const float e0 = exp2f(cg0), e1 = exp2f(cg1);
+        const float e0 = exp2_fast(cg0), e1 = exp2_fast(cg1);
 #pragma unroll
         for (int j = 0; j < NJ; ++j) { out[j][0] *= e0; out[j][1] *= e0; out[j][2] *= e1; out[j][3] *= e1; }
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int col = c0 + 8 * j + 2 * q4, ra = r0 + g, rb = ra + 8;
             const float cc0 = cum[col], cc1 = cum[col + 1], w0 = wt[col], w1 = wt[col + 1];
-            const float p0 = col <= ra ? sc[j][0] * exp2f(cg0 - cc0) * w0 : 0.f, p1 = col + 1 <= ra ? sc[j][1] * exp2f(cg0 - cc1) * w1 : 0.f;
-            const float p2 = col <= rb ? sc[j][2] * exp2f(cg1 - cc0) * w0 : 0.f, p3 = col + 1 <= rb ? sc[j][3] * exp2f(cg1 - cc1) * w1 : 0.f;
+            const float p0 = col <= ra ? sc[j][0] * exp2_fast(cg0 - cc0) * w0 : 0.f, p1 = col + 1 <= ra ? sc[j][1] * exp2_fast(cg0 - cc1) * w1 : 0.f;
+            const float p2 = col <= rb ? sc[j][2] * exp2_fast(cg1 - cc0) * w0 : 0.f, p3 = col + 1 <= rb ? sc[j][3] * exp2_fast(cg1 - cc1) * w1 : 0.f;
             uint32_t hi, lo;
             unsigned char* pd = smem + L.p_off + ra * kPRow + col * 2;
             split_bf16(p0, p1, hi, lo);
@@ -317,7 +317,7 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
         for (int i = t; i < kChunk * VT / 2; i += 256) {
             const int row = i / (VT / 2), col = (i % (VT / 2)) * 2;
             const uint32_t vv = *reinterpret_cast<const uint32_t*>(smem + buf * L.buf + L.v_off + row * kVRow + col * 2);
-            const float f = exp2f(total - cum[row]) * wt[row];
+            const float f = left[row];
             uint32_t hi, lo;
             split_bf16(__uint_as_float(vv << 16) * f, __uint_as_float(vv & 0xFFFF0000u) * f, hi, lo);
             *reinterpret_cast<uint32_t*>(smem + L.vw_off + row * kVRow + col * 2) = hi;
@@ -359,7 +359,7 @@ __global__ void __launch_bounds__(256) recurrence_chunk_kernel(const RecurrenceA
                 }
             }
         // state: S = exp(total) S + k^T (weighted v)
-        const float et = exp2f(total);
+        const float et = exp2_fast(total);
 #pragma unroll
         for (int i = 0; i < NTW; ++i) {
             const int n0 = 16 * (i * 8 + warp);
