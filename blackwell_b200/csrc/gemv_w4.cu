@@ -21,6 +21,7 @@ void set_attn_mma(int v);  // attention_decode.cu
 cudaError_t attn_reserve_scratch(size_t bytes);
 size_t attn_scratch_bytes(int M, int nqh, int nkv, int ctx);
 namespace peer { void set_two_step_min_kb(int kb); void set_wait_limit_ms(int ms); }  // peer_allreduce.cu
+namespace lm { void set_linear_stream_max(int rows); }  // linear_bf16.cu
 
 namespace tc {  // tensor-core path, gemm_w4a8_tc.cu
 bool eligible(const GemvArgs& a, int M);
@@ -709,6 +710,7 @@ extern "C" int bw_set_tuning(int key, int value) {
         case 20: g_tune_prep_min = value; return 0;
         case 21: g_tune_prep_min_swiglu = value; return 0;
         case 22: set_attn_slots_pct(value); return 0;
+        case 23: lm::set_linear_stream_max(value); return 0;
         default: return cudaErrorInvalidValue;
     }
 }

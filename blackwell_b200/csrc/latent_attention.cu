@@ -55,7 +55,7 @@ cudaError_t decode(const LatentArgs& a, const Rows& r, int nbuf, cudaStream_t st
     cudaError_t e = allow_smem(latent_decode_kernel<NT>, once);
     if (e != cudaSuccess) return e;
     count_launch(1);
-    return launch_pdl(latent_decode_kernel<NT>, dim3(a.splits, (a.heads + 15) / 16, r.T), dim3(256), DecodeSmem(a.R, a.rot, nbuf).total,
+    return launch_pdl(latent_decode_kernel<NT>, dim3(a.splits, (a.heads + 15) / 16, r.T), dim3(kDecThreads), DecodeSmem(a.R, a.rot, nbuf).total,
                       st, a, r, nbuf);
 }
 
@@ -95,10 +95,9 @@ cudaError_t latent_absorbed(const LatentArgs& a, const Rows& r, int f32, cudaStr
     const int keys = by_scalar ? kScalarKeys : kDecKeys;
     if (f32) e = scalar<float>(a, r, st);
     else if (by_scalar) e = scalar<bf16>(a, r, st);
-    else if (a.R <= 128) e = decode<2>(a, r, nbuf, st);
-    else if (a.R <= 256) e = decode<4>(a, r, nbuf, st);
-    else if (a.R <= 512) e = decode<8>(a, r, nbuf, st);
-    else e = decode<16>(a, r, nbuf, st);
+    else if (a.R <= 256) e = decode<2>(a, r, nbuf, st);
+    else if (a.R <= 512) e = decode<4>(a, r, nbuf, st);
+    else e = decode<8>(a, r, nbuf, st);
     if (e != cudaSuccess) return e;
     return f32 ? out<float, 1>(a, r, keys, st) : rb4 ? out<bf16, 4>(a, r, keys, st) : out<bf16, 1>(a, r, keys, st);
 }

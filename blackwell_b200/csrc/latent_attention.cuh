@@ -237,6 +237,7 @@ __global__ void __launch_bounds__(256) latent_scalar_kernel(const LatentArgs a, 
 }
 
 constexpr int kDecKeys = 64;
+constexpr int kDecThreads = 512;
 constexpr int kDecP = kDecKeys * 2 + 16;   // bytes of a row of softmax weights
 constexpr int kDecS = kDecKeys + 4;        // floats of a row of partial scores
 struct DecodeSmem {
@@ -253,11 +254,11 @@ struct DecodeSmem {
     }
 };
 
-// Block (split, 16 heads, row); 8 warps.  Scores: a warp takes every eighth 16-wide step of the query / key dimension for
-// all 64 keys of a tile, and the partial scores meet in shared memory, where 16 neighbouring threads own one head's row
-// (softmax without further exchange).  Output: a warp accumulates latent columns [w * NT * 8, (w + 1) * NT * 8).
+// Block (split, 16 heads, row); 16 warps.  Scores: a warp takes every eighth 16-wide step of the query / key dimension for
+// half of the 64 keys of a tile, and the partial scores meet in shared memory, where one warp owns one head's row (softmax
+// without further exchange).  Output: a warp accumulates latent columns [w * NT * 8, (w + 1) * NT * 8).
 template <int NT>
-__global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, const Rows r, int nbuf) {
+__global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const LatentArgs a, const Rows r, int nbuf) {
     extern __shared__ __align__(16) unsigned char smem[];
     const DecodeSmem L(a.R, a.rot, nbuf);
     const int Dp = latent_dp(a.R, a.rot), R8 = pad8(a.R), D8 = R8 + pad8(a.rot);
@@ -274,7 +275,7 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
     if (slot < 0 || t0 >= t1) return;   // the merge reads the splits that hold positions
     const bf16* cache = static_cast<const bf16*>(a.cache) + (long)slot * a.max_seq * a.ldc;
     const int nc = Dp / 8;
-    const RowWalk walk(t, 256, nc);
+    const RowWalk walk(t, kDecThreads, nc);
     auto issue = [&](int tile, int buf) {
         const uint32_t dst = sb + L.k_off + buf * L.kbuf;
         for (RowWalk w = walk; w.row < kDecKeys; w.next()) {
@@ -292,7 +293,8 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
     }
     issue(t0, 0);
     float O[NT][4] = {};
-    const int srow = t >> 4, skey = (t & 15) * 4;     // this thread's head row and keys in the softmax
+    const int skey = lane * 2;                        // this thread's keys in the softmax of head row `warp`
+    const int kslice = (warp & 7) * 16, khalf = (warp >> 3) * 32;
     float m = -INFINITY, l = 0.f;
     for (int tile = t0; tile < t1; ++tile) {
         const int buf = nbuf == 2 ? (tile - t0) & 1 : 0;
@@ -300,59 +302,55 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
         cp_async_wait<0>();
         __syncthreads();
         if (nbuf == 2 && tile + 1 < t1) issue(tile + 1, buf ^ 1);
-        float s[8][4] = {};
-        for (int k0 = warp * 16; k0 < Dp; k0 += 128) {
+        float s[4][4] = {};
+        for (int k0 = kslice; k0 < Dp; k0 += 128) {
             uint32_t ah[4], al[4];
             const uint32_t qa = sb + L.q_off + (lane & 15) * L.row + (k0 + (lane >> 4) * 8) * 2;
             ldsm4(qa, ah);
             ldsm4(qa + 16 * L.row, al);
-            const uint32_t ka = kb + ((lane & 7) + (lane >> 4) * 8) * L.row + (k0 + ((lane >> 3) & 1) * 8) * 2;
-            uint32_t b[4][4];
+            const uint32_t ka = kb + (khalf + (lane & 7) + (lane >> 4) * 8) * L.row + (k0 + ((lane >> 3) & 1) * 8) * 2;
+            uint32_t b[2][4];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) ldsm4(ka + 16 * j * L.row, b[j]);
+            for (int j = 0; j < 2; ++j) ldsm4(ka + 16 * j * L.row, b[j]);
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
+            for (int j = 0; j < 2; ++j) {
                 mma_bf16(s[2 * j], ah[0], ah[1], ah[2], ah[3], b[j][0], b[j][1]);
                 mma_bf16(s[2 * j + 1], ah[0], ah[1], ah[2], ah[3], b[j][2], b[j][3]);
             }
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
+            for (int j = 0; j < 2; ++j) {
                 mma_bf16(s[2 * j], al[0], al[1], al[2], al[3], b[j][0], b[j][1]);
                 mma_bf16(s[2 * j + 1], al[0], al[1], al[2], al[3], b[j][2], b[j][3]);
             }
         }
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            float* p = part + (warp * 16 + g) * kDecS + 8 * j + 2 * q4;
+        for (int j = 0; j < 4; ++j) {
+            float* p = part + ((warp & 7) * 16 + g) * kDecS + khalf + 8 * j + 2 * q4;
             *reinterpret_cast<float2*>(p) = make_float2(s[j][0], s[j][1]);
             *reinterpret_cast<float2*>(p + 8 * kDecS) = make_float2(s[j][2], s[j][3]);
         }
         __syncthreads();
-        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        float2 x = make_float2(0.f, 0.f);
 #pragma unroll
         for (int w = 0; w < 8; ++w) {
-            const float4 y = *reinterpret_cast<const float4*>(part + (w * 16 + srow) * kDecS + skey);
-            x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
+            const float2 y = *reinterpret_cast<const float2*>(part + (w * 16 + warp) * kDecS + skey);
+            x.x += y.x;
+            x.y += y.y;
         }
         const int key = tile * kDecKeys + skey;
         x.x = key < len ? x.x * a.scale : -INFINITY;
         x.y = key + 1 < len ? x.y * a.scale : -INFINITY;
-        x.z = key + 2 < len ? x.z * a.scale : -INFINITY;
-        x.w = key + 3 < len ? x.w * a.scale : -INFINITY;
-        float mx = fmaxf(fmaxf(x.x, x.y), fmaxf(x.z, x.w));
-#pragma unroll
-        for (int o = 1; o < 16; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-        mx = fmaxf(mx, m);                           // finite: the first key of a tile is always visible
+        const float mx = fmaxf(warp_max(fmaxf(x.x, x.y)), m);   // finite: the first key of a tile is always visible
         const float alpha = expf(m - mx);
         m = mx;
-        x.x = expf(x.x - mx); x.y = expf(x.y - mx); x.z = expf(x.z - mx); x.w = expf(x.w - mx);
-        l = l * alpha + ((x.x + x.y) + (x.z + x.w));
-        uint2 hi, lo;
-        split_bf16(x.x, x.y, hi.x, lo.x);
-        split_bf16(x.z, x.w, hi.y, lo.y);
-        *reinterpret_cast<uint2*>(smem + L.p_off + srow * kDecP + skey * 2) = hi;
-        *reinterpret_cast<uint2*>(smem + L.p_off + (16 + srow) * kDecP + skey * 2) = lo;
-        if ((t & 15) == 0) alphas[srow] = alpha;
+        x.x = expf(x.x - mx);
+        x.y = expf(x.y - mx);
+        l = l * alpha + (x.x + x.y);
+        uint32_t hi, lo;
+        split_bf16(x.x, x.y, hi, lo);
+        *reinterpret_cast<uint32_t*>(smem + L.p_off + warp * kDecP + skey * 2) = hi;
+        *reinterpret_cast<uint32_t*>(smem + L.p_off + (16 + warp) * kDecP + skey * 2) = lo;
+        if (lane == 0) alphas[warp] = alpha;
         __syncthreads();
         const float al0 = alphas[g], al1 = alphas[g + 8];
 #pragma unroll
@@ -392,10 +390,9 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
             if (col < R8) *reinterpret_cast<float2*>(out + col) = make_float2(O[j][2 * p], O[j][2 * p + 1]);
         }
     }
-#pragma unroll
-    for (int o = 1; o < 16; o <<= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-    if ((t & 15) == 0 && h0 + srow < a.heads) {
-        float* stats = part_ptr(a, row, h0 + srow, split) + R8;
+    l = warp_sum(l);
+    if (lane == 0 && h0 + warp < a.heads) {
+        float* stats = part_ptr(a, row, h0 + warp, split) + R8;
         stats[0] = m;
         stats[1] = l;
     }

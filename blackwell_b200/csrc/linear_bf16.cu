@@ -50,17 +50,16 @@ int stream_xs_stride(int ldw) {
     const int nkb = (ldw + 31) / 32;
     return nkb * 64 + (nkb % 2 == 0 ? 64 : 0);   // odd multiple of 64 bytes: conflict-free fragment reads
 }
-int stream_smem(int T, int NT, int ldw) { return kStreamWarps * NT * 8 * 16 * 4 + T * stream_xs_stride(ldw); }
+int stream_smem(int T, int ldw) { return kStreamWarps * 8 * 16 * 4 + T * stream_xs_stride(ldw); }
 
-template <int NT>
 cudaError_t launch_stream(const LinearArgs& a, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
-    cudaError_t e = allow_smem(linear_stream_kernel<NT>, once, kMaxDynSmem);
+    cudaError_t e = allow_smem(linear_stream_kernel, once, kMaxDynSmem);
     if (e != cudaSuccess) return e;
-    const int smem = stream_smem(a.T, NT, (int)a.ldw), tiles = (a.N + 15) / 16;
+    const int smem = stream_smem(a.T, (int)a.ldw), tiles = (a.N + 15) / 16;
     const int per_sm = smem > 110 * 1024 ? 1 : smem > 72 * 1024 ? 2 : 3;
     const int grid = std::min(tiles, sm_count(current_device()) * per_sm);
-    e = launch_pdl(linear_stream_kernel<NT>, dim3(grid), dim3(kStreamWarps * 32), smem, st, a, stream_xs_stride((int)a.ldw));
+    e = launch_pdl(linear_stream_kernel, dim3(grid), dim3(kStreamWarps * 32), smem, st, a, stream_xs_stride((int)a.ldw));
     count_launch(1);
     return e;
 }
@@ -97,11 +96,11 @@ cudaError_t launch_tc(const LinearArgs& a, int ksplit, cudaStream_t st) {
     return e;
 }
 
-std::atomic<int> g_stream_max{32};
+std::atomic<int> g_stream_max{-1};   // rows up to which the streaming kernel is used; -1: automatic
 
 }  // namespace
 
-void set_linear_stream_max(int rows) { g_stream_max = rows > 0 ? std::min(rows, 32) : 32; }
+void set_linear_stream_max(int rows) { g_stream_max = rows > 0 ? rows - 1 : -1; }
 
 cudaError_t linear(const LinearArgs& a, cudaStream_t st) {
     if (a.T < 1 || a.N < 1 || a.K < 1 || a.ldw % 8 != 0 || a.ldw < a.K || (reinterpret_cast<uintptr_t>(a.W) & 15) ||
@@ -114,23 +113,30 @@ cudaError_t linear(const LinearArgs& a, cudaStream_t st) {
         return e;
     }
     if (a.ldx % 8 != 0) return cudaErrorInvalidValue;
-    const int nt = a.T <= 8 ? 1 : a.T <= 16 ? 2 : 4;
-    if (a.T <= g_stream_max && stream_smem(a.T, nt, (int)a.ldw) <= kMaxDynSmem)
-        return nt == 1 ? launch_stream<1>(a, st) : nt == 2 ? launch_stream<2>(a, st) : launch_stream<4>(a, st);
+    // measured borders: the streaming kernel wins on small matrices and few rows (its launch has less to set up)
+    const long size = (long)a.N * a.K;
+    const int limit = g_stream_max.load();
+    const bool stream = limit >= 0 ? a.T <= limit : a.K <= 4096 && ((a.T <= 2 && size <= 25000000) || (a.K <= 2048 && size <= 8000000));
+    if (stream && a.T <= 8 && stream_smem(a.T, (int)a.ldw) <= kMaxDynSmem) return launch_stream(a, st);
     // enough tiles for the SMs: persistent tiles of 256 / 128 rows; otherwise the K range is split over a cluster
     const int sms = sm_count(current_device()), rtiles = (a.N + kTcRows - 1) / kTcRows, nk = (a.K + kTcK - 1) / kTcK;
     auto tiles = [&](int nt_) { return rtiles * ((a.T + nt_ - 1) / nt_); };
     if (a.T > 64) {
         if (tiles(256) >= sms) return launch_tc<256, false>(a, 1, st);
-        if (a.T > 128 || tiles(128) >= sms / 2) {
+        if (a.T > 512 || tiles(128) >= sms / 2) {
             // fewer, larger tiles only when they fill the machine as well as the small ones do
             const long w128 = (long)((tiles(128) + sms - 1) / sms), w64 = (long)((tiles(64) + sms - 1) / sms);
             return 2 * w64 < 2 * w128 + 1 && w64 * 64 < w128 * 128 ? launch_tc<64, false>(a, 1, st) : launch_tc<128, false>(a, 1, st);
         }
     }
     const int ntile = a.T <= 16 ? 16 : a.T <= 32 ? 32 : 64;
+    // K split that finishes first: waves of CTAs (two per SM), each its share of the K blocks plus a constant
     int ks = 1;
-    while (ks < 8 && 2 * ks <= nk && tiles(ntile) * 2 * ks <= sms + sms / 4) ks *= 2;
+    long best = 0;
+    for (int k = 1; k <= 8 && k <= nk; k *= 2) {
+        const long cost = (long)((tiles(ntile) * k + 2 * sms - 1) / (2 * sms)) * ((nk + k - 1) / k + 8);
+        if (k == 1 || cost < best) { best = cost; ks = k; }
+    }
     return ntile == 16 ? launch_tc<16, true>(a, ks, st) : ntile == 32 ? launch_tc<32, true>(a, ks, st) : launch_tc<64, true>(a, ks, st);
 }
 

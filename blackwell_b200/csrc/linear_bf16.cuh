@@ -1,13 +1,14 @@
 // y = W x for bfloat16 weights.  Three kernels:
-//   linear_stream_kernel  up to 32 rows (decode steps): weights go straight from HBM to registers as the A operand of
+//   linear_stream_kernel  few rows of a small matrix: weights go straight from HBM to registers as the A operand of
 //                         mma.sync -- the order of k inside a 32-wide block is permuted identically for both operands,
 //                         which a dot product does not see, so that a thread's fragment is one 16-byte load -- and the
-//                         activations sit in shared memory as the B operand.  The first weights are in flight before
-//                         the kernel waits for its predecessor.
-//   linear_tc_kernel      more rows (prompts): tcgen05.mma kind::f16, weights as the 128-row operand, up to 256 rows of
-//                         activations as the other, both through 128-byte-swizzled TMA; accumulators double-buffered in
-//                         tensor memory.  With few tiles the K range is split over a cluster and the partial sums
-//                         are added through distributed shared memory in a fixed order.
+//                         activations sit in shared memory as the B operand.
+//   linear_tc_kernel      tcgen05.mma kind::f16, weights as the 128-row operand, up to 256 rows of activations as the
+//                         other, both through 128-byte-swizzled TMA.  Prompts: persistent CTAs, accumulators
+//                         double-buffered in tensor memory.  Decode steps and short portions: the K range is split over a
+//                         cluster of up to eight CTAs, two of which share an SM, and the partial sums are added through
+//                         distributed shared memory in a fixed order.
+//                         Both have their first weights in flight before they wait for the preceding kernel.
 //   linear_f32_kernel     32-bit mode: fp32 activations, fp32 FMAs (the weights are bfloat16 values, exact in fp32).
 #pragma once
 #include <cuda.h>
@@ -32,15 +33,14 @@ __device__ __forceinline__ void store_out(const LinearArgs& a, int t, int n, flo
     }
 }
 
-// ---------------------------------------------------------------------------------------------- up to 32 rows
+// ---------------------------------------------------------------------------------------------- up to 8 rows
 constexpr int kStreamWarps = 8;
 constexpr int kStreamU = 4;   // 32-wide k blocks per warp and load batch
 
-template <int NT>  // 8-row tiles of the activations
 __global__ void __launch_bounds__(kStreamWarps * 32) linear_stream_kernel(const LinearArgs a, int xs_stride) {
     extern __shared__ __align__(16) unsigned char smem[];
-    float* red = reinterpret_cast<float*>(smem);                         // [warps][NT * 8][16]
-    unsigned char* xs = smem + kStreamWarps * NT * 8 * 16 * 4;           // [T][xs_stride] bytes
+    float* red = reinterpret_cast<float*>(smem);                         // [warps][8][16]
+    unsigned char* xs = smem + kStreamWarps * 8 * 16 * 4;                // [T][xs_stride] bytes
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, q = lane & 3;
     const int tiles = (a.N + 15) / 16, kw = (int)a.ldw;
     const int nkb = (kw + 31) / 32;
@@ -82,11 +82,7 @@ __global__ void __launch_bounds__(kStreamWarps * 32) linear_stream_kernel(const 
     }
     __syncthreads();
 
-    float acc[NT][4];
-#pragma unroll
-    for (int j = 0; j < NT; ++j)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
+    float acc[4] = {};
     int it = 0;
     while (tile < tiles) {
         int ntile = tile, nit = it + 1;
@@ -96,34 +92,28 @@ __global__ void __launch_bounds__(kStreamWarps * 32) linear_stream_kernel(const 
         for (int u = 0; u < kStreamU; ++u) {
             const int kb = (it * kStreamU + u) * kStreamWarps + warp;
             if (kb < nkb) {
-#pragma unroll
-                for (int j = 0; j < NT; ++j) {
-                    uint4 b = zero4;
-                    if (j * 8 + g < a.T) b = *reinterpret_cast<const uint4*>(xs + (j * 8 + g) * xs_stride + (kb * 32 + q * 8) * 2);
-                    mma_bf16(acc[j], cur[u][0].x, cur[u][1].x, cur[u][0].y, cur[u][1].y, b.x, b.y);
-                    mma_bf16(acc[j], cur[u][0].z, cur[u][1].z, cur[u][0].w, cur[u][1].w, b.z, b.w);
-                }
+                uint4 b = zero4;
+                if (g < a.T) b = *reinterpret_cast<const uint4*>(xs + g * xs_stride + (kb * 32 + q * 8) * 2);
+                mma_bf16(acc, cur[u][0].x, cur[u][1].x, cur[u][0].y, cur[u][1].y, b.x, b.y);
+                mma_bf16(acc, cur[u][0].z, cur[u][1].z, cur[u][0].w, cur[u][1].w, b.z, b.w);
             }
         }
         if (nit == 0) {   // tile finished: add the warps' K shares
+            float* p = red + warp * 8 * 16;
+            p[(2 * q) * 16 + g] = acc[0];
+            p[(2 * q + 1) * 16 + g] = acc[1];
+            p[(2 * q) * 16 + g + 8] = acc[2];
+            p[(2 * q + 1) * 16 + g + 8] = acc[3];
 #pragma unroll
-            for (int j = 0; j < NT; ++j) {
-                float* p = red + ((long)warp * NT * 8 + j * 8) * 16;
-                p[(2 * q) * 16 + g] = acc[j][0];
-                p[(2 * q + 1) * 16 + g] = acc[j][1];
-                p[(2 * q) * 16 + g + 8] = acc[j][2];
-                p[(2 * q + 1) * 16 + g + 8] = acc[j][3];
-#pragma unroll
-                for (int i = 0; i < 4; ++i) acc[j][i] = 0.f;
-            }
+            for (int i = 0; i < 4; ++i) acc[i] = 0.f;
             __syncthreads();
             if (a.epi == kEpiSwiglu) {
-                for (int i = t; i < NT * 8 * 8; i += kStreamWarps * 32) {
-                    const int m = i >> 3, j = i & 7, n = tile * 16 + 2 * j;
+                if (t < 8 * 8) {
+                    const int m = t >> 3, j = t & 7, n = tile * 16 + 2 * j;
                     float gt = 0.f, up = 0.f;
 #pragma unroll
                     for (int w = 0; w < kStreamWarps; ++w) {
-                        const float2 s = *reinterpret_cast<const float2*>(red + ((long)w * NT * 8 + m) * 16 + 2 * j);
+                        const float2 s = *reinterpret_cast<const float2*>(red + (w * 8 + m) * 16 + 2 * j);
                         gt += s.x;
                         up += s.y;
                     }
@@ -131,11 +121,11 @@ __global__ void __launch_bounds__(kStreamWarps * 32) linear_stream_kernel(const 
                         static_cast<bf16*>(a.y)[(long)m * a.ldy + (n >> 1)] = __float2bfloat16_rn(silu_f(gt) * up);
                 }
             } else {
-                for (int i = t; i < NT * 8 * 16; i += kStreamWarps * 32) {
-                    const int m = i >> 4, n = tile * 16 + (i & 15);
+                if (t < 8 * 16) {
+                    const int m = t >> 4, n = tile * 16 + (t & 15);
                     float s = 0.f;
 #pragma unroll
-                    for (int w = 0; w < kStreamWarps; ++w) s += red[((long)w * NT * 8 + m) * 16 + (i & 15)];
+                    for (int w = 0; w < kStreamWarps; ++w) s += red[(w * 8 + m) * 16 + (t & 15)];
                     if (m < a.T && n < a.N) store_out<false>(a, m, n, s);
                 }
             }
@@ -197,11 +187,10 @@ constexpr int kTcK = 64;          // k per stage: one 128-byte swizzle atom of b
 constexpr int kTcThreads = 384;   // warp 0 copies, warp 1 MMAs, warps 4-11 epilogue (two per TMEM lane quarter)
 
 __host__ __device__ constexpr int tc_stage_bytes(int NT) { return kTcRows * 128 + NT * 128; }
-__host__ __device__ constexpr int tc_stages(int NT) { return NT >= 256 ? 4 : NT >= 128 ? 6 : 8; }
-// one CTA's accumulator tile for the cluster reduction, [NT][128] fp32
-__host__ __device__ constexpr int tc_smem_bytes(int NT, bool split) {
-    return 1024 + 1024 + tc_stages(NT) * tc_stage_bytes(NT) + (split ? NT * kTcRows * 4 : 0);
-}
+// split form: two CTAs share an SM; its accumulator tile for the cluster reduction, [NT][128] fp32, takes the place of the
+// operand ring once the products are done
+__host__ __device__ constexpr int tc_stages(int NT, bool split) { return split ? (NT >= 64 ? 4 : 5) : NT >= 256 ? 4 : NT >= 128 ? 6 : 8; }
+__host__ __device__ constexpr int tc_smem_bytes(int NT, bool split) { return 1024 + 1024 + tc_stages(NT, split) * tc_stage_bytes(NT); }
 
 // Shared-memory matrix descriptor: K-major rows of 128 bytes in the 128-byte swizzle, 8-row groups 1024 bytes apart.
 __device__ __forceinline__ uint64_t desc_sw128(uint32_t addr) {
@@ -231,10 +220,10 @@ __device__ __forceinline__ void cluster_sync_all() {
 
 // SPLIT: one tile per cluster of `ksplit` CTAs; otherwise persistent CTAs walk the tiles (row tile fastest).
 template <int NT, bool SPLIT>
-__global__ void __launch_bounds__(kTcThreads, 1)
+__global__ void __launch_bounds__(kTcThreads, SPLIT ? 2 : 1)
 linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, const LinearArgs a,
                  int ksplit, int* status) {
-    constexpr int S = tc_stages(NT), BYTES = tc_stage_bytes(NT), NACC = SPLIT ? 1 : 2;
+    constexpr int S = tc_stages(NT, SPLIT), BYTES = tc_stage_bytes(NT), NACC = SPLIT ? 1 : 2;
     constexpr int COLS = SPLIT ? (NT < 32 ? 32 : NT) : 2 * NT;
     extern __shared__ unsigned char smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -242,7 +231,8 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
     volatile uint32_t* tmem_ptr = reinterpret_cast<volatile uint32_t*>(smem + 512);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + 520);
     unsigned char* stage0 = smem + 1024;
-    float* part = reinterpret_cast<float*>(stage0 + S * BYTES);
+    float* part = reinterpret_cast<float*>(stage0);
+    static_assert(!SPLIT || NT * kTcRows * 4 <= S * BYTES, "accumulator tile");
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
     auto full = [&](int i) { return smem_u32(&bars[i]); };
     auto empty = [&](int i) { return smem_u32(&bars[S + i]); };

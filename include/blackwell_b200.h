@@ -397,7 +397,7 @@ int bw_decode_watch_layers(bw_decode* d, float* buffer, long rows);
 /* y[t][n] = sum_k x[t][k] W[n][k] with bfloat16 W [N][ldw] (ldw a multiple of 8, zero beyond K): the product of the
  * layered models.  x bfloat16 [T][ldx] (ldx a multiple of 8), or fp32 when x_f32 (32-bit FMAs); y bfloat16 or, with y_f32
  * (or x_f32), fp32.  epilogue 0: none; 1: rows 2j / 2j+1 of W are gate / up, y[t][j] = silu(gate) * up, N / 2 columns in
- * x's format; 2: softcap * tanh(y / softcap).  Up to 32 rows a weight-streaming kernel, beyond that tcgen05. */
+ * x's format; 2: softcap * tanh(y / softcap).  Few rows of a small matrix take a weight-streaming kernel, everything else tcgen05. */
 int bw_linear_bf16(void* y, long ldy, const void* x, long ldx, const uint16_t* W, long ldw, int T, int N, int K,
                    int y_f32, int x_f32, int epilogue, float softcap, void* stream);
 
@@ -507,7 +507,9 @@ int bw_reserve_scratch(size_t gemv_bytes, size_t attention_bytes);
  * activation-scale copies, 64 no weight-scale loads: results are then meaningless), key 20 = smallest batch whose
  * float activations are quantized once by a separate kernel before a streaming GEMV (0 = default 2), key 21 = the
  * same for the SwiGLU prologue (0 = default 1), key 22 = decode attention: the earlier split rule with pct % of the SMs
- * as CTA slots (0 = default rule: one wave of two CTAs per SM, at least 224 positions per split). */
+ * as CTA slots (0 = default rule: one wave of two CTAs per SM, at least 224 positions per split),
+ * key 23 = bfloat16 linear: up to value - 1 rows (8 at most) take the weight-streaming kernel, more the tcgen05 kernel (0 =
+ * automatic). */
 int bw_set_tuning(int key, int value);
 /* Number of kernels launched by this library since the last call with reset != 0. */
 long long bw_launch_count(int reset);

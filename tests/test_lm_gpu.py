@@ -61,9 +61,22 @@ def _linear(x, W, T, N, K, x_f32, epilogue=0, cap=0.0, y_f32=1):
     return y[:, :cols]
 
 
+@pytest.mark.parametrize("stream_rows", [0, 8])
 @pytest.mark.parametrize("T", [1, 2, 7, 8, 9, 16, 20, 32, 33, 64, 65, 129, 300])
 @pytest.mark.parametrize("N, K", [(130, 40), (77, 200), (515, 328), (16, 1032)])
-def test_linear_shapes(cuda, T, N, K):
+def test_linear_shapes(cuda, T, N, K, stream_rows):
+    from blackwell_b200 import kernels
+
+    if stream_rows and T > 8:
+        pytest.skip("more than eight rows always take the tcgen05 kernel")
+    kernels.set_tuning(23, stream_rows + 1)
+    try:
+        check_linear_shapes(T, N, K)
+    finally:
+        kernels.set_tuning(23, 0)
+
+
+def check_linear_shapes(T, N, K):
     rng = np.random.default_rng(T * 1000 + N)
     _, W = lm.to_bf16(rng.standard_normal((N, K)))
     _, x = lm.to_bf16(rng.standard_normal((T, K)))
