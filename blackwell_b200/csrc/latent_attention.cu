@@ -32,14 +32,14 @@ cudaError_t prep(const LatentArgs& a, const Rows& r, cudaStream_t st) {
 }
 
 template <typename A, int RB>
-cudaError_t out(const LatentArgs& a, const Rows& r, int keys, cudaStream_t st) {
+cudaError_t out(const LatentArgs& a, const Rows& r, int keys, int groups, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
     cudaError_t e = allow_smem(latent_out_kernel<A, RB>, once);
     if (e != cudaSuccess) return e;
-    const size_t smem = (size_t)(3 * RB * pad8(a.R) + ((RB * a.splits + 3) & ~3)) * 4;
+    const size_t smem = (size_t)(3 * RB * pad8(a.R) + ((RB * groups * a.splits + 3) & ~3)) * 4;
     if (smem > kMaxDynSmem) return cudaErrorInvalidValue;
     count_launch(1);
-    return launch_pdl(latent_out_kernel<A, RB>, dim3(a.heads * ((pad8(a.V) + kOutV - 1) / kOutV), (r.T + RB - 1) / RB), dim3(256), smem, st, a, r, keys);
+    return launch_pdl(latent_out_kernel<A, RB>, dim3(a.heads * ((pad8(a.V) + kOutV - 1) / kOutV), (r.T + RB - 1) / RB), dim3(256), smem, st, a, r, keys, groups);
 }
 
 template <typename A>
@@ -50,13 +50,13 @@ cudaError_t scalar(const LatentArgs& a, const Rows& r, cudaStream_t st) {
 }
 
 template <int NT>
-cudaError_t decode(const LatentArgs& a, const Rows& r, int nbuf, cudaStream_t st) {
+cudaError_t decode(const LatentArgs& a, const Rows& r, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
     cudaError_t e = allow_smem(latent_decode_kernel<NT>, once);
     if (e != cudaSuccess) return e;
     count_launch(1);
-    return launch_pdl(latent_decode_kernel<NT>, dim3(a.splits, (a.heads + 15) / 16, r.T), dim3(kDecThreads), DecodeSmem(a.R, a.rot, nbuf).total,
-                      st, a, r, nbuf);
+    return launch_pdl(latent_decode_kernel<NT>, dim3(a.splits, (a.heads + 15) / 16, r.T), dim3(kDecThreads), DecodeSmem(a.R, a.rot).total,
+                      st, a, r);
 }
 
 template <int VT, int MT>
@@ -90,16 +90,15 @@ cudaError_t latent_absorbed(const LatentArgs& a, const Rows& r, int f32, cudaStr
     const bool rb4 = r.T >= 8 && !f32 && a.R <= 1024 && (pad8(a.dim) + pad8(a.rot)) <= 1024;
     cudaError_t e = f32 ? prep<float, 1, 64>(a, r, st) : rb4 ? prep<bf16, 4, 256>(a, r, st) : prep<bf16, 1, 64>(a, r, st);
     if (e != cudaSuccess) return e;
-    const int nbuf = DecodeSmem(a.R, a.rot, 2).total <= kMaxDynSmem ? 2 : 1;
-    const bool by_scalar = f32 || a.R > 1024 || DecodeSmem(a.R, a.rot, nbuf).total > kMaxDynSmem;
-    const int keys = by_scalar ? kScalarKeys : kDecKeys;
+    const bool by_scalar = f32 || a.R > 512 || latent_dp(a.R, a.rot) > kDecSteps * 128 || DecodeSmem(a.R, a.rot).total > kMaxDynSmem;
     if (f32) e = scalar<float>(a, r, st);
     else if (by_scalar) e = scalar<bf16>(a, r, st);
-    else if (a.R <= 256) e = decode<2>(a, r, nbuf, st);
-    else if (a.R <= 512) e = decode<4>(a, r, nbuf, st);
-    else e = decode<8>(a, r, nbuf, st);
+    else if (a.R <= 128) e = decode<2>(a, r, st);
+    else if (a.R <= 256) e = decode<4>(a, r, st);
+    else e = decode<8>(a, r, st);
     if (e != cudaSuccess) return e;
-    return f32 ? out<float, 1>(a, r, keys, st) : rb4 ? out<bf16, 4>(a, r, keys, st) : out<bf16, 1>(a, r, keys, st);
+    const int keys = by_scalar ? kScalarKeys : kDecKeys, groups = by_scalar ? 1 : 2;
+    return f32 ? out<float, 1>(a, r, keys, groups, st) : rb4 ? out<bf16, 4>(a, r, keys, groups, st) : out<bf16, 1>(a, r, keys, groups, st);
 }
 
 cudaError_t latent_expanded(const LatentArgs& a, const Rows& r, cudaStream_t st) {

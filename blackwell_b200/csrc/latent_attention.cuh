@@ -167,9 +167,10 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentA
         }
 }
 
-// One partial result per (row, head, split): pad8(R) un-normalised outputs, then the running maximum and the sum.
-__device__ __forceinline__ float* part_ptr(const LatentArgs& a, int row, int h, int split) {
-    return a.part + (((long)row * a.heads + h) * a.splits + split) * (pad8(a.R) + kPartStats);
+// Partial results of a (row, head): two per split (the scalar kernel uses the first `splits` of them), each pad8(R)
+// un-normalised outputs, then the running maximum and the sum.
+__device__ __forceinline__ float* part_ptr(const LatentArgs& a, int row, int h, int i) {
+    return a.part + (((long)row * a.heads + h) * 2 * a.splits + i) * (pad8(a.R) + kPartStats);
 }
 // Splits of a context of `len` positions that hold any (tiles of `keys` are dealt out in runs of equal length).
 __device__ __forceinline__ int used_splits(int len, int keys, int splits) {
@@ -236,34 +237,41 @@ __global__ void __launch_bounds__(256) latent_scalar_kernel(const LatentArgs a, 
     if (t == 0) { stats[0] = m; stats[1] = l; }
 }
 
-constexpr int kDecKeys = 64;
-constexpr int kDecThreads = 512;
+constexpr int kDecKeys = 32;               // keys per tile of a warp group
+constexpr int kDecThreads = 512;           // two groups of eight warps
+constexpr int kDecSteps = 5;               // 16-wide query steps a warp holds: padded query size up to 640
 constexpr int kDecP = kDecKeys * 2 + 16;   // bytes of a row of softmax weights
 constexpr int kDecS = kDecKeys + 4;        // floats of a row of partial scores
-struct DecodeSmem {
-    int row, q_off, k_off, kbuf, p_off, s_off, f_off, total;
-    __host__ __device__ DecodeSmem(int R, int rot, int nbuf) {
+struct DecodeSmem {                        // per group: two key tiles, softmax weights, partial scores, rescale factors
+    int row, kbuf, p_off, s_off, f_off, group, total;
+    __host__ __device__ DecodeSmem(int R, int rot) {
         row = latent_dp(R, rot) * 2 + 16;
-        q_off = 0;
-        k_off = 2 * 16 * row;
         kbuf = kDecKeys * row;
-        p_off = k_off + nbuf * kbuf;
+        p_off = 2 * kbuf;
         s_off = p_off + 2 * 16 * kDecP;
         f_off = s_off + 8 * 16 * kDecS * 4;
-        total = f_off + 16 * 4;
+        group = f_off + 16 * 4;
+        total = 2 * group;
     }
 };
+__device__ __forceinline__ void group_sync(int group) {
+    if (group) asm volatile("bar.sync 2, 256;" ::: "memory");
+    else asm volatile("bar.sync 1, 256;" ::: "memory");
+}
 
-// Block (split, 16 heads, row); 16 warps.  Scores: a warp takes every eighth 16-wide step of the query / key dimension for
-// half of the 64 keys of a tile, and the partial scores meet in shared memory, where one warp owns one head's row (softmax
-// without further exchange).  Output: a warp accumulates latent columns [w * NT * 8, (w + 1) * NT * 8).
+// Block (split, 16 heads, row): the tiles of the split alternate between two warp groups that run independently, so that
+// one group's products overlap the other's softmax; each leaves its own partial result.  Inside a group a warp holds every
+// eighth 16-wide step of the queries in registers and multiplies it with all keys of the tile; the partial scores meet
+// in shared memory, where 16 neighbouring threads own one head's row.  Output: a warp accumulates latent columns
+// [w * NT * 8, (w + 1) * NT * 8).
 template <int NT>
-__global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const LatentArgs a, const Rows r, int nbuf) {
-    extern __shared__ __align__(16) unsigned char smem[];
-    const DecodeSmem L(a.R, a.rot, nbuf);
+__global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const LatentArgs a, const Rows r) {
+    extern __shared__ __align__(16) unsigned char smem_all[];
+    const DecodeSmem L(a.R, a.rot);
     const int Dp = latent_dp(a.R, a.rot), R8 = pad8(a.R), D8 = R8 + pad8(a.rot);
-    const int t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, q4 = lane & 3;
+    const int group = threadIdx.x >> 8, t = threadIdx.x & 255, warp = t >> 5, lane = t & 31, g = lane >> 2, q4 = lane & 3;
     const int split = blockIdx.x, h0 = blockIdx.y * 16, row = blockIdx.z;
+    unsigned char* smem = smem_all + group * L.group;
     const uint32_t sb = smem_u32(smem);
     float* part = reinterpret_cast<float*>(smem + L.s_off);    // [8][16][kDecS]
     float* alphas = reinterpret_cast<float*>(smem + L.f_off);  // [16]
@@ -274,10 +282,9 @@ __global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const Latent
     const int t0 = split * per, t1 = min(tiles, t0 + per);
     if (slot < 0 || t0 >= t1) return;   // the merge reads the splits that hold positions
     const bf16* cache = static_cast<const bf16*>(a.cache) + (long)slot * a.max_seq * a.ldc;
-    const int nc = Dp / 8;
-    const RowWalk walk(t, kDecThreads, nc);
+    const RowWalk walk(t, 256, Dp / 8);
     auto issue = [&](int tile, int buf) {
-        const uint32_t dst = sb + L.k_off + buf * L.kbuf;
+        const uint32_t dst = sb + buf * L.kbuf;
         for (RowWalk w = walk; w.row < kDecKeys; w.next()) {
             const int key = tile * kDecKeys + w.row;
             const bool ok = key < len && w.col * 8 < D8;
@@ -285,62 +292,77 @@ __global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const Latent
         }
         cp_async_commit();
     };
-    for (RowWalk w = walk; w.row < 32; w.next()) {   // 16 heads' high parts, then their remainders
-        const int hh = w.row & 15, lo = w.row >> 4;
-        const bool ok = h0 + hh < a.heads;
-        const bf16* q = static_cast<const bf16*>(a.qabs);
-        cp_async16z(sb + L.q_off + w.row * L.row + w.col * 16, ok ? q + (((long)row * a.heads + h0 + hh) * 2 + lo) * Dp + w.col * 8 : q, ok);
-    }
-    issue(t0, 0);
-    float O[NT][4] = {};
-    const int skey = lane * 2;                        // this thread's keys in the softmax of head row `warp`
-    const int kslice = (warp & 7) * 16, khalf = (warp >> 3) * 32;
-    float m = -INFINITY, l = 0.f;
-    for (int tile = t0; tile < t1; ++tile) {
-        const int buf = nbuf == 2 ? (tile - t0) & 1 : 0;
-        const uint32_t kb = sb + L.k_off + buf * L.kbuf;
-        cp_async_wait<0>();
-        __syncthreads();
-        if (nbuf == 2 && tile + 1 < t1) issue(tile + 1, buf ^ 1);
-        float s[4][4] = {};
-        for (int k0 = kslice; k0 < Dp; k0 += 128) {
-            uint32_t ah[4], al[4];
-            const uint32_t qa = sb + L.q_off + (lane & 15) * L.row + (k0 + (lane >> 4) * 8) * 2;
-            ldsm4(qa, ah);
-            ldsm4(qa + 16 * L.row, al);
-            const uint32_t ka = kb + (khalf + (lane & 7) + (lane >> 4) * 8) * L.row + (k0 + ((lane >> 3) & 1) * 8) * 2;
-            uint32_t b[2][4];
+    int tile = t0 + group;
+    if (tile < t1) issue(tile, 0);
+    uint32_t qh[kDecSteps][4], ql[kDecSteps][4];   // query fragments: high parts, remainders
+    {
+        const long stride = 2L * Dp;               // bf16 per head: high parts, then remainders
+        const uint32_t* q0 = reinterpret_cast<const uint32_t*>(static_cast<const bf16*>(a.qabs) + ((long)row * a.heads + h0 + g) * stride) + q4;
+        const uint32_t* q1 = q0 + 8 * (stride / 2);
+        const bool v0 = h0 + g < a.heads, v1 = h0 + g + 8 < a.heads;
 #pragma unroll
-            for (int j = 0; j < 2; ++j) ldsm4(ka + 16 * j * L.row, b[j]);
+        for (int i = 0; i < kDecSteps; ++i) {
+            const int k = (warp + 8 * i) * 8;      // in 32-bit words
+            const bool in = 2 * k < Dp;
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                mma_bf16(s[2 * j], ah[0], ah[1], ah[2], ah[3], b[j][0], b[j][1]);
-                mma_bf16(s[2 * j + 1], ah[0], ah[1], ah[2], ah[3], b[j][2], b[j][3]);
+            for (int e = 0; e < 2; ++e) {
+                qh[i][2 * e] = in && v0 ? q0[k + 4 * e] : 0u;
+                qh[i][2 * e + 1] = in && v1 ? q1[k + 4 * e] : 0u;
+                ql[i][2 * e] = in && v0 ? q0[Dp / 2 + k + 4 * e] : 0u;
+                ql[i][2 * e + 1] = in && v1 ? q1[Dp / 2 + k + 4 * e] : 0u;
             }
+        }
+    }
+    float O[NT][4] = {};
+    const int srow = t >> 4, skey = (t & 15) * 2;   // this thread's head row and keys in the softmax
+    float m = -INFINITY, l = 0.f;
+    for (int buf = 0; tile < t1; tile += 2, buf ^= 1) {
+        const uint32_t kb = sb + buf * L.kbuf;
+        cp_async_wait<0>();
+        group_sync(group);
+        if (tile + 2 < t1) issue(tile + 2, buf ^ 1);
+        float s[4][4] = {};
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                mma_bf16(s[2 * j], al[0], al[1], al[2], al[3], b[j][0], b[j][1]);
-                mma_bf16(s[2 * j + 1], al[0], al[1], al[2], al[3], b[j][2], b[j][3]);
+        for (int i = 0; i < kDecSteps; ++i) {
+            const int k0 = (warp + 8 * i) * 16;
+            if (k0 < Dp) {
+                const uint32_t ka = kb + ((lane & 7) + (lane >> 4) * 8) * L.row + (k0 + ((lane >> 3) & 1) * 8) * 2;
+                uint32_t b[2][4];
+                ldsm4(ka, b[0]);
+                ldsm4(ka + 16 * L.row, b[1]);
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    mma_bf16(s[2 * j], qh[i][0], qh[i][1], qh[i][2], qh[i][3], b[j][0], b[j][1]);
+                    mma_bf16(s[2 * j + 1], qh[i][0], qh[i][1], qh[i][2], qh[i][3], b[j][2], b[j][3]);
+                }
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    mma_bf16(s[2 * j], ql[i][0], ql[i][1], ql[i][2], ql[i][3], b[j][0], b[j][1]);
+                    mma_bf16(s[2 * j + 1], ql[i][0], ql[i][1], ql[i][2], ql[i][3], b[j][2], b[j][3]);
+                }
             }
         }
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-            float* p = part + ((warp & 7) * 16 + g) * kDecS + khalf + 8 * j + 2 * q4;
+            float* p = part + (warp * 16 + g) * kDecS + 8 * j + 2 * q4;
             *reinterpret_cast<float2*>(p) = make_float2(s[j][0], s[j][1]);
             *reinterpret_cast<float2*>(p + 8 * kDecS) = make_float2(s[j][2], s[j][3]);
         }
-        __syncthreads();
+        group_sync(group);
         float2 x = make_float2(0.f, 0.f);
 #pragma unroll
         for (int w = 0; w < 8; ++w) {
-            const float2 y = *reinterpret_cast<const float2*>(part + (w * 16 + warp) * kDecS + skey);
+            const float2 y = *reinterpret_cast<const float2*>(part + (w * 16 + srow) * kDecS + skey);
             x.x += y.x;
             x.y += y.y;
         }
         const int key = tile * kDecKeys + skey;
         x.x = key < len ? x.x * a.scale : -INFINITY;
         x.y = key + 1 < len ? x.y * a.scale : -INFINITY;
-        const float mx = fmaxf(warp_max(fmaxf(x.x, x.y)), m);   // finite: the first key of a tile is always visible
+        float mx = fmaxf(x.x, x.y);
+#pragma unroll
+        for (int o = 1; o < 16; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        mx = fmaxf(mx, m);                          // finite: the first key of a tile is always visible
         const float alpha = expf(m - mx);
         m = mx;
         x.x = expf(x.x - mx);
@@ -348,13 +370,15 @@ __global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const Latent
         l = l * alpha + (x.x + x.y);
         uint32_t hi, lo;
         split_bf16(x.x, x.y, hi, lo);
-        *reinterpret_cast<uint32_t*>(smem + L.p_off + warp * kDecP + skey * 2) = hi;
-        *reinterpret_cast<uint32_t*>(smem + L.p_off + (16 + warp) * kDecP + skey * 2) = lo;
-        if (lane == 0) alphas[warp] = alpha;
-        __syncthreads();
+        *reinterpret_cast<uint32_t*>(smem + L.p_off + srow * kDecP + skey * 2) = hi;
+        *reinterpret_cast<uint32_t*>(smem + L.p_off + (16 + srow) * kDecP + skey * 2) = lo;
+        if ((t & 15) == 0) alphas[srow] = alpha;
+        group_sync(group);
         const float al0 = alphas[g], al1 = alphas[g + 8];
+        if (__any_sync(0xffffffffu, al0 != 1.f || al1 != 1.f)) {
 #pragma unroll
-        for (int j = 0; j < NT; ++j) { O[j][0] *= al0; O[j][1] *= al0; O[j][2] *= al1; O[j][3] *= al1; }
+            for (int j = 0; j < NT; ++j) { O[j][0] *= al0; O[j][1] *= al0; O[j][2] *= al1; O[j][3] *= al1; }
+        }
 #pragma unroll
         for (int k0 = 0; k0 < kDecKeys; k0 += 16) {
             uint32_t ph[4], pl[4];
@@ -374,25 +398,22 @@ __global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const Latent
                 }
             }
         }
-        if (nbuf == 1) {
-            __syncthreads();
-            if (tile + 1 < t1) issue(tile + 1, 0);
-        }
     }
 #pragma unroll
     for (int p = 0; p < 2; ++p) {
         const int h = h0 + g + 8 * p;
         if (h >= a.heads) continue;
-        float* out = part_ptr(a, row, h, split);
+        float* out = part_ptr(a, row, h, 2 * split + group);
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
             const int col = (warp * NT + j) * 8 + 2 * q4;
             if (col < R8) *reinterpret_cast<float2*>(out + col) = make_float2(O[j][2 * p], O[j][2 * p + 1]);
         }
     }
-    l = warp_sum(l);
-    if (lane == 0 && h0 + warp < a.heads) {
-        float* stats = part_ptr(a, row, h0 + warp, split) + R8;
+#pragma unroll
+    for (int o = 1; o < 16; o <<= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+    if ((t & 15) == 0 && h0 + srow < a.heads) {
+        float* stats = part_ptr(a, row, h0 + srow, 2 * split + group) + R8;
         stats[0] = m;
         stats[1] = l;
     }
@@ -403,12 +424,13 @@ constexpr int kOutV = 32;   // value columns per block
 // Block (head and 32 value columns, RB rows): merges the splits, adds the sink to the denominator, applies W_uv and the gate.
 // A warp has four value columns; their first weights are fetched before the kernel waits for its predecessor.
 template <typename A, int RB>
-__global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, const Rows r, int keys) {
+__global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, const Rows r, int keys, int groups) {
     extern __shared__ float sm[];
     const int R8 = pad8(a.R), dim8 = pad8(a.dim), V8 = pad8(a.V), nq = R8 / 4;
     float* lat = sm;                     // [RB][R8]
-    float* wsp = lat + RB * R8;          // [RB][splits] weights of the splits
-    float* red = wsp + ((RB * a.splits + 3) & ~3);   // [RB][R8], second half of the splits
+    const int nparts = groups * a.splits;
+    float* wsp = lat + RB * R8;          // [RB][nparts] weights of the partial results
+    float* red = wsp + ((RB * nparts + 3) & ~3);   // [RB][R8], second half of the splits
     const int vblocks = (V8 + kOutV - 1) / kOutV;
     const int h = blockIdx.x / vblocks, v0 = (blockIdx.x - h * vblocks) * kOutV, row0 = blockIdx.y * RB;
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
@@ -425,7 +447,7 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, con
         }
     pdl_wait();
     if (warp < RB && row0 + warp < r.T) {
-        const int row = row0 + warp, ns = r.slot_of(row) < 0 ? 0 : used_splits(min(r.pos_of(row) + 1, a.max_seq), keys, a.splits);
+        const int row = row0 + warp, ns = r.slot_of(row) < 0 ? 0 : groups * used_splits(min(r.pos_of(row) + 1, a.max_seq), keys, a.splits);
         const float sink = a.sink[h];
         float m = sink;
         for (int s = lane; s < ns; s += 32) m = fmaxf(m, part_ptr(a, row, h, s)[R8]);
@@ -434,12 +456,12 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, con
         for (int s = lane; s < ns; s += 32) {
             const float* p = part_ptr(a, row, h, s) + R8;
             const float w = expf(p[0] - m);
-            wsp[warp * a.splits + s] = w;
+            wsp[warp * nparts + s] = w;
             l = fmaf(w, p[1], l);
         }
         l = warp_sum(l) + expf(sink - m);
         __syncwarp();
-        for (int s = lane; s < ns; s += 32) wsp[warp * a.splits + s] /= l;
+        for (int s = lane; s < ns; s += 32) wsp[warp * nparts + s] /= l;
     }
     __syncthreads();
     const int halves = nq <= 128 ? 2 : 1, part = halves == 2 ? t >> 7 : 0;
@@ -447,12 +469,12 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, con
         const int b = i / nq, c = (i - b * nq) * 4, row = row0 + b;
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
         if (row < r.T) {
-            const int ns = r.slot_of(row) < 0 ? 0 : used_splits(min(r.pos_of(row) + 1, a.max_seq), keys, a.splits);
+            const int ns = r.slot_of(row) < 0 ? 0 : groups * used_splits(min(r.pos_of(row) + 1, a.max_seq), keys, a.splits);
             const float* p = part_ptr(a, row, h, 0) + c;
             const long step = R8 + kPartStats;
 #pragma unroll 8
             for (int s = part; s < ns; s += halves) {
-                const float w = wsp[b * a.splits + s];
+                const float w = wsp[b * nparts + s];
                 const float4 x = *reinterpret_cast<const float4*>(p + s * step);
                 acc.x = fmaf(w, x.x, acc.x);
                 acc.y = fmaf(w, x.y, acc.y);
