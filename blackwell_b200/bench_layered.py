@@ -160,7 +160,7 @@ def latent_records(peak, bf16_peak, size):
         splits = max(1, min(64, ctx // 64, 148 // (M * -(-H // 16))))
         rows = M if not expanded else 1
         qabs = torch.empty((rows * H * 2 * D,), device="cuda", dtype=torch.bfloat16)
-        part = torch.empty((rows * H * 2 * splits * (R + 4),), device="cuda")
+        part = torch.empty((rows * H * splits * (R + 4),), device="cuda")
         kv = torch.empty((ctx if expanded else 1, H * (dim + V)), device="cuda", dtype=torch.bfloat16)
         ids = torch.arange(slots, device="cuda", dtype=torch.int32)
         pos = torch.full((slots,), ctx - 1, device="cuda", dtype=torch.int32)

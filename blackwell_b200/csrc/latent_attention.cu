@@ -32,14 +32,14 @@ cudaError_t prep(const LatentArgs& a, const Rows& r, cudaStream_t st) {
 }
 
 template <typename A, int RB>
-cudaError_t out(const LatentArgs& a, const Rows& r, int keys, int groups, cudaStream_t st) {
+cudaError_t out(const LatentArgs& a, const Rows& r, int keys, cudaStream_t st) {
     static std::once_flag once[kMaxDevices];
     cudaError_t e = allow_smem(latent_out_kernel<A, RB>, once);
     if (e != cudaSuccess) return e;
-    const size_t smem = (size_t)(3 * RB * pad8(a.R) + ((RB * groups * a.splits + 3) & ~3)) * 4;
+    const size_t smem = (size_t)(3 * RB * pad8(a.R) + ((RB * a.splits + 3) & ~3)) * 4;
     if (smem > kMaxDynSmem) return cudaErrorInvalidValue;
     count_launch(1);
-    return launch_pdl(latent_out_kernel<A, RB>, dim3(a.heads * ((pad8(a.V) + kOutV - 1) / kOutV), (r.T + RB - 1) / RB), dim3(256), smem, st, a, r, keys, groups);
+    return launch_pdl(latent_out_kernel<A, RB>, dim3(a.heads * ((pad8(a.V) + kOutV - 1) / kOutV), (r.T + RB - 1) / RB), dim3(256), smem, st, a, r, keys);
 }
 
 template <typename A>
@@ -56,7 +56,7 @@ cudaError_t decode(const LatentArgs& a, const Rows& r, cudaStream_t st) {
     if (e != cudaSuccess) return e;
     count_launch(1);
     return launch_pdl(latent_decode_kernel<NT>, dim3(a.splits, (a.heads + 15) / 16, r.T), dim3(kDecThreads), DecodeSmem(a.R, a.rot).total,
-                      st, a, r);
+                      st, a, r, status_word_ptr());
 }
 
 template <int VT, int MT>
@@ -97,8 +97,8 @@ cudaError_t latent_absorbed(const LatentArgs& a, const Rows& r, int f32, cudaStr
     else if (a.R <= 256) e = decode<4>(a, r, st);
     else e = decode<8>(a, r, st);
     if (e != cudaSuccess) return e;
-    const int keys = by_scalar ? kScalarKeys : kDecKeys, groups = by_scalar ? 1 : 2;
-    return f32 ? out<float, 1>(a, r, keys, groups, st) : rb4 ? out<bf16, 4>(a, r, keys, groups, st) : out<bf16, 1>(a, r, keys, groups, st);
+    const int keys = by_scalar ? kScalarKeys : kDecKeys;
+    return f32 ? out<float, 1>(a, r, keys, st) : rb4 ? out<bf16, 4>(a, r, keys, st) : out<bf16, 1>(a, r, keys, st);
 }
 
 cudaError_t latent_expanded(const LatentArgs& a, const Rows& r, cudaStream_t st) {

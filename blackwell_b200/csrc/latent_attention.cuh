@@ -167,10 +167,9 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentA
         }
 }
 
-// Partial results of a (row, head): two per split (the scalar kernel uses the first `splits` of them), each pad8(R)
-// un-normalised outputs, then the running maximum and the sum.
-__device__ __forceinline__ float* part_ptr(const LatentArgs& a, int row, int h, int i) {
-    return a.part + (((long)row * a.heads + h) * 2 * a.splits + i) * (pad8(a.R) + kPartStats);
+// One partial result per (row, head, split): pad8(R) un-normalised outputs, then the running maximum and the sum.
+__device__ __forceinline__ float* part_ptr(const LatentArgs& a, int row, int h, int split) {
+    return a.part + (((long)row * a.heads + h) * a.splits + split) * (pad8(a.R) + kPartStats);
 }
 // Splits of a context of `len` positions that hold any (tiles of `keys` are dealt out in runs of equal length).
 __device__ __forceinline__ int used_splits(int len, int keys, int splits) {
@@ -243,14 +242,15 @@ constexpr int kDecSteps = 5;               // 16-wide query steps a warp holds: 
 constexpr int kDecP = kDecKeys * 2 + 16;   // bytes of a row of softmax weights
 constexpr int kDecS = kDecKeys + 4;        // floats of a row of partial scores
 struct DecodeSmem {                        // per group: two key tiles, softmax weights, partial scores, rescale factors
-    int row, kbuf, p_off, s_off, f_off, group, total;
+    int row, kbuf, p_off, s_off, f_off, bar_off, group, total;
     __host__ __device__ DecodeSmem(int R, int rot) {
         row = latent_dp(R, rot) * 2 + 16;
         kbuf = kDecKeys * row;
         p_off = 2 * kbuf;
         s_off = p_off + 2 * 16 * kDecP;
         f_off = s_off + 8 * 16 * kDecS * 4;
-        group = f_off + 16 * 4;
+        bar_off = f_off + 2 * 16 * 4;
+        group = bar_off + 16;
         total = 2 * group;
     }
 };
@@ -260,12 +260,12 @@ __device__ __forceinline__ void group_sync(int group) {
 }
 
 // Block (split, 16 heads, row): the tiles of the split alternate between two warp groups that run independently, so that
-// one group's products overlap the other's softmax; each leaves its own partial result.  Inside a group a warp holds every
+// one group's products overlap the other's softmax; their results are merged at the end.  Inside a group a warp holds every
 // eighth 16-wide step of the queries in registers and multiplies it with all keys of the tile; the partial scores meet
 // in shared memory, where 16 neighbouring threads own one head's row.  Output: a warp accumulates latent columns
 // [w * NT * 8, (w + 1) * NT * 8).
 template <int NT>
-__global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const LatentArgs a, const Rows r) {
+__global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const LatentArgs a, const Rows r, int* status) {
     extern __shared__ __align__(16) unsigned char smem_all[];
     const DecodeSmem L(a.R, a.rot);
     const int Dp = latent_dp(a.R, a.rot), R8 = pad8(a.R), D8 = R8 + pad8(a.rot);
@@ -274,7 +274,7 @@ __global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const Latent
     unsigned char* smem = smem_all + group * L.group;
     const uint32_t sb = smem_u32(smem);
     float* part = reinterpret_cast<float*>(smem + L.s_off);    // [8][16][kDecS]
-    float* alphas = reinterpret_cast<float*>(smem + L.f_off);  // [16]
+    float* alphas = reinterpret_cast<float*>(smem + L.f_off);  // [2][16]
     pdl_trigger();
     pdl_wait();
     const int slot = r.slot_of(row), len = min(r.pos_of(row) + 1, a.max_seq);
@@ -282,18 +282,24 @@ __global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const Latent
     const int t0 = split * per, t1 = min(tiles, t0 + per);
     if (slot < 0 || t0 >= t1) return;   // the merge reads the splits that hold positions
     const bf16* cache = static_cast<const bf16*>(a.cache) + (long)slot * a.max_seq * a.ldc;
-    const RowWalk walk(t, 256, Dp / 8);
-    auto issue = [&](int tile, int buf) {
-        const uint32_t dst = sb + buf * L.kbuf;
-        for (RowWalk w = walk; w.row < kDecKeys; w.next()) {
-            const int key = tile * kDecKeys + w.row;
-            const bool ok = key < len && w.col * 8 < D8;
-            cp_async16z(dst + w.row * L.row + w.col * 16, ok ? cache + (long)key * a.ldc + w.col * 8 : cache, ok);
-        }
-        cp_async_commit();
+    // rows past the sequence's end keep what the buffer held before (zeros or earlier keys): their weights are zero
+    zero_smem(smem, 2 * L.kbuf, t, 256);
+    if (t == 0) {
+        mbar_init(sb + L.bar_off, 1);
+        mbar_init(sb + L.bar_off + 8, 1);
+        mbar_fence_init();
+    }
+    fence_proxy_async();
+    group_sync(group);
+    auto issue = [&](int tile, int buf) {   // one row per lane of the group's first warp
+        const uint32_t bar = sb + L.bar_off + 8 * buf;
+        const int key = tile * kDecKeys + lane;
+        if (lane == 0) mbar_expect_tx(bar, min(kDecKeys, len - tile * kDecKeys) * D8 * 2);
+        __syncwarp();
+        if (key < len) bulk_row(sb + buf * L.kbuf + lane * L.row, cache + (long)key * a.ldc, D8 * 2, bar);
     };
     int tile = t0 + group;
-    if (tile < t1) issue(tile, 0);
+    if (tile < t1 && warp == 0) issue(tile, 0);
     uint32_t qh[kDecSteps][4], ql[kDecSteps][4];   // query fragments: high parts, remainders
     {
         const long stride = 2L * Dp;               // bf16 per head: high parts, then remainders
@@ -316,11 +322,14 @@ __global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const Latent
     float O[NT][4] = {};
     const int srow = t >> 4, skey = (t & 15) * 2;   // this thread's head row and keys in the softmax
     float m = -INFINITY, l = 0.f;
+    CopyWait copied{status};
+    uint32_t phases = 0;
     for (int buf = 0; tile < t1; tile += 2, buf ^= 1) {
         const uint32_t kb = sb + buf * L.kbuf;
-        cp_async_wait<0>();
-        group_sync(group);
-        if (tile + 2 < t1) issue(tile + 2, buf ^ 1);
+        copied(sb + L.bar_off + 8 * buf, (phases >> buf) & 1);
+        phases ^= 1u << buf;
+        group_sync(group);                          // everybody is done with the other buffer
+        if (tile + 2 < t1 && warp == 0) issue(tile + 2, buf ^ 1);
         float s[4][4] = {};
 #pragma unroll
         for (int i = 0; i < kDecSteps; ++i) {
@@ -399,23 +408,38 @@ __global__ void __launch_bounds__(kDecThreads) latent_decode_kernel(const Latent
             }
         }
     }
+    // the second group hands its result to the first through its key buffers
+#pragma unroll
+    for (int o = 1; o < 16; o <<= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+    if ((t & 15) == 0) { alphas[srow] = m; alphas[16 + srow] = l; }
+    float* other = reinterpret_cast<float*>(smem_all + L.group);
+    __syncthreads();   // both groups are done with their keys
+    if (group == 1) {
+#pragma unroll
+        for (int j = 0; j < NT; ++j)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) other[(4 * j + i) * 256 + t] = O[j][i];
+    }
+    __syncthreads();
+    if (group == 1) return;
+    const float* second = reinterpret_cast<const float*>(smem_all + L.group + L.f_off);
 #pragma unroll
     for (int p = 0; p < 2; ++p) {
-        const int h = h0 + g + 8 * p;
+        const int hr = g + 8 * p, h = h0 + hr;
         if (h >= a.heads) continue;
-        float* out = part_ptr(a, row, h, 2 * split + group);
+        const float ma = alphas[hr], mb = second[hr], mm = fmaxf(ma, mb), fa = expf(ma - mm), fb = expf(mb - mm);
+        float* out = part_ptr(a, row, h, split);
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
             const int col = (warp * NT + j) * 8 + 2 * q4;
-            if (col < R8) *reinterpret_cast<float2*>(out + col) = make_float2(O[j][2 * p], O[j][2 * p + 1]);
+            if (col < R8)
+                *reinterpret_cast<float2*>(out + col) = make_float2(O[j][2 * p] * fa + other[(4 * j + 2 * p) * 256 + t] * fb,
+                                                                    O[j][2 * p + 1] * fa + other[(4 * j + 2 * p + 1) * 256 + t] * fb);
         }
-    }
-#pragma unroll
-    for (int o = 1; o < 16; o <<= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-    if ((t & 15) == 0 && h0 + srow < a.heads) {
-        float* stats = part_ptr(a, row, h0 + srow, 2 * split + group) + R8;
-        stats[0] = m;
-        stats[1] = l;
+        if (warp == 0 && q4 == 0) {
+            out[R8] = mm;
+            out[R8 + 1] = alphas[16 + hr] * fa + second[16 + hr] * fb;
+        }
     }
 }
 
@@ -424,13 +448,12 @@ constexpr int kOutV = 32;   // value columns per block
 // Block (head and 32 value columns, RB rows): merges the splits, adds the sink to the denominator, applies W_uv and the gate.
 // A warp has four value columns; their first weights are fetched before the kernel waits for its predecessor.
 template <typename A, int RB>
-__global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, const Rows r, int keys, int groups) {
+__global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, const Rows r, int keys) {
     extern __shared__ float sm[];
     const int R8 = pad8(a.R), dim8 = pad8(a.dim), V8 = pad8(a.V), nq = R8 / 4;
     float* lat = sm;                     // [RB][R8]
-    const int nparts = groups * a.splits;
-    float* wsp = lat + RB * R8;          // [RB][nparts] weights of the partial results
-    float* red = wsp + ((RB * nparts + 3) & ~3);   // [RB][R8], second half of the splits
+    float* wsp = lat + RB * R8;          // [RB][splits] weights of the splits
+    float* red = wsp + ((RB * a.splits + 3) & ~3);   // [RB][R8], second half of the splits
     const int vblocks = (V8 + kOutV - 1) / kOutV;
     const int h = blockIdx.x / vblocks, v0 = (blockIdx.x - h * vblocks) * kOutV, row0 = blockIdx.y * RB;
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
@@ -447,7 +470,7 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, con
         }
     pdl_wait();
     if (warp < RB && row0 + warp < r.T) {
-        const int row = row0 + warp, ns = r.slot_of(row) < 0 ? 0 : groups * used_splits(min(r.pos_of(row) + 1, a.max_seq), keys, a.splits);
+        const int row = row0 + warp, ns = r.slot_of(row) < 0 ? 0 : used_splits(min(r.pos_of(row) + 1, a.max_seq), keys, a.splits);
         const float sink = a.sink[h];
         float m = sink;
         for (int s = lane; s < ns; s += 32) m = fmaxf(m, part_ptr(a, row, h, s)[R8]);
@@ -456,12 +479,12 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, con
         for (int s = lane; s < ns; s += 32) {
             const float* p = part_ptr(a, row, h, s) + R8;
             const float w = expf(p[0] - m);
-            wsp[warp * nparts + s] = w;
+            wsp[warp * a.splits + s] = w;
             l = fmaf(w, p[1], l);
         }
         l = warp_sum(l) + expf(sink - m);
         __syncwarp();
-        for (int s = lane; s < ns; s += 32) wsp[warp * nparts + s] /= l;
+        for (int s = lane; s < ns; s += 32) wsp[warp * a.splits + s] /= l;
     }
     __syncthreads();
     const int halves = nq <= 128 ? 2 : 1, part = halves == 2 ? t >> 7 : 0;
@@ -469,12 +492,12 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, con
         const int b = i / nq, c = (i - b * nq) * 4, row = row0 + b;
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
         if (row < r.T) {
-            const int ns = r.slot_of(row) < 0 ? 0 : groups * used_splits(min(r.pos_of(row) + 1, a.max_seq), keys, a.splits);
+            const int ns = r.slot_of(row) < 0 ? 0 : used_splits(min(r.pos_of(row) + 1, a.max_seq), keys, a.splits);
             const float* p = part_ptr(a, row, h, 0) + c;
             const long step = R8 + kPartStats;
 #pragma unroll 8
             for (int s = part; s < ns; s += halves) {
-                const float w = wsp[b * nparts + s];
+                const float w = wsp[b * a.splits + s];
                 const float4 x = *reinterpret_cast<const float4*>(p + s * step);
                 acc.x = fmaf(w, x.x, acc.x);
                 acc.y = fmaf(w, x.y, acc.y);

@@ -305,7 +305,7 @@ public:
         w->proj32 = std::max(w->proj32, (long)in_.N - split_);
         w->mixed = std::max(w->mixed, (long)mixed_ld());
         w->absorbed_bytes = std::max(w->absorbed_bytes, 4L * rows * s_.heads * lm::latent_dp(s_.kv_rank, s_.rot_dim));
-        for (int T = 1; T <= rows; ++T) w->part = std::max(w->part, (long)T * s_.heads * 2 * splits(e, T) * (pad8(s_.kv_rank) + lm::kPartStats));
+        for (int T = 1; T <= rows; ++T) w->part = std::max(w->part, (long)T * s_.heads * splits(e, T) * (pad8(s_.kv_rank) + lm::kPartStats));
         if (expanded_) w->kv = std::max(w->kv, (long)e.max_seq * s_.heads * (pad8(s_.dim) + pad8(s_.vdim)));
         if (owner_) return 0;
         char* c = nullptr;

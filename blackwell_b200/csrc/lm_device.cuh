@@ -15,12 +15,6 @@ template <typename A> __device__ __forceinline__ A from_f(float v);
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16_rn(v); }
 
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const bf16* p) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16),
-                       __uint_as_float(u.y & 0xFFFF0000u));
-}
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
@@ -35,9 +29,6 @@ __device__ __forceinline__ void split_bf16(float x, float y, uint32_t& hi, uint3
     lo = pack_bf16(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xFFFF0000u));
 }
 
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
 // 16 bytes, or zeros when !valid (src must still be a readable address)
 __device__ __forceinline__ void cp_async16z(uint32_t dst, const void* src, bool valid) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
@@ -53,9 +44,6 @@ __device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
 __device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm2(uint32_t addr, uint32_t (&r)[2]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
 }
 // D(16x8) += A(16x16) B(16x8), bf16 operands, fp32 accumulators.  Thread (g = lane / 4, t = lane % 4): a0 row g, a1 row
 // g + 8 (columns 2t, 2t+1), a2 / a3 the same rows, columns 2t+8, 2t+9; b0 / b1 rows 2t, 2t+1 / 2t+8, 2t+9 of column g;
@@ -86,6 +74,29 @@ struct RowWalk {
         if (col >= cols) { col -= cols; ++row; }
     }
 };
+
+// Bulk copy of one row (16-byte aligned on both sides, size a multiple of 16), counted in bytes on an mbarrier.
+__device__ __forceinline__ void bulk_row(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                 ::"r"(dst), "l"(src), "r"(bytes), "r"(bar)
+                 : "memory");
+}
+// Waits for a copy phase; after a wait that gave up (status word set) the thread does not wait again, so that every thread
+// still meets its block's barriers and the kernel ends.
+struct CopyWait {
+    int* status;
+    bool dead = false;
+    __device__ __forceinline__ void operator()(uint32_t bar, uint32_t parity) {
+        if (!dead && !mbar_wait(bar, parity)) {
+            dead = true;
+            if (status) *status = kStatusMbarTimeout;
+        }
+    }
+};
+// Zeroes `bytes` (a multiple of 16) of shared memory that bulk copies will fill: rows and columns they do not cover stay zero.
+__device__ __forceinline__ void zero_smem(unsigned char* p, int bytes, int t, int threads) {
+    for (int i = t * 16; i < bytes; i += threads * 16) *reinterpret_cast<uint4*>(p + i) = make_uint4(0, 0, 0, 0);
+}
 
 // Sum over a block of up to 1024 threads; every thread gets the total.  `buf`: 32 floats of shared memory.
 __device__ __forceinline__ float block_sum(float v, float* buf) {

@@ -121,7 +121,7 @@ struct LatentArgs {
     long ldout;
     // scratch
     void* qabs;                       // [T][heads][2][Dp] bf16 (high, remainder) or [T][heads][Dp] fp32
-    float* part;                      // [T][heads][2 * splits][pad8(R) + kPartStats]
+    float* part;                      // [T][heads][splits][pad8(R) + kPartStats]
     int splits;
     void* kv;                         // expanded keys and values [max_seq][heads * (pad8(dim) + pad8(V))]
 };

@@ -431,7 +431,7 @@ int bw_linear_recurrence(const bw_recurrence_args* a, const bw_rows* rows, int c
  * norm and the key part before rotation (NULL: the rows are in the cache already), gate [T][ld32] one logit per head,
  * Wkv rows uk (head h at h * P8(dim)) then uv, cs cos / sin [max_seq][rot_dims / 2], sink [heads];
  * out [T][heads * P8(V)] = sigmoid(gate) * softmax-with-sink attention.  Scratch: absorbed form qabs
- * (4 * T * heads * P16(P8(R) + P8(rot)) bytes) and part (T * heads * 2 * splits * (P8(R) + 4) floats); expanded form kv
+ * (4 * T * heads * P16(P8(R) + P8(rot)) bytes) and part (T * heads * splits * (P8(R) + 4) floats); expanded form kv
  * (max_seq * heads * (P8(dim) + P8(V)) elements; bfloat16, rows of one sequence only). */
 typedef struct bw_latent_args {
     int heads, dim, rot, V, R, rot_dims;
