@@ -89,8 +89,10 @@ cudaError_t launch_tc(const LinearArgs& a, int ksplit, cudaStream_t st) {
     attr[1].val.clusterDim.y = 1;
     attr[1].val.clusterDim.z = 1;
     cfg.attrs = attr;
-    cfg.numAttrs = SPLIT ? 2 : 1;
+    cfg.numAttrs = SPLIT ? 2 : 1;   // no cluster in the persistent form
     int* status = status_word_ptr();
+    // persistent form: ksplit says whether the weights are too large for L2
+    if (!SPLIT) ksplit = (long)a.N * a.K > (24l << 20) && (long)a.N * a.K > (long)a.T * a.K;
     e = cudaLaunchKernelEx(&cfg, kern, mw, mx, a, ksplit, status);
     count_launch(1);
     return e;

@@ -218,7 +218,8 @@ __device__ __forceinline__ void cluster_sync_all() {
     asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 
-// SPLIT: one tile per cluster of `ksplit` CTAs; otherwise persistent CTAs walk the tiles (row tile fastest).
+// SPLIT: one tile per cluster of `ksplit` CTAs; otherwise persistent CTAs walk the tiles, weight rows fastest while the
+// weights stay in L2, activation rows fastest when they do not (`ksplit` != 0 there).
 template <int NT, bool SPLIT>
 __global__ void __launch_bounds__(kTcThreads, SPLIT ? 2 : 1)
 linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, const LinearArgs a,
@@ -261,6 +262,9 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
     pdl_trigger();
 
     const int rtiles = (a.N + kTcRows - 1) / kTcRows, ttiles = (a.T + NT - 1) / NT, tiles = rtiles * ttiles;
+    const bool tok_fast = !SPLIT && ksplit != 0;
+    auto row_tile = [&](int tile) { return tok_fast ? tile / ttiles : tile % rtiles; };
+    auto tok_tile = [&](int tile) { return tok_fast ? tile % ttiles : tile / rtiles; };
     const int nk = (a.K + kTcK - 1) / kTcK;
     const int kpart = SPLIT ? (int)(blockIdx.x % ksplit) : 0;
     const int kb0 = SPLIT ? (int)((long)nk * kpart / ksplit) : 0, kb1 = SPLIT ? (int)((long)nk * (kpart + 1) / ksplit) : nk;
@@ -272,7 +276,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             int n = 0;
             bool ok = true, waited = false;
             for (int tile = first; tile < tiles && ok; tile += stride) {
-                const int row0 = (tile % rtiles) * kTcRows, tok0 = (tile / rtiles) * NT;
+                const int row0 = row_tile(tile) * kTcRows, tok0 = tok_tile(tile) * NT;
                 int kb = kb0;
                 if (!waited) {   // weights do not depend on the kernel before: fill the ring with them first
                     const int pre = min(S, kb1 - kb0);
@@ -330,7 +334,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             const int d = w % NACC;
             if (!wait(dfull(d), (w / NACC) & 1)) break;
             tc::tc_fence_after();
-            const int row = (tile % rtiles) * kTcRows + quarter * 32 + lane, tok0 = (tile / rtiles) * NT;
+            const int row = row_tile(tile) * kTcRows + quarter * 32 + lane, tok0 = tok_tile(tile) * NT;
             const uint32_t src = tmem + d * NT + ((uint32_t)(quarter * 32) << 16);
             const int g0 = row - lane;                       // the warp's 32 rows
             const bool whole = g0 + 32 <= a.N && (g0 + 32 <= a.split || g0 >= a.split);
@@ -390,7 +394,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
         cluster_sync_all();   // every CTA's partial tile is in its shared memory
         if (!*abort_flag) {
             pdl_wait();
-            const int row0 = (first % rtiles) * kTcRows, tok0 = (first / rtiles) * NT;
+            const int row0 = row_tile(first) * kTcRows, tok0 = tok_tile(first) * NT;
             const int c0 = NT * kpart / ksplit, c1 = NT * (kpart + 1) / ksplit;
             const uint32_t base = smem_u32(part);
             for (int i = c0 * kTcRows + t; i < c1 * kTcRows; i += kTcThreads) {

@@ -61,14 +61,11 @@ def _linear(x, W, T, N, K, x_f32, epilogue=0, cap=0.0, y_f32=1):
     return y[:, :cols]
 
 
-@pytest.mark.parametrize("stream_rows", [0, 8])
-@pytest.mark.parametrize("T", [1, 2, 7, 8, 9, 16, 20, 32, 33, 64, 65, 129, 300])
+@pytest.mark.parametrize("T, stream_rows", [(t, 0) for t in (1, 2, 8, 9, 16, 20, 32, 33, 64, 65, 129, 300)] + [(t, 8) for t in (1, 2, 7, 8)])
 @pytest.mark.parametrize("N, K", [(130, 40), (77, 200), (515, 328), (16, 1032)])
 def test_linear_shapes(cuda, T, N, K, stream_rows):
     from blackwell_b200 import kernels
 
-    if stream_rows and T > 8:
-        pytest.skip("more than eight rows always take the tcgen05 kernel")
     kernels.set_tuning(23, stream_rows + 1)
     try:
         check_linear_shapes(T, N, K)
@@ -95,7 +92,7 @@ def check_linear_shapes(T, N, K):
         assert np.abs(cap - 5.0 * np.tanh(want / 5.0)).max() < 1e-4
 
 
-@pytest.mark.parametrize("T, N, K", [(700, 2048, 512), (3000, 1400, 320), (4096, 4096, 192), (40, 3000, 1024), (100, 20000, 264)])
+@pytest.mark.parametrize("T, N, K", [(700, 2048, 512), (3000, 1400, 320), (4096, 4096, 192), (600, 26000, 1032), (40, 3000, 1024), (100, 20000, 264)])
 def test_linear_large(cuda, T, N, K):
     rng = np.random.default_rng(T)
     _, W = lm.to_bf16(rng.standard_normal((N, K)).astype(np.float32))
