@@ -74,7 +74,7 @@ def vifivik_config(width: int, ff: int, vocab: int, layers: int, head_scale: int
         kind, mixer = [("mamba2", mamba), ("latent_attention", latent), ("latent_attention", {**latent, "kv_from": i - 1}),
                        ("retention", ret)][i % 4]
         out.append({"type": kind, "mixer": dict(mixer), "mlp": {"kind": "dense", "ff": ff}})
-    return {"architecture": "Vifivik", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "layers": out}
+    return {"architecture": "Vifivik", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "logit_softcap": 25.0, "layers": out}
 
 
 # name -> (config.json model, the INT4 decode model of the same width, feed-forward size, layer count and vocabulary)
