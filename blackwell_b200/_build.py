@@ -30,7 +30,7 @@ TRACE_RUN = os.path.join(LIBDIR, "trace_run")
 # what a program that serves config.json models alone needs (no INT4 kernels); model_registry.cu is compiled for it
 # once more with the INT4 family left out
 CONFIG_MODEL_SOURCES = ["service", "decode_glue", "decode_engine", "layered_model", "model_spec", "lm_glue", "linear_bf16",
-                        "recurrence", "latent_attention"]
+                        "recurrence", "latent_attention", "diff_attention"]
 
 # IEEE division and square root are requested explicitly: the quantizers must
 # round exactly like the reference's (v / sc, roundf).

@@ -1,15 +1,17 @@
-// Models described by a config.json (model_spec.h): a list of layers, each a mixer and an optional feed-forward, with
-// the norm on the sublayer's output -- x <- x + norm1(mixer(x)), x <- x + norm2(ff(x)) -- an fp32 residual stream, and
-// logits = softcap(head norm(x)).  Mixers: mamba2, retention (both on the gated linear recurrence), latent attention.
+// Models described by a config.json (model_spec.h): a list of layers, each a mixer and an optional feed-forward, with norms
+// on the sublayers' outputs -- x <- x + norm1(mixer(x)), x <- x + norm2(ff(x)) -- or on both sides -- x <- x +
+// norm1b(mixer(norm1(x))), x <- x + norm2b(ff(norm2(x))) --, an fp32 residual stream, and logits = softcap(head norm(x)).
+// Mixers: mamba2, retention, gated delta rule (all on the gated linear recurrence), latent attention, differential attention.
 //
 // Weights are bfloat16 and stay so on the device; matrices that read the same input are stacked by rows, gate and up
 // rows are interleaved (the product's epilogue applies silu(gate) * up), head blocks are padded to multiples of eight
 // with zero rows / columns.  Two activation formats: bfloat16 (serving) and fp32 (cfg.compute_f32).
 //
-// Per-slot state: for every latent layer that owns a cache [slot][max_seq][latent | rotated key part] in the activation
-// format; for every recurrent layer the fp32 state and, for mamba2, the last inputs of the convolution.  A slot needs no
-// clearing when it is used again: at position 0 states and convolution inputs count as zero, and attention reads
-// positions below the current one only.
+// Per-slot state: for every attention layer that owns a cache, in the activation format, [slot][max_seq][latent | rotated key
+// part] (latent) or a ring [slot][cap][key / value heads] that holds the longest window of the layers that read it and one
+// portion (differential); for every recurrent layer the fp32 state and, for mamba2 and delta, the last inputs of the
+// convolution.  A slot needs no clearing when it is used again: at position 0 states and convolution inputs count as zero,
+// and attention reads positions below the current one only.
 #include <cuda_runtime.h>
 #include <math.h>
 
@@ -60,14 +62,22 @@ struct Loader {
     int tensor(const std::string& name, const std::vector<long>& shape, std::vector<uint16_t>* out) {
         return st.read_bf16(name, shape, out, &ctx.error) ? 0 : bad();
     }
-    int vec(const std::string& name, const std::vector<long>& shape, float** dev) {   // fp32 on the device
+    int floats(const std::string& name, const std::vector<long>& shape, std::vector<float>* f) {   // appended
         std::vector<uint16_t> h;
         BW_TRY(tensor(name, shape, &h));
-        std::vector<float> f(h.size());
-        for (size_t i = 0; i < h.size(); ++i) {
-            const uint32_t u = (uint32_t)h[i] << 16;
-            memcpy(&f[i], &u, 4);
+        for (uint16_t v : h) {
+            const uint32_t u = (uint32_t)v << 16;
+            float x;
+            memcpy(&x, &u, 4);
+            f->push_back(x);
         }
+        return 0;
+    }
+    int vec(const std::string& name, const std::vector<long>& shape, float** dev, double offset = 0) {   // fp32 on the device
+        std::vector<float> f;
+        BW_TRY(floats(name, shape, &f));
+        if (offset != 0)
+            for (float& x : f) x = (float)(x + offset);
         return ctx.upload(dev, f);
     }
     int upload(const Stack& s, Mat* m) {
@@ -101,10 +111,10 @@ struct Loader {
 // Work buffers shared by all layers: largest need over the layers, in elements per row unless noted.
 struct Work {
     long proj = 0, proj32 = 0, conv = 0, mixed = 0, ff = 0, o32 = 0, heads = 0;   // per row
-    long absorbed_bytes = 0, part = 0, kv = 0;                                    // whole buffers
+    long absorbed_bytes = 0, part = 0, kv = 0, chunk_bytes = 0;                   // whole buffers
     void *xb = nullptr, *proj_b = nullptr, *conv_b = nullptr, *mixed_b = nullptr, *ff_b = nullptr, *fin_b = nullptr;
     float *proj32_b = nullptr, *o32_b = nullptr, *log_decay = nullptr, *weight = nullptr, *sub = nullptr, *part_b = nullptr;
-    void *qabs_b = nullptr, *kv_b = nullptr;
+    void *qabs_b = nullptr, *kv_b = nullptr, *chunk_b = nullptr;
     long ldx = 0;
 };
 
@@ -132,10 +142,14 @@ public:
     virtual int run(const Env& e, const Work& w, const lm::Rows& r, cudaStream_t st) = 0;   // w.xb -> w.mixed_b
     int mixed_ld() const { return s_.heads * pad8(s_.vdim); }
     const Mat& out() const { return o_; }
+    const MixerSpec& spec() const { return s_; }
+    virtual bool rotates() const { return false; }   // takes cos / sin of spec().rot
+    void set_rotation(const float2* cs) { cs_ = cs; }
 
 protected:
     MixerSpec s_;
     Mat in_, o_;
+    const float2* cs_ = nullptr;
 };
 
 // Recurrent mixers: N x vdim state per head, gated norm on the read-out.
@@ -159,7 +173,10 @@ protected:
     }
     // chunks on the tensor cores from 16 rows on (bf16); token by token with fp32 FMAs otherwise
     int recur(const Env& e, const lm::RecurrenceArgs& a, const lm::Rows& r, cudaStream_t st) const {
-        if (!e.f32 && !r.row_slot && r.T >= 16 && lm::recurrence_chunk_supported(a)) return lm::recurrence_chunk(a, r, st);
+        if (!e.f32 && !r.row_slot && r.T >= 16) {
+            if (a.delta && lm::delta_chunk_supported(a)) return lm::delta_chunk(a, r, st);
+            if (!a.delta && lm::recurrence_chunk_supported(a)) return lm::recurrence_chunk(a, r, st);
+        }
         return lm::recurrence_step(a, nullptr, r, e.f32, st);
     }
 };
@@ -266,6 +283,145 @@ private:
     float* log_decay_ = nullptr;
 };
 
+class GatedDelta : public RecurrentMixer {
+public:
+    explicit GatedDelta(const MixerSpec& s) : RecurrentMixer(s) { N_ = s.dim; }
+    int load(Loader& l, const std::string& p, int width) override {
+        const int H = s_.heads, qk = s_.kv_heads * s_.dim, v = H * s_.vdim;
+        std::vector<uint16_t> h;
+        std::vector<float> taps, norm;
+        Stack st(width);
+        BW_TRY(l.tensor(p + "g", {v, width}, &h));
+        st.add(h, v, s_.vdim, pad8(s_.vdim));
+        for (const char* name : {"v", "k", "q"}) {
+            const bool values = name[0] == 'v';
+            const int n = values ? v : qk, per = values ? s_.vdim : s_.dim;
+            BW_TRY(l.tensor(p + name, {n, width}, &h));
+            st.add(h, n, per, pad8(per));
+            BW_TRY(l.floats(p + name + ".conv", {n, s_.conv}, &taps));
+        }
+        split_ = st.rows;
+        for (const char* name : {"a", "b"}) {
+            BW_TRY(l.tensor(p + name, {H, width}, &h));
+            st.add(h, H);
+        }
+        BW_TRY(l.upload(st, &in_));
+        BW_TRY(l.ctx.upload(&conv_w_, taps));
+        BW_TRY(l.vec(p + "dt_bias", {H}, &dt_bias_));
+        BW_TRY(l.vec(p + "A_log", {H}, &A_log_));
+        for (int i = 0; i < H; ++i) BW_TRY(l.floats(p + "norm", {s_.vdim}, &norm));   // shared by the heads
+        BW_TRY(l.ctx.upload(&norm_, norm));
+        return l.matrix_by_heads(p + "o", width, H, s_.vdim, &o_);
+    }
+    int alloc(DecodeContext& ctx, const Env& e, Work* w) override {
+        w->proj = std::max(w->proj, (long)split_);
+        w->proj32 = std::max(w->proj32, 2L * s_.heads);
+        w->conv = std::max(w->conv, (long)split_ - mixed_ld());
+        w->heads = std::max(w->heads, (long)s_.heads);
+        if (!e.f32) w->chunk_bytes = std::max(w->chunk_bytes, (long)lm::delta_chunk_bytes(e.max_rows, s_.heads));
+        BW_TRY(ctx.alloc(&ring_, (size_t)e.slots * s_.conv * (s_.heads * s_.vdim + 2 * s_.kv_heads * s_.dim)));
+        return alloc_recurrent(ctx, e, w);
+    }
+    int run(const Env& e, const Work& w, const lm::Rows& r, cudaStream_t st) override {
+        const int H = s_.heads, inner8 = mixed_ld(), qk8 = s_.kv_heads * pad8(s_.dim);
+        BW_TRY(project(e, w, in_, w.xb, w.ldx, r.T, w.proj_b, split_, w.proj32_b, 2 * H, split_, st));
+        lm::ConvArgs c{};
+        c.u = w.proj_b; c.ldu = split_; c.w = conv_w_; c.ring = ring_; c.taps = s_.conv; c.heads = H; c.V = s_.vdim; c.N = s_.dim;
+        c.groups = s_.kv_heads; c.off = inner8; c.out = w.conv_b; c.ldo = split_ - inner8; c.dt_raw = w.proj32_b; c.ld_dt = 2 * H;
+        c.beta_raw = w.proj32_b + H; c.dt_bias = dt_bias_; c.A_log = A_log_; c.log_decay = w.log_decay; c.weight = w.weight;
+        lm::RecurrenceArgs a = recurrence(w);
+        a.groups = s_.kv_heads; a.delta = 1; a.unit_eps = 1e-6f; a.q_scale = (float)(1.0 / sqrt((double)s_.dim)); a.chunk_scratch = w.chunk_b;
+        if (r.row_slot) {
+            BW_TRY(lm::recurrence_step(a, &c, r, e.f32, st));
+        } else {
+            BW_TRY(lm::conv_silu(c, r, e.f32, st));
+            BW_TRY(lm::conv_ring_store(c, r, e.f32, st));
+            a.v = w.conv_b; a.k = e.at(w.conv_b, inner8); a.q = e.at(w.conv_b, inner8 + qk8);
+            a.ldq = a.ldk = a.ldv = c.ldo;
+            a.log_decay = w.log_decay; a.weight = w.weight;
+            BW_TRY(recur(e, a, r, st));
+        }
+        return lm::gated_norm(w.mixed_b, inner8, w.o32_b, inner8, w.proj_b, split_, norm_, r.T, H, s_.vdim, H, 0, e.eps, e.f32, st);
+    }
+
+private:
+    int split_ = 0;
+    float *conv_w_ = nullptr, *dt_bias_ = nullptr, *A_log_ = nullptr, *norm_ = nullptr, *ring_ = nullptr;
+};
+
+class DiffAttention : public Mixer {
+public:
+    DiffAttention(const MixerSpec& s, DiffAttention* owner) : Mixer(s), owner_(owner), reach_(s.window) {
+        if (owner && (reach_ == 0 || (owner->reach_ > 0 && reach_ > owner->reach_))) owner->reach_ = reach_;
+    }
+    int load(Loader& l, const std::string& p, int width) override {
+        const int H = s_.heads, G = s_.kv_heads;
+        std::vector<uint16_t> h;
+        Stack st(width);
+        BW_TRY(l.tensor(p + "q", {2L * H * s_.dim, width}, &h));
+        st.add(h, 2 * H * s_.dim, s_.dim, pad8(s_.dim));
+        if (!owner_) {
+            k_ = st.rows;
+            BW_TRY(l.tensor(p + "k", {2L * G * s_.dim, width}, &h));
+            st.add(h, 2 * G * s_.dim, s_.dim, pad8(s_.dim));
+            v_ = st.rows;
+            BW_TRY(l.tensor(p + "v", {(long)G * s_.vdim, width}, &h));
+            st.add(h, G * s_.vdim, s_.vdim, pad8(s_.vdim));
+        }
+        BW_TRY(l.upload(st, &in_));
+        double dot[2] = {};
+        const char* pairs[2][2] = {{"lq1", "lk1"}, {"lq2", "lk2"}};
+        for (int i = 0; i < 2; ++i) {
+            std::vector<float> a, b;
+            BW_TRY(l.floats(p + pairs[i][0], {s_.dim}, &a));
+            BW_TRY(l.floats(p + pairs[i][1], {s_.dim}, &b));
+            for (int d = 0; d < s_.dim; ++d) dot[i] += (double)a[d] * b[d];
+        }
+        lambda_ = (float)(exp(dot[0]) - exp(dot[1]) + s_.diff);
+        return l.matrix_by_heads(p + "o", width, H, s_.vdim, &o_);
+    }
+    int alloc(DecodeContext& ctx, const Env& e, Work* w) override {
+        if (!lm::diff_attention_supported(base(e))) { ctx.error = "differential attention: these sizes are not supported"; return cudaErrorInvalidValue; }
+        w->proj = std::max(w->proj, (long)in_.N);
+        w->mixed = std::max(w->mixed, (long)mixed_ld());
+        if (owner_) return 0;
+        cap_ = reach_ > 0 ? (int)std::min<long>(e.max_seq, (long)reach_ - 1 + e.max_rows) : e.max_seq;
+        char* c = nullptr;
+        BW_TRY(ctx.alloc(&c, (size_t)e.slots * cap_ * s_.kv_heads * lm::diff_row(s_.dim, s_.vdim) * e.elem()));
+        cache_ = c;
+        return 0;
+    }
+    int run(const Env& e, const Work& w, const lm::Rows& r, cudaStream_t st) override {
+        BW_TRY(project(e, w, in_, w.xb, w.ldx, r.T, w.proj_b, in_.N, nullptr, 0, in_.N, st));
+        lm::DiffAttnArgs a = base(e);
+        const DiffAttention* own = owner_ ? owner_ : this;
+        a.cache = own->cache_; a.cap = own->cap_;
+        a.q = w.proj_b; a.ld = in_.N;
+        if (!owner_) {
+            a.k = e.at(w.proj_b, k_);
+            a.v = e.at(w.proj_b, v_);
+        }
+        a.out = w.mixed_b; a.ldout = mixed_ld();
+        a.splits = lm::diff_attention_splits(a, r.T, e.f32);
+        return lm::diff_attention(a, r, e.f32, st);
+    }
+    bool rotates() const override { return true; }
+
+private:
+    lm::DiffAttnArgs base(const Env& e) const {
+        lm::DiffAttnArgs a{};
+        a.heads = s_.heads; a.kv_heads = s_.kv_heads; a.dim = s_.dim; a.V = s_.vdim; a.window = s_.window; a.rot_dims = s_.rot.dims; a.cs = cs_;
+        a.max_seq = e.max_seq; a.scale = (float)s_.scale; a.lambda = lambda_; a.out_scale = (float)(1.0 - s_.diff); a.eps = e.eps;
+        return a;
+    }
+    DiffAttention* owner_;
+    int reach_;                // longest window over this layer's cache, 0: everything
+    int k_ = 0, v_ = 0;        // columns of the projection
+    int cap_ = 0;
+    float lambda_ = 0;
+    void* cache_ = nullptr;
+};
+
 class LatentAttention : public Mixer {
 public:
     LatentAttention(const MixerSpec& s, LatentAttention* owner) : Mixer(s), owner_(owner) {}
@@ -326,8 +482,7 @@ public:
         if (expanded_ && !r.row_slot && r.T > kAbsorbedRows) return lm::latent_expanded(a, r, st);
         return lm::latent_absorbed(a, r, e.f32, st);
     }
-    void set_rotation(const float2* cs) { cs_ = cs; }
-    const MixerSpec& spec() const { return s_; }
+    bool rotates() const override { return true; }
 
 private:
     int q8() const { return pad8(s_.dim) + pad8(s_.rot_dim); }
@@ -338,7 +493,7 @@ private:
     }
     lm::LatentArgs base(const Env& e) const {
         lm::LatentArgs a{};
-        a.heads = s_.heads; a.dim = s_.dim; a.rot = s_.rot_dim; a.V = s_.vdim; a.R = s_.kv_rank; a.rot_dims = s_.rot_dims;
+        a.heads = s_.heads; a.dim = s_.dim; a.rot = s_.rot_dim; a.V = s_.vdim; a.R = s_.kv_rank; a.rot_dims = s_.rot.dims;
         a.scale = (float)s_.scale; a.eps = e.eps; a.cs = cs_; a.max_seq = e.max_seq; a.ldc = lm::latent_row(s_.kv_rank, s_.rot_dim);
         return a;
     }
@@ -348,12 +503,12 @@ private:
     Mat kv_;
     float *dkv_norm_ = nullptr, *sink_ = nullptr;
     void* cache_ = nullptr;
-    const float2* cs_ = nullptr;
 };
 
 struct Layer {
     std::unique_ptr<Mixer> mixer;
-    float *norm1 = nullptr, *norm2 = nullptr;
+    float *in1 = nullptr, *in2 = nullptr;     // norms of the sublayers' inputs, NULL: none
+    float *out1 = nullptr, *out2 = nullptr;   // norms of the sublayers' outputs
     Mat gu, down;
     int ff = 0;
 };
@@ -419,7 +574,8 @@ int LayeredModel::load(DecodeContext& ctx, const std::string& dir) {
     if (!l.st.open(dir + "/model.safetensors", &ctx.error)) return -1;
     BW_TRY(l.matrix("embed", spec_.vocab, spec_.width, &embed_));
     BW_TRY(l.matrix("head", spec_.vocab, spec_.width, &head_));
-    BW_TRY(l.vec("final.norm", {spec_.width}, &final_norm_));
+    auto norm = [&](const std::string& name, float** dev) { return l.vec(name, {spec_.width}, dev, spec_.norm_offset); };
+    BW_TRY(norm("final.norm", &final_norm_));
     layers_.resize(spec_.layers.size());
     for (size_t i = 0; i < layers_.size(); ++i) {
         const LayerSpec& s = spec_.layers[i];
@@ -432,12 +588,19 @@ int LayeredModel::load(DecodeContext& ctx, const std::string& dir) {
                 L.mixer.reset(new LatentAttention(
                     s.mixer, s.mixer.kv_from >= 0 ? static_cast<LatentAttention*>(layers_[s.mixer.kv_from].mixer.get()) : nullptr));
                 break;
+            case MixerSpec::kDelta: L.mixer.reset(new GatedDelta(s.mixer)); break;
+            case MixerSpec::kDiffAttention:
+                L.mixer.reset(new DiffAttention(
+                    s.mixer, s.mixer.kv_from >= 0 ? static_cast<DiffAttention*>(layers_[s.mixer.kv_from].mixer.get()) : nullptr));
+                break;
         }
         BW_TRY(L.mixer->load(l, p + "mix.", spec_.width));
-        BW_TRY(l.vec(p + "norm1", {spec_.width}, &L.norm1));
+        if (spec_.input_norms) BW_TRY(norm(p + "norm1", &L.in1));
+        BW_TRY(norm(p + (spec_.input_norms ? "norm1b" : "norm1"), &L.out1));
         L.ff = s.ff;
         if (s.ff > 0) {
-            BW_TRY(l.vec(p + "norm2", {spec_.width}, &L.norm2));
+            if (spec_.input_norms) BW_TRY(norm(p + "norm2", &L.in2));
+            BW_TRY(norm(p + (spec_.input_norms ? "norm2b" : "norm2"), &L.out2));
             std::vector<uint16_t> g, u;
             BW_TRY(l.tensor(p + "mlp.gate", {s.ff, spec_.width}, &g));
             BW_TRY(l.tensor(p + "mlp.up", {s.ff, spec_.width}, &u));
@@ -456,21 +619,23 @@ int LayeredModel::load(DecodeContext& ctx, const std::string& dir) {
 
 int LayeredModel::alloc_state(DecodeContext& ctx) {
     // cos / sin of every rotation in use, computed in double precision
-    std::map<std::pair<int, double>, float2*> tables;
+    std::map<Rotation, float2*> tables;
     for (Layer& L : layers_) {
-        LatentAttention* a = dynamic_cast<LatentAttention*>(L.mixer.get());
-        if (a) {
-            const int half = a->spec().rot_dims / 2;
-            float2*& t = tables[{a->spec().rot_dims, a->spec().rot_base}];
+        if (L.mixer->rotates()) {
+            const Rotation& rot = L.mixer->spec().rot;
+            const int half = rot.dims / 2;
+            float2*& t = tables[rot];
             if (!t) {
                 std::vector<float2> h((size_t)std::max(1, half) * env_.max_seq);
+                const double gain = rot.gain();
                 for (int i = 0; i < half; ++i) {
-                    const double f = pow(a->spec().rot_base, -2.0 * i / a->spec().rot_dims);
-                    for (int p = 0; p < env_.max_seq; ++p) h[(size_t)p * half + i] = make_float2((float)cos(p * f), (float)sin(p * f));
+                    const double f = rot.frequency(i);
+                    for (int p = 0; p < env_.max_seq; ++p)
+                        h[(size_t)p * half + i] = make_float2((float)(cos(p * f) * gain), (float)(sin(p * f) * gain));
                 }
                 BW_TRY(ctx.upload(&t, h));
             }
-            a->set_rotation(t);
+            L.mixer->set_rotation(t);
         }
         BW_TRY(L.mixer->alloc(ctx, env_, &w_));
         w_.ff = std::max(w_.ff, (long)pad8(L.ff));
@@ -499,6 +664,8 @@ int LayeredModel::alloc_state(DecodeContext& ctx) {
     char* q = nullptr;
     BW_TRY(ctx.alloc(&q, w_.absorbed_bytes));
     w_.qabs_b = q;
+    BW_TRY(ctx.alloc(&q, w_.chunk_bytes));
+    w_.chunk_b = q;
     BW_TRY(ctx.alloc(&x_, rows * env_.width));
     ctx.x = x_;
     return ctx.alloc(&ctx.logits, (size_t)env_.slots * spec_.vocab);
@@ -506,16 +673,18 @@ int LayeredModel::alloc_state(DecodeContext& ctx) {
 
 int LayeredModel::enqueue_layers(DecodeContext& ctx, const lm::Rows& r, const int* tokens, cudaStream_t st) {
     const Env& e = env_;
-    BW_TRY(lm::embed(x_, w_.xb, w_.ldx, embed_.p, embed_.ld, tokens, r.T, e.width, spec_.vocab, e.f32, st));
+    BW_TRY(lm::embed(x_, w_.xb, w_.ldx, embed_.p, embed_.ld, tokens, r.T, e.width, spec_.vocab, (float)spec_.embed_scale, layers_[0].in1,
+                     e.eps, e.f32, st));
     for (size_t i = 0; i < layers_.size(); ++i) {
         Layer& L = layers_[i];
+        const float* next = i + 1 < layers_.size() ? layers_[i + 1].in1 : nullptr;   // the next layer's input norm
         lm::LinearArgs a{};
         a.T = r.T; a.f32 = e.f32; a.y = w_.sub; a.ldy = e.width; a.y_f32 = 1; a.N = a.split = e.width;
         BW_TRY(L.mixer->run(e, w_, r, st));
         const Mat& o = L.mixer->out();
         a.x = w_.mixed_b; a.ldx = L.mixer->mixed_ld(); a.W = o.p; a.ldw = o.ld; a.K = o.K;
         BW_TRY(lm::linear(a, st));
-        BW_TRY(lm::norm_add(x_, w_.xb, w_.ldx, w_.sub, L.norm1, r.T, e.width, e.eps, e.f32, st));
+        BW_TRY(lm::norm_add(x_, w_.xb, w_.ldx, w_.sub, L.out1, L.ff > 0 ? L.in2 : next, r.T, e.width, e.eps, e.f32, st));
         if (L.ff > 0) {
             lm::LinearArgs g{};
             g.x = w_.xb; g.ldx = w_.ldx; g.W = L.gu.p; g.ldw = L.gu.ld; g.T = r.T; g.N = g.split = L.gu.N; g.K = L.gu.K;
@@ -523,7 +692,7 @@ int LayeredModel::enqueue_layers(DecodeContext& ctx, const lm::Rows& r, const in
             BW_TRY(lm::linear(g, st));
             a.x = w_.ff_b; a.ldx = pad8(L.ff); a.W = L.down.p; a.ldw = L.down.ld; a.K = L.down.K;
             BW_TRY(lm::linear(a, st));
-            BW_TRY(lm::norm_add(x_, w_.xb, w_.ldx, w_.sub, L.norm2, r.T, e.width, e.eps, e.f32, st));
+            BW_TRY(lm::norm_add(x_, w_.xb, w_.ldx, w_.sub, L.out2, next, r.T, e.width, e.eps, e.f32, st));
         }
         if (ctx.watch)
             BW_TRY(cudaMemcpyAsync(ctx.watch + ((size_t)i * ctx.watch_rows + ctx.watch_row0) * e.width, x_, (size_t)r.T * e.width * 4,

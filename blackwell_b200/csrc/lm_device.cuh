@@ -98,6 +98,18 @@ __device__ __forceinline__ void zero_smem(unsigned char* p, int bytes, int t, in
     for (int i = t * 16; i < bytes; i += threads * 16) *reinterpret_cast<uint4*>(p + i) = make_uint4(0, 0, 0, 0);
 }
 
+// Shared memory of another block of the cluster, and the cluster's barrier.
+__device__ __forceinline__ float ld_dsmem(uint32_t addr, uint32_t rank) {
+    uint32_t ra;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(addr), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(ra) : "memory");
+    return v;
+}
+__device__ __forceinline__ void cluster_sync_all() {
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+
 // Sum over a block of up to 1024 threads; every thread gets the total.  `buf`: 32 floats of shared memory.
 __device__ __forceinline__ float block_sum(float v, float* buf) {
     v = warp_sum(v);

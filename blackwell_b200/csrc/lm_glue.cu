@@ -11,24 +11,53 @@ namespace bw {
 namespace lm {
 namespace {
 
+constexpr int kKeep = 8;   // values of a row that a thread of a norm kernel keeps in registers
+
+// xb = x / rms(x) * next (next NULL: x) for the block's row x, of which keep[] holds the first values.
 template <typename A>
-__global__ void __launch_bounds__(256) embed_kernel(float* x, A* xb, long ldxb, const bf16* table, long ldt, const int* tokens,
-                                                    int width, int vocab) {
-    pdl_trigger();
-    pdl_wait();
-    const int r = blockIdx.y, i = blockIdx.x * 256 + threadIdx.x;
-    if (i >= width) return;
-    int tok = tokens[r];
-    tok = tok < 0 ? 0 : tok >= vocab ? vocab - 1 : tok;
-    const float v = to_f(table[(long)tok * ldt + i]);
-    x[(long)r * width + i] = v;
-    xb[(long)r * ldxb + i] = from_f<A>(v);
+__device__ __forceinline__ void next_input(A* xb, const float* x, const float* next, const float (&keep)[kKeep], int width, float eps,
+                                           float* buf) {
+    float f = 1.f;
+    if (next) {
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < kKeep; ++j) ss = fmaf(keep[j], keep[j], ss);
+        for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
+        f = 1.0f / sqrtf(block_sum(ss, buf) / (float)width + eps);
+    }
+#pragma unroll
+    for (int j = 0; j < kKeep; ++j) {
+        const int i = j * blockDim.x + threadIdx.x;
+        if (i < width) xb[i] = from_f<A>(next ? keep[j] * f * next[i] : keep[j]);
+    }
+    for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) xb[i] = from_f<A>(next ? x[i] * f * next[i] : x[i]);
 }
 
-// ADD: x += y / rms(y) * w and xb = x; otherwise xb = x / rms(x) * w for a listed row.
+template <typename A>
+__global__ void __launch_bounds__(512) embed_kernel(float* x, A* xb, long ldxb, const bf16* table, long ldt, const int* tokens,
+                                                    int width, int vocab, float scale, const float* next, float eps) {
+    __shared__ float buf[32];
+    pdl_trigger();
+    pdl_wait();
+    const long r = blockIdx.x;
+    int tok = tokens[r];
+    tok = tok < 0 ? 0 : tok >= vocab ? vocab - 1 : tok;
+    const bf16* row = table + (long)tok * ldt;
+    float keep[kKeep];
+#pragma unroll
+    for (int j = 0; j < kKeep; ++j) {
+        const int i = j * blockDim.x + threadIdx.x;
+        keep[j] = i < width ? to_f(row[i]) * scale : 0.f;
+        if (i < width) x[r * width + i] = keep[j];
+    }
+    for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) x[r * width + i] = to_f(row[i]) * scale;
+    next_input<A>(xb + r * ldxb, x + r * width, next, keep, width, eps, buf);
+}
+
+// ADD: x += y / rms(y) * w and xb = the next sublayer's input; otherwise xb = x / rms(x) * w for a listed row.
 template <typename A, bool ADD>
-__global__ void __launch_bounds__(512) norm_kernel(float* x, A* xb, long ldxb, const float* y, const float* w, const int* rows,
-                                                   int width, float eps) {
+__global__ void __launch_bounds__(512) norm_kernel(float* x, A* xb, long ldxb, const float* y, const float* w, const float* next,
+                                                   const int* rows, int width, float eps) {
     __shared__ float buf[32];
     pdl_trigger();
     pdl_wait();
@@ -36,7 +65,6 @@ __global__ void __launch_bounds__(512) norm_kernel(float* x, A* xb, long ldxb, c
     const long r = rows ? rows[out_row] : out_row;
     const float* src = (ADD ? y : x) + r * width;
     float ss = 0.f;
-    constexpr int kKeep = 8;   // the first values stay in registers
     float keep[kKeep];
 #pragma unroll
     for (int j = 0; j < kKeep; ++j) {
@@ -51,15 +79,18 @@ __global__ void __launch_bounds__(512) norm_kernel(float* x, A* xb, long ldxb, c
         if (ADD) {
             v += x[r * width + i];
             x[r * width + i] = v;
+        } else {
+            xb[(long)out_row * ldxb + i] = from_f<A>(v);
         }
-        xb[(long)out_row * ldxb + i] = from_f<A>(v);
+        return v;
     };
 #pragma unroll
     for (int j = 0; j < kKeep; ++j) {
         const int i = j * blockDim.x + threadIdx.x;
-        if (i < width) emit(i, keep[j]);
+        if (i < width) keep[j] = emit(i, keep[j]);
     }
     for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) emit(i, src[i]);
+    if (ADD) next_input<A>(xb + r * ldxb, x + r * width, next, keep, width, eps, buf);
 }
 
 template <typename A>
@@ -115,7 +146,7 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const ConvArgs c, const 
         }
         const A* u = static_cast<const A*>(c.u) + c.off + col;
         const float* ring = c.ring + (long)r.slot * c.taps * channels + ch;
-        const float bias = c.bias[ch];
+        const float bias = c.bias ? c.bias[ch] : 0.f;
         for (int t = t0; t < t1; ++t) {
             float y = bias;
             for (int j = 0; j < c.taps; ++j) {
@@ -133,7 +164,7 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const ConvArgs c, const 
         for (int t = t0; t < t1; ++t) {
             const float dt = softplus_f(c.dt_raw[(long)t * c.ld_dt + h] + b);
             c.log_decay[(long)t * c.heads + h] = a * dt;
-            c.weight[(long)t * c.heads + h] = dt;
+            c.weight[(long)t * c.heads + h] = c.beta_raw ? sigmoid_f(c.beta_raw[(long)t * c.ld_dt + h]) : dt;
         }
     }
 }
@@ -151,23 +182,25 @@ __global__ void __launch_bounds__(128) conv_ring_kernel(const ConvArgs c, const 
 
 }  // namespace
 
-cudaError_t embed(float* x, void* xb, long ldxb, const bf16* table, long ldt, const int* tokens, int T, int width, int vocab,
-                  int f32, cudaStream_t st) {
-    const dim3 grid((width + 255) / 256, T), block(256);
-    count_launch(1);
-    return f32 ? launch_pdl(embed_kernel<float>, grid, block, 0, st, x, static_cast<float*>(xb), ldxb, table, ldt, tokens, width, vocab)
-               : launch_pdl(embed_kernel<bf16>, grid, block, 0, st, x, static_cast<bf16*>(xb), ldxb, table, ldt, tokens, width, vocab);
-}
-
 static int norm_threads(int width) { return width <= 256 ? 64 : width <= 1024 ? 128 : width <= 2048 ? 256 : 512; }
 
-cudaError_t norm_add(float* x, void* xb, long ldxb, const float* y, const float* w, int T, int width, float eps, int f32,
-                     cudaStream_t st) {
+cudaError_t embed(float* x, void* xb, long ldxb, const bf16* table, long ldt, const int* tokens, int T, int width, int vocab,
+                  float scale, const float* next, float eps, int f32, cudaStream_t st) {
+    const dim3 grid(T), block(norm_threads(width));
+    count_launch(1);
+    return f32 ? launch_pdl(embed_kernel<float>, grid, block, 0, st, x, static_cast<float*>(xb), ldxb, table, ldt, tokens, width, vocab,
+                            scale, next, eps)
+               : launch_pdl(embed_kernel<bf16>, grid, block, 0, st, x, static_cast<bf16*>(xb), ldxb, table, ldt, tokens, width, vocab,
+                            scale, next, eps);
+}
+
+cudaError_t norm_add(float* x, void* xb, long ldxb, const float* y, const float* w, const float* next, int T, int width, float eps,
+                     int f32, cudaStream_t st) {
     const dim3 grid(T), block(norm_threads(width));
     const int* none = nullptr;
     count_launch(1);
-    return f32 ? launch_pdl(norm_kernel<float, true>, grid, block, 0, st, x, static_cast<float*>(xb), ldxb, y, w, none, width, eps)
-               : launch_pdl(norm_kernel<bf16, true>, grid, block, 0, st, x, static_cast<bf16*>(xb), ldxb, y, w, none, width, eps);
+    return f32 ? launch_pdl(norm_kernel<float, true>, grid, block, 0, st, x, static_cast<float*>(xb), ldxb, y, w, next, none, width, eps)
+               : launch_pdl(norm_kernel<bf16, true>, grid, block, 0, st, x, static_cast<bf16*>(xb), ldxb, y, w, next, none, width, eps);
 }
 
 cudaError_t norm_rows(void* xb, long ldxb, const float* x, const float* w, const int* rows, int T, int width, float eps, int f32,
@@ -176,8 +209,8 @@ cudaError_t norm_rows(void* xb, long ldxb, const float* x, const float* w, const
     float* xm = const_cast<float*>(x);
     const float* none = nullptr;
     count_launch(1);
-    return f32 ? launch_pdl(norm_kernel<float, false>, grid, block, 0, st, xm, static_cast<float*>(xb), ldxb, none, w, rows, width, eps)
-               : launch_pdl(norm_kernel<bf16, false>, grid, block, 0, st, xm, static_cast<bf16*>(xb), ldxb, none, w, rows, width, eps);
+    return f32 ? launch_pdl(norm_kernel<float, false>, grid, block, 0, st, xm, static_cast<float*>(xb), ldxb, none, w, none, rows, width, eps)
+               : launch_pdl(norm_kernel<bf16, false>, grid, block, 0, st, xm, static_cast<bf16*>(xb), ldxb, none, w, none, rows, width, eps);
 }
 
 cudaError_t gated_norm(void* out, long ldout, const float* o, long ldo, const void* gate, long ldg, const float* w, int T,

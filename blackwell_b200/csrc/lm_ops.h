@@ -47,11 +47,13 @@ struct Rows {
 };
 
 // ---------------------------------------------------------------- embedding, norms
+// xb = norm(x) * next in the activation type, or x itself where next is NULL: the next sublayer's input.
+// x <- table[token] * scale
 cudaError_t embed(float* x, void* xb, long ldxb, const bf16* table, long ldt, const int* tokens, int T, int width, int vocab,
-                  int f32, cudaStream_t st);
-// x <- x + y / sqrt(mean y^2 + eps) * w; xb = x in the activation type
-cudaError_t norm_add(float* x, void* xb, long ldxb, const float* y, const float* w, int T, int width, float eps, int f32,
-                     cudaStream_t st);
+                  float scale, const float* next, float eps, int f32, cudaStream_t st);
+// x <- x + y / sqrt(mean y^2 + eps) * w
+cudaError_t norm_add(float* x, void* xb, long ldxb, const float* y, const float* w, const float* next, int T, int width, float eps,
+                     int f32, cudaStream_t st);
 // xb = x / sqrt(mean x^2 + eps) * w for the rows listed in `rows` (NULL: all)
 cudaError_t norm_rows(void* xb, long ldxb, const float* x, const float* w, const int* rows, int T, int width, float eps, int f32,
                       cudaStream_t st);
@@ -65,7 +67,7 @@ struct ConvArgs {
     const void* u;          // projection rows: channel c (conv order) at column off_x + padded position
     long ldu;
     const float* w;         // [channels][taps]
-    const float* bias;      // [channels]
+    const float* bias;      // [channels] or NULL
     float* ring;            // [slot][taps][channels] last inputs, entry = position % taps
     int taps, heads, V, N, groups;   // channels: heads * V, then groups * N (k), then groups * N (q)
     int off;                // first padded column of the convolved part in u
@@ -74,6 +76,7 @@ struct ConvArgs {
     const float* dt_raw;    // [T][ld_dt]
     long ld_dt;
     const float *dt_bias, *A_log;    // [heads]
+    const float* beta_raw;           // [T][ld_dt] or NULL: the weight is sigmoid(beta_raw) instead of the step size
     float *log_decay, *weight;       // [T][heads]
 };
 cudaError_t conv_silu(const ConvArgs& c, const Rows& r, int f32, cudaStream_t st);     // several rows of one sequence
@@ -81,6 +84,9 @@ cudaError_t conv_ring_store(const ConvArgs& c, const Rows& r, int f32, cudaStrea
 
 // ---------------------------------------------------------------- gated linear recurrence
 //   S_t = exp(log_decay_t) S_(t-1) + weight_t k_t v_t^T,   o_t = S_t^T q_t + D v_t        (per head; S is N x V, fp32)
+// Delta rule (`delta`): k and q enter as unit vectors, x / sqrt(sum x^2 + unit_eps), q times q_scale, and what is written is the
+// part of v_t that the decayed state does not hold yet:
+//   S_t = S' + k_t u_t^T  with  S' = exp(log_decay_t) S_(t-1),  u_t = weight_t (v_t - S'^T k_t),   o_t = S_t^T q_t
 struct RecurrenceArgs {
     const void *q, *k, *v;           // q/k of head h at column (h / (heads / groups)) * pad8(N), v at h * pad8(V)
     long ldq, ldk, ldv;
@@ -92,11 +98,17 @@ struct RecurrenceArgs {
     float* S;                         // [slot][heads][N][pad8(V)]
     float* o;                         // [T][ldo], head h at column h * pad8(V)
     long ldo;
+    int delta;                        // log_decay and weight are given, D is not
+    float unit_eps, q_scale;
+    void* chunk_scratch;              // delta_chunk_bytes, delta chunks only
 };
 // `conv` != NULL (one row per sequence): q, k, v and the decays come from the projection through the convolution.
 cudaError_t recurrence_step(const RecurrenceArgs& a, const ConvArgs* conv, const Rows& r, int f32, cudaStream_t st);
 bool recurrence_chunk_supported(const RecurrenceArgs& a);
 cudaError_t recurrence_chunk(const RecurrenceArgs& a, const Rows& r, cudaStream_t st);   // bf16, rows of one sequence
+size_t delta_chunk_bytes(int rows, int heads);
+bool delta_chunk_supported(const RecurrenceArgs& a);
+cudaError_t delta_chunk(const RecurrenceArgs& a, const Rows& r, cudaStream_t st);        // bf16, rows of one sequence
 
 // ---------------------------------------------------------------- latent attention
 constexpr int kPartStats = 4;   // floats after a split's outputs: running maximum, sum, padding
@@ -133,6 +145,31 @@ bool latent_expanded_supported(const LatentArgs& a);
 cudaError_t latent_absorbed(const LatentArgs& a, const Rows& r, int f32, cudaStream_t st);
 // Expanded form, rows of one sequence, bf16: keys and values of the whole context through Wkv, then flash attention.
 cudaError_t latent_expanded(const LatentArgs& a, const Rows& r, cudaStream_t st);
+
+// ---------------------------------------------------------------- differential attention
+// Two softmax maps per query head over the same values, causal, over the last `window` positions:
+//   o = a1 - lambda a2,   out = o / sqrt(mean o^2 + eps) * out_scale        (per head, a_i = softmax(scale q_i k_i^T) v)
+// Query head h reads key / value head h / (heads / kv_heads).  Rotated pairs are (i, i + rot_dims / 2).
+struct DiffAttnArgs {
+    int heads, kv_heads, dim, V;
+    int window;                       // 0: all earlier positions
+    int rot_dims;
+    const float2* cs;                 // cos / sin [max_seq][rot_dims / 2]
+    int max_seq;
+    float scale, lambda, out_scale, eps;
+    void* cache;                      // [slot][cap] rows of kv_heads * diff_row: position p at row p % cap
+    int cap;                          // max_seq, or at least window - 1 + the rows of a call
+    void* q;                          // [T][ld], head h's map i at (2 h + i) * pad8(dim), not rotated yet; portions rotate in place
+    const void *k, *v;                // [T][ld], laid out the same way / head g at g * pad8(V); NULL: already in the cache
+    long ld;
+    void* out;                        // [T][ldout], head h at h * pad8(V)
+    long ldout;
+    int splits;                       // context splits of a token step (a cluster of 1, 2, 4 or 8 blocks)
+};
+inline __host__ __device__ int diff_row(int dim, int V) { return 2 * pad8(dim) + pad8(V); }   // map 1 key, map 2 key, value
+bool diff_attention_supported(const DiffAttnArgs& a);
+int diff_attention_splits(const DiffAttnArgs& a, int rows, int f32);
+cudaError_t diff_attention(const DiffAttnArgs& a, const Rows& r, int f32, cudaStream_t st);
 
 }  // namespace lm
 }  // namespace bw

@@ -1,12 +1,27 @@
 // Readers of config.json, one per architecture, and the table of the architectures.
 #include "model_spec.h"
 
+#include <math.h>
 #include <stdio.h>
 #include <string.h>
+
+#include <algorithm>
 
 #include "../../include/blackwell_b200.h"
 
 namespace bw {
+
+double Rotation::frequency(int i) const {
+    const double f = pow(base, -2.0 * i / dims);
+    if (factor == 0) return f;
+    const double pi = 3.14159265358979323846;
+    auto pair_of = [&](double turns) { return dims * log(original / (2 * pi * turns)) / (2 * log(base)); };
+    const double lo = std::max(floor(pair_of(fast)), 0.0), hi = std::min(ceil(pair_of(slow)), dims - 1.0);
+    const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+    return f / factor * ramp + f * (1 - ramp);
+}
+double Rotation::gain() const { return factor == 0 ? 1.0 : 0.1 * log(factor) + 1.0; }
+
 namespace {
 
 struct Reader {   // typed access with one error message
@@ -56,26 +71,101 @@ bool read_retention(const Json& m, const std::string& at, Reader& r, MixerSpec* 
     return r.ok;
 }
 
+// 'rot' of a mixer: dims (even, at most `size`), base and, optionally, YaRN scaling.
+void read_rotation(const Json& m, const std::string& at, int size, Reader& r, Rotation* rot) {
+    const Json* j = r.need(m, "rot", at);
+    if (!j) return;
+    rot->dims = r.integer(*j, "dims", at + " rot", 0, size);
+    rot->base = r.real(*j, "base", at + " rot");
+    if (r.ok && (rot->dims % 2 != 0 || !(rot->base > 0))) r.fail(at + ": bad rotation");
+    const Json* s = j->get("scaling");
+    if (!r.ok || !s || s->is_null()) return;
+    rot->factor = r.real(*s, "factor", at + " rot scaling");
+    rot->original = r.real(*s, "original", at + " rot scaling");
+    rot->fast = r.real(*s, "fast", at + " rot scaling");
+    rot->slow = r.real(*s, "slow", at + " rot scaling");
+    if (r.ok && !(rot->factor > 0 && rot->original > 0 && rot->fast > 0 && rot->slow > 0 && rot->base != 1))
+        r.fail(at + ": bad rotation scaling");
+}
+
+// 'kv_from': an earlier layer of the same kind that has a cache of its own.
+bool read_kv_from(const Json& m, const std::string& at, int layer, const ModelSpec& model, Reader& r, MixerSpec* s) {
+    const Json* from = m.get("kv_from");
+    if (!r.ok || !from || from->is_null()) return false;
+    s->kv_from = r.integer(m, "kv_from", at, 0, layer - 1);
+    if (!r.ok) return false;
+    const MixerSpec& o = model.layers[s->kv_from].mixer;
+    if (o.kind != s->kind || o.kv_from >= 0 || o.kv_rank != s->kv_rank || o.rot_dim != s->rot_dim || !(o.rot == s->rot) ||
+        (s->kind == MixerSpec::kDiffAttention && (o.kv_heads != s->kv_heads || o.dim != s->dim || o.vdim != s->vdim)))
+        r.fail(at + ": 'kv_from' names a layer whose cache does not fit");
+    return r.ok;
+}
+
 bool read_latent(const Json& m, const std::string& at, int layer, const ModelSpec& model, Reader& r, MixerSpec* s) {
     s->kind = MixerSpec::kLatentAttention;
     s->dim = r.integer(m, "dim", at, 1);
     s->rot_dim = r.integer(m, "rot_dim", at, 1);
     s->kv_rank = r.integer(m, "kv_rank", at, 1, 2048);
     s->scale = r.real(m, "scale", at);
-    const Json* rot = r.need(m, "rot", at);
-    if (rot) {
-        s->rot_dims = r.integer(*rot, "dims", at + " rot", 0, s->rot_dim);
-        s->rot_base = r.real(*rot, "base", at + " rot");
-        if (r.ok && (s->rot_dims % 2 != 0 || !(s->rot_base > 0))) r.fail(at + ": bad rotation");
-    }
-    const Json* from = m.get("kv_from");
-    if (from && !from->is_null()) {
-        s->kv_from = r.integer(m, "kv_from", at, 0, layer - 1);
+    read_rotation(m, at, s->rot_dim, r, &s->rot);
+    read_kv_from(m, at, layer, model, r, s);
+    return r.ok;
+}
+
+bool read_kv_heads(const Json& m, const std::string& at, Reader& r, MixerSpec* s) {
+    s->kv_heads = r.integer(m, "kv_heads", at, 1);
+    if (r.ok && s->heads % s->kv_heads != 0) r.fail(at + ": 'kv_heads' does not divide 'heads'");
+    return r.ok;
+}
+
+bool read_delta(const Json& m, const std::string& at, Reader& r, MixerSpec* s) {
+    s->kind = MixerSpec::kDelta;
+    s->dim = r.integer(m, "dim", at, 1, 512);
+    s->conv = r.integer(m, "conv", at, 1, 64);
+    return read_kv_heads(m, at, r, s);
+}
+
+bool read_diff_attention(const Json& m, const std::string& at, int layer, const ModelSpec& model, Reader& r, MixerSpec* s) {
+    s->kind = MixerSpec::kDiffAttention;
+    s->dim = r.integer(m, "dim", at, 1, 4096);
+    if (r.ok && s->vdim > 2048) r.fail(at + ": 'vdim' is out of range");
+    read_kv_heads(m, at, r, s);
+    s->scale = r.real(m, "scale", at);
+    s->diff = r.real(m, "diff", at);
+    const Json* mask = m.get("mask");
+    if (mask && !mask->is_null()) s->window = r.integer(*mask, "size", at + " mask", 1);
+    read_rotation(m, at, s->dim, r, &s->rot);
+    read_kv_from(m, at, layer, model, r, s);
+    return r.ok;
+}
+
+// 'mlp' of a layer: dense, or null for none.
+void read_mlp(const Json& l, const std::string& at, Reader& r, LayerSpec* s) {
+    const Json* mlp = l.get("mlp");
+    if (!r.ok || !mlp || mlp->is_null()) return;
+    const Json* kind = mlp->get("kind");
+    if (!kind || kind->str != "dense") r.fail(at + ": unknown feed-forward kind");
+    s->ff = r.integer(*mlp, "ff", at + " mlp", 1);
+}
+
+// The list 'layers'; `mixer` reads the mixer of one layer by its type.
+template <typename F>
+bool read_layers(const Json& j, Reader& r, ModelSpec* spec, F mixer) {
+    const Json* layers = r.need(j, "layers", "the model");
+    if (!r.ok) return false;
+    if (layers->type != Json::kArray || layers->arr.empty()) { r.fail("'layers' is not a list"); return false; }
+    for (size_t i = 0; i < layers->arr.size() && r.ok; ++i) {
+        const Json& l = layers->arr[i];
+        const std::string at = "layer " + std::to_string(i);
+        const Json *type = r.need(l, "type", at), *m = r.need(l, "mixer", at);
         if (!r.ok) return false;
-        const MixerSpec& o = model.layers[s->kv_from].mixer;
-        if (o.kind != MixerSpec::kLatentAttention || o.kv_from >= 0 || o.kv_rank != s->kv_rank || o.rot_dim != s->rot_dim ||
-            o.rot_dims != s->rot_dims || o.rot_base != s->rot_base)
-            r.fail(at + ": 'kv_from' names a layer whose cache does not fit");
+        LayerSpec s;
+        s.mixer.heads = r.integer(*m, "heads", at, 1);
+        s.mixer.vdim = r.integer(*m, "vdim", at, 1);
+        if (!r.ok) return false;
+        mixer(type->str, *m, at, (int)i, &s.mixer);
+        read_mlp(l, at, r, &s);
+        spec->layers.push_back(s);
     }
     return r.ok;
 }
@@ -91,31 +181,29 @@ bool read_vifivik(const Json& j, ModelSpec* spec, std::string* err) {
         spec->softcap = r.real(j, "logit_softcap", "the model");
         if (r.ok && spec->softcap < 0) r.fail("'logit_softcap' is negative");
     }
-    const Json* layers = r.need(j, "layers", "the model");
-    if (!r.ok) return false;
-    if (layers->type != Json::kArray || layers->arr.empty()) { r.fail("'layers' is not a list"); return false; }
-    for (size_t i = 0; i < layers->arr.size() && r.ok; ++i) {
-        const Json& l = layers->arr[i];
-        const std::string at = "layer " + std::to_string(i);
-        const Json *type = r.need(l, "type", at), *m = r.need(l, "mixer", at);
-        if (!r.ok) return false;
-        LayerSpec s;
-        s.mixer.heads = r.integer(*m, "heads", at, 1);
-        s.mixer.vdim = r.integer(*m, "vdim", at, 1);
-        if (!r.ok) return false;
-        if (type->str == "mamba2") read_mamba2(*m, at, r, &s.mixer);
-        else if (type->str == "latent_attention") read_latent(*m, at, (int)i, *spec, r, &s.mixer);
-        else if (type->str == "retention") read_retention(*m, at, r, &s.mixer);
-        else r.fail(at + ": unknown type '" + type->str + "'");
-        const Json* mlp = l.get("mlp");
-        if (r.ok && mlp && !mlp->is_null()) {
-            const Json* kind = mlp->get("kind");
-            if (!kind || kind->str != "dense") r.fail(at + ": unknown feed-forward kind");
-            s.ff = r.integer(*mlp, "ff", at + " mlp", 1);
-        }
-        spec->layers.push_back(s);
-    }
-    return r.ok;
+    return read_layers(j, r, spec, [&](const std::string& type, const Json& m, const std::string& at, int i, MixerSpec* s) {
+        if (type == "mamba2") read_mamba2(m, at, r, s);
+        else if (type == "latent_attention") read_latent(m, at, i, *spec, r, s);
+        else if (type == "retention") read_retention(m, at, r, s);
+        else r.fail(at + ": unknown type '" + type + "'");
+    });
+}
+
+// Lanedra: norms around every sublayer; gated delta-rule and windowed differential-attention mixers in any order; gated
+// feed-forward or none.
+bool read_lanedra(const Json& j, ModelSpec* spec, std::string* err) {
+    Reader r{err};
+    spec->vocab = r.integer(j, "vocab", "the model", 1);
+    spec->width = r.integer(j, "width", "the model", 1);
+    if (const Json* n = r.need(j, "norm", "the model")) spec->eps = r.real(*n, "eps", "norm");
+    if (const Json* e = r.need(j, "embedding", "the model")) spec->embed_scale = r.real(*e, "scale", "embedding");
+    spec->input_norms = true;
+    spec->norm_offset = 1;
+    return read_layers(j, r, spec, [&](const std::string& type, const Json& m, const std::string& at, int i, MixerSpec* s) {
+        if (type == "delta") read_delta(m, at, r, s);
+        else if (type == "attention") read_diff_attention(m, at, i, *spec, r, s);
+        else r.fail(at + ": unknown type '" + type + "'");
+    });
 }
 
 struct Architecture {
@@ -124,6 +212,7 @@ struct Architecture {
 };
 const Architecture kArchitectures[] = {
     {"Vifivik", read_vifivik},
+    {"Lanedra", read_lanedra},
 };
 
 }  // namespace
@@ -168,6 +257,8 @@ extern "C" int bw_model_probe(const char* dir, bw_model_info* out, char* message
         if (l.mixer.kind == bw::MixerSpec::kMamba2) ++out->mamba2_layers;
         if (l.mixer.kind == bw::MixerSpec::kRetention) ++out->retention_layers;
         if (l.mixer.kind == bw::MixerSpec::kLatentAttention) ++out->latent_layers;
+        if (l.mixer.kind == bw::MixerSpec::kDelta) ++out->delta_layers;
+        if (l.mixer.kind == bw::MixerSpec::kDiffAttention) ++out->diff_attention_layers;
         if (l.mixer.kv_from >= 0) ++out->shared_cache_layers;
     }
     return 0;

@@ -1,9 +1,10 @@
 // Gated linear recurrence  S_t = exp(a_t) S_(t-1) + w_t k_t v_t^T,  o_t = S_t^T q_t + D v_t  with an fp32 state per
 // head, N x V.  Mamba-2 (a_t, w_t from the token, q / k shared by a group of heads) and retention (constant a per head)
-// are both instances.
+// are both instances; the delta rule replaces w_t v_t by w_t (v_t - exp(a_t) S_(t-1)^T k_t), with unit vectors k and q.
 //   recurrence_step_kernel   one token per sequence (decode) or a short / 32-bit run of tokens: the state tile of a CTA
 //                            stays in registers, fp32 FMAs.  CONV: the convolution over the last inputs, silu and the
-//                            step size are computed in the same launch.
+//                            step size are computed in the same launch.  DELTA: both products of the state (with k and with
+//                            q) are taken before the write, o = S'^T q + (k q) u, so that one reduction serves both.
 //   recurrence_chunk_kernel  prompts: 64 tokens at a time on the tensor cores (mma.sync bf16).  q, k and v are bf16 values;
 //                            the decayed scores, the weighted values and the state enter their products as a bf16 high part
 //                            plus a bf16 remainder.  State, decays and sums are fp32.
@@ -18,14 +19,15 @@ constexpr int kRecV = 32;      // state columns per CTA
 constexpr int kRecThreads = 256;
 
 // NR: state rows per thread (rows n = ng + 32 i of 32 row groups); 8 lanes hold 4 columns each.
-template <typename A, int NR, bool CONV>
+template <typename A, int NR, bool CONV, bool DELTA>
 __global__ void __launch_bounds__(kRecThreads) recurrence_step_kernel(const RecurrenceArgs a, const ConvArgs c, const Rows r) {
     extern __shared__ float sm[];
     const int N = a.N, N8 = pad8(a.N), V8 = pad8(a.V);
     float* qs = sm;                 // [32 * NR] (zero beyond N)
     float* ks = qs + 32 * NR;
     float* vs = ks + 32 * NR;       // [32]
-    float* red = vs + kRecV;        // [2][8 warps][32]
+    float* red = vs + kRecV;        // [2][8 warps][32], DELTA: once for k, once for q
+    constexpr int kRed = (DELTA ? 2 : 1) * 8 * kRecV;
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
     const int c4 = (lane & 7) * 4, ng = warp * 4 + (lane >> 3);
     const int h = blockIdx.y, v0 = blockIdx.x * kRecV;
@@ -68,7 +70,7 @@ __global__ void __launch_bounds__(kRecThreads) recurrence_step_kernel(const Recu
                 float y = 0.f;
                 if (ch >= 0) {
                     const float now = to_f(u[col]);
-                    y = c.bias[ch];
+                    y = c.bias ? c.bias[ch] : 0.f;
                     for (int j = 0; j < c.taps - 1; ++j) {
                         const int p = pos0 - (c.taps - 1) + j;
                         if (p >= 0) y = fmaf(c.w[ch * c.taps + j], ring[(long)(p % c.taps) * channels + ch], y);
@@ -83,7 +85,7 @@ __global__ void __launch_bounds__(kRecThreads) recurrence_step_kernel(const Recu
             }
             const float dt = softplus_f(c.dt_raw[(long)row * c.ld_dt + h] + c.dt_bias[h]);
             la = -expf(c.A_log[h]) * dt;
-            w = dt;
+            w = c.beta_raw ? sigmoid_f(c.beta_raw[(long)row * c.ld_dt + h]) : dt;
         } else {
             const A* q = static_cast<const A*>(a.q) + (long)row * a.ldq + grp * N8;
             const A* k = static_cast<const A*>(a.k) + (long)row * a.ldk + grp * N8;
@@ -100,6 +102,84 @@ __global__ void __launch_bounds__(kRecThreads) recurrence_step_kernel(const Recu
         const float d = expf(la);
         const float4 v = *reinterpret_cast<const float4*>(vs + c4);
         float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (DELTA) {
+            float sq = 0.f, sk = 0.f, kq = 0.f;
+            for (int i = lane; i < 32 * NR; i += 32) {
+                const float qi = qs[i], ki = ks[i];
+                sq = fmaf(qi, qi, sq);
+                sk = fmaf(ki, ki, sk);
+                kq = fmaf(ki, qi, kq);
+            }
+            const float rq = a.q_scale / sqrtf(warp_sum(sq) + a.unit_eps), rk = 1.0f / sqrtf(warp_sum(sk) + a.unit_eps);
+            kq = warp_sum(kq) * rq * rk;
+            float kn[NR];
+            float4 z = make_float4(0.f, 0.f, 0.f, 0.f);   // S'^T k, y: S'^T q
+#pragma unroll
+            for (int i = 0; i < NR; ++i) {
+                const int n = ng + 32 * i;
+                const float qn = qs[n] * rq;
+                kn[i] = ks[n] * rk;
+                S[i].x *= d;
+                S[i].y *= d;
+                S[i].z *= d;
+                S[i].w *= d;
+                z.x = fmaf(S[i].x, kn[i], z.x);
+                z.y = fmaf(S[i].y, kn[i], z.y);
+                z.z = fmaf(S[i].z, kn[i], z.z);
+                z.w = fmaf(S[i].w, kn[i], z.w);
+                y.x = fmaf(S[i].x, qn, y.x);
+                y.y = fmaf(S[i].y, qn, y.y);
+                y.z = fmaf(S[i].z, qn, y.z);
+                y.w = fmaf(S[i].w, qn, y.w);
+            }
+#pragma unroll
+            for (int o = 8; o <= 16; o <<= 1) {
+                z.x += __shfl_xor_sync(0xffffffffu, z.x, o);
+                z.y += __shfl_xor_sync(0xffffffffu, z.y, o);
+                z.z += __shfl_xor_sync(0xffffffffu, z.z, o);
+                z.w += __shfl_xor_sync(0xffffffffu, z.w, o);
+                y.x += __shfl_xor_sync(0xffffffffu, y.x, o);
+                y.y += __shfl_xor_sync(0xffffffffu, y.y, o);
+                y.z += __shfl_xor_sync(0xffffffffu, y.z, o);
+                y.w += __shfl_xor_sync(0xffffffffu, y.w, o);
+            }
+            float *rz = red + (rr & 1) * kRed, *ry = rz + 8 * kRecV;
+            if (lane < 8) {
+                *reinterpret_cast<float4*>(rz + warp * kRecV + c4) = z;
+                *reinterpret_cast<float4*>(ry + warp * kRecV + c4) = y;
+            }
+            __syncthreads();   // also frees qs / ks / vs for the next row
+            z = y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float4 p = *reinterpret_cast<const float4*>(rz + i * kRecV + c4);
+                z.x += p.x;
+                z.y += p.y;
+                z.z += p.z;
+                z.w += p.w;
+            }
+            const float4 u = make_float4(w * (v.x - z.x), w * (v.y - z.y), w * (v.z - z.z), w * (v.w - z.w));
+#pragma unroll
+            for (int i = 0; i < NR; ++i) {
+                S[i].x = fmaf(kn[i], u.x, S[i].x);
+                S[i].y = fmaf(kn[i], u.y, S[i].y);
+                S[i].z = fmaf(kn[i], u.z, S[i].z);
+                S[i].w = fmaf(kn[i], u.w, S[i].w);
+            }
+            if (warp == 0 && lane < 8 && colv) {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const float4 p = *reinterpret_cast<const float4*>(ry + i * kRecV + c4);
+                    y.x += p.x;
+                    y.y += p.y;
+                    y.z += p.z;
+                    y.w += p.w;
+                }
+                *reinterpret_cast<float4*>(a.o + (long)row * a.ldo + h * V8 + v0 + c4) =
+                    make_float4(fmaf(kq, u.x, y.x), fmaf(kq, u.y, y.y), fmaf(kq, u.z, y.z), fmaf(kq, u.w, y.w));
+            }
+            continue;
+        }
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
             const int n = ng + 32 * i;
@@ -120,7 +200,7 @@ __global__ void __launch_bounds__(kRecThreads) recurrence_step_kernel(const Recu
             y.z += __shfl_xor_sync(0xffffffffu, y.z, o);
             y.w += __shfl_xor_sync(0xffffffffu, y.w, o);
         }
-        float* rb = red + (rr & 1) * 8 * kRecV;
+        float* rb = red + (rr & 1) * kRed;
         if (lane < 8) *reinterpret_cast<float4*>(rb + warp * kRecV + c4) = y;
         const float vt = t < kRecV ? vs[t] : 0.f;
         __syncthreads();   // also frees qs / ks / vs for the next row

@@ -39,7 +39,7 @@ _L.bw_decode_watch_layers.argtypes = [C.c_void_p, C.c_void_p, C.c_long]
 class ModelInfo(C.Structure):
     _fields_ = [("architecture", C.c_char * 64), ("layers", C.c_int), ("width", C.c_int), ("vocab", C.c_int),
                 ("mamba2_layers", C.c_int), ("retention_layers", C.c_int), ("latent_layers", C.c_int),
-                ("shared_cache_layers", C.c_int)]
+                ("shared_cache_layers", C.c_int), ("delta_layers", C.c_int), ("diff_attention_layers", C.c_int)]
 
 
 _L.bw_model_probe.argtypes = [C.c_char_p, C.POINTER(ModelInfo), C.c_char_p, C.c_int]

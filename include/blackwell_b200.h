@@ -370,8 +370,8 @@ int bw_decode_buffers(bw_decode* d, float** logits, float** hidden, int** positi
 int bw_decode_destroy(bw_decode* d);
 
 /* Model families.  bw_decode_create looks at the weight directory: one with a config.json is a layered model whose
- * architecture config.json names ("Vifivik": mamba2, latent-attention and retention layers; weights in
- * model.safetensors, bfloat16) -- sizes and constants come from config.json, the corresponding fields of bw_decode_config
+ * architecture config.json names ("Vifivik": mamba2, latent-attention and retention layers; "Lanedra": gated delta-rule and
+ * windowed differential-attention layers; weights in model.safetensors, bfloat16) -- sizes and constants come from config.json, the corresponding fields of bw_decode_config
  * are ignored and bw_decode_get_config returns them; any other directory is the INT4 container format above.
  * bw_model_probe reads config.json only (no GPU) and, where it is not usable, leaves the reason in message.
  *   Layered models take portions: bw_decode_begin runs each prompt but its last token through the prompt kernels, so
@@ -385,6 +385,7 @@ typedef struct bw_model_info {
     char architecture[64];
     int layers, width, vocab;
     int mamba2_layers, retention_layers, latent_layers, shared_cache_layers;
+    int delta_layers, diff_attention_layers;
 } bw_model_info;
 int bw_model_probe(const char* dir, bw_model_info* out, char* message, int message_bytes);
 int bw_decode_steps(const bw_decode* d, int longest_prompt, int new_tokens);
@@ -426,6 +427,13 @@ typedef struct bw_recurrence_args {
     long ldo;
 } bw_recurrence_args;
 int bw_linear_recurrence(const bw_recurrence_args* a, const bw_rows* rows, int chunked, int f32, void* stream);
+/* Gated delta rule on the same operands (log_decay and weight required, D unused): with k and q taken as unit vectors
+ * x / sqrt(sum x^2 + unit_eps), q times q_scale,
+ *   S' = exp(log_decay) S_(t-1),  u_t = weight (v_t - S'^T k_t),  S_t = S' + k_t u_t^T,  o_t = S_t^T q_t.
+ * scratch: bw_delta_rule_scratch_bytes(T, heads), chunked calls only (bfloat16, rows of one sequence, N <= 256). */
+size_t bw_delta_rule_scratch_bytes(int rows, int heads);
+int bw_delta_rule(const bw_recurrence_args* a, float unit_eps, float q_scale, void* scratch, const bw_rows* rows, int chunked, int f32,
+                  void* stream);
 /* Latent attention: a position is cached as [latent (R) | rotated key part (rot)], blocks padded to P8, one vector for all
  * heads.  q [T][heads * (P8(dim) + P8(rot))] (the expanded form rotates it in place), dkv [T][ld32] the latent before its
  * norm and the key part before rotation (NULL: the rows are in the cache already), gate [T][ld32] one logit per head,
@@ -456,6 +464,28 @@ typedef struct bw_latent_args {
     void* kv;
 } bw_latent_args;
 int bw_latent_attention(const bw_latent_args* a, const bw_rows* rows, int expanded, int f32, void* stream);
+/* Differential attention: two causal softmax maps per query head over the last `window` positions (0: all), both over the same
+ * values; out = o / sqrt(mean o^2 + eps) * out_scale with o = a1 - lambda a2.  q [T][ld]: head h's map i at
+ * (2 h + i) * P8(dim); k likewise over the key / value heads, v: head g at g * P8(V); all before rotation (portions and the 32-bit
+ * form rotate q in place); k, v NULL: the positions are in the cache already.  Pairs (i, i + rot_dims / 2) are rotated by
+ * cs [max_seq][rot_dims / 2] cos / sin.  cache [slot][cap][kv_heads * (2 * P8(dim) + P8(V))], position p in row p % cap; cap is
+ * max_seq or at least window - 1 + rows of one sequence.  dim <= 4096, V <= 2048.  splits: blocks (1, 2, 4, 8) that share the
+ * context of a token step, 0 = automatic. */
+typedef struct bw_diff_attention_args {
+    int heads, kv_heads, dim, V, window, rot_dims;
+    const void* cs;
+    int max_seq;
+    float scale, lambda, out_scale, eps;
+    void* cache;
+    int cap;
+    void* q;
+    const void *k, *v;
+    long ld;
+    void* out;
+    long ldout;
+    int splits;
+} bw_diff_attention_args;
+int bw_diff_attention(const bw_diff_attention_args* a, const bw_rows* rows, int f32, void* stream);
 
 /* ---- Tensor-parallel exchange over peer memory (no counterpart in the reference, which is single-GPU) ----
  * All-reduce of the K-split projections' partial sums across the GPUs of one box through NVLink peer loads.

@@ -135,8 +135,139 @@ def feed_forward(w, p, x):
     return linear(w[p + "down"], silu(linear(w[p + "gate"], x)) * linear(w[p + "up"], x))
 
 
-def forward(config, w, tokens):
-    """(logits [T, vocab], residual streams [layers, T, width])"""
+def offset_norm(x, w, eps):
+    """RMS norm whose weight is stored as its distance from one."""
+    return rms_unit(x, eps) * (1.0 + np.asarray(w, F))
+
+
+def yarn_frequencies(dims, base, scaling):
+    """(frequency of every rotated pair, factor on cos and sin).  Pairs that turn more than ``fast`` times within the original
+    context keep their frequency, those that turn less than ``slow`` times are divided by ``factor``, with a ramp between."""
+    i = np.arange(dims // 2)
+    f = np.asarray(base, F) ** (-2.0 * i / dims)
+    if scaling is None:
+        return f, 1.0
+
+    def pair_of(turns):
+        return dims * np.log(scaling["original"] / (2 * np.pi * turns)) / (2 * np.log(base))
+
+    lo = max(np.floor(pair_of(scaling["fast"])), 0)
+    hi = min(np.ceil(pair_of(scaling["slow"])), dims - 1)
+    ramp = np.clip((i - lo) / max(hi - lo, 0.001), 0, 1)
+    return f / scaling["factor"] * ramp + f * (1 - ramp), 0.1 * np.log(scaling["factor"]) + 1.0
+
+
+def rotate_half(x, positions, dims, freq, gain):
+    """x [T, ..., D]: the pairs (i, i + dims/2) below ``dims`` turn by position * freq_i, scaled by gain; the rest passes."""
+    out = np.array(x, F)
+    h = dims // 2
+    for t, p in enumerate(positions):
+        c, s = np.cos(p * freq) * gain, np.sin(p * freq) * gain
+        u, v = np.array(x[t, ..., :h]), np.array(x[t, ..., h:dims])
+        out[t, ..., :h] = u * c - v * s
+        out[t, ..., h:dims] = v * c + u * s
+    return out
+
+
+def unit_vectors(x):
+    return x / np.sqrt(np.sum(np.square(x), axis=-1, keepdims=True) + 1e-6)
+
+
+def delta_rule(q, k, v, decay, beta):
+    """S <- decay_t S; u = beta_t (v_t - S^T k_t); S <- S + k_t u^T; o_t = S^T q_t.  q, k [T, H, N]; v [T, H, V]."""
+    T, H, N = q.shape
+    S = np.zeros((H, N, v.shape[2]))
+    o = np.zeros(v.shape)
+    for t in range(T):
+        S = decay[t][:, None, None] * S
+        u = beta[t][:, None] * (v[t] - np.einsum("hnv,hn->hv", S, k[t]))
+        S = S + k[t][:, :, None] * u[:, None, :]
+        o[t] = np.einsum("hnv,hn->hv", S, q[t])
+    return o
+
+
+def delta(w, p, m, eps, x):
+    H, G, D, V, T = m["heads"], m["kv_heads"], m["dim"], m["vdim"], x.shape[0]
+
+    def mixed(name):
+        taps = np.asarray(w[p + name + ".conv"], F)
+        return silu(causal_conv(linear(w[p + name], x), taps, np.zeros(len(taps))))
+
+    of = [h // (H // G) for h in range(H)]
+    q = unit_vectors(mixed("q").reshape(T, G, D))[:, of] * D ** -0.5
+    k = unit_vectors(mixed("k").reshape(T, G, D))[:, of]
+    v = mixed("v").reshape(T, H, V)
+    beta = sigmoid(linear(w[p + "b"], x))
+    decay = np.exp(-np.exp(np.asarray(w[p + "A_log"], F)) * softplus(linear(w[p + "a"], x) + np.asarray(w[p + "dt_bias"], F)))
+    o = rms_norm(delta_rule(q, k, v, decay, beta), w[p + "norm"], eps)
+    return linear(w[p + "o"], o.reshape(T, H * V) * silu(linear(w[p + "g"], x)))
+
+
+def rotated_maps(y, heads, m):
+    """Projection rows [T, heads * 2 * dim] -> rotated [T, heads, 2 maps, dim]"""
+    r = m["rot"]
+    freq, gain = yarn_frequencies(r["dims"], r["base"], r.get("scaling"))
+    return rotate_half(y.reshape(len(y), heads, 2, m["dim"]), np.arange(len(y)), r["dims"], freq, gain)
+
+
+def attention_entries(w, p, m, x):
+    """What an attention layer caches: (rotated keys [T, kv_heads, 2, dim], values [T, kv_heads, vdim])."""
+    return rotated_maps(linear(w[p + "k"], x), m["kv_heads"], m), linear(w[p + "v"], x).reshape(len(x), m["kv_heads"], m["vdim"])
+
+
+def visible(T, size):
+    """[T, T]: position i sees j with 0 <= i - j < size"""
+    i, j = np.arange(T)[:, None], np.arange(T)[None, :]
+    return (j <= i) & (i - j < size)
+
+
+def softmax(scores):
+    e = np.exp(scores - np.max(scores, axis=-1, keepdims=True))
+    return e / np.sum(e, axis=-1, keepdims=True)
+
+
+def map_lambda(w, p, diff):
+    lq1, lk1, lq2, lk2 = (np.asarray(w[p + n], F) for n in ("lq1", "lk1", "lq2", "lk2"))
+    return np.exp(lq1 @ lk1) - np.exp(lq2 @ lk2) + diff
+
+
+def differential_attention(w, p, m, eps, x, entries):
+    H, G, V, T = m["heads"], m["kv_heads"], m["vdim"], x.shape[0]
+    k, v = entries
+    q = rotated_maps(linear(w[p + "q"], x), H, m)
+    seen = visible(T, m["mask"]["size"])
+    out = np.zeros((T, H, V))
+    for h in range(H):
+        g = h // (H // G)
+        a1, a2 = (softmax(np.where(seen, (q[:, h, i] @ k[:, g, i].T) * m["scale"], -np.inf)) @ v[:, g] for i in range(2))
+        out[:, h] = a1 - map_lambda(w, p, m["diff"]) * a2
+    return linear(w[p + "o"], (rms_unit(out, eps) * (1.0 - m["diff"])).reshape(T, H * V))
+
+
+def forward_lanedra(config, w, tokens):
+    eps = config["norm"]["eps"]
+    x = np.asarray(w["embed"], F)[np.asarray(tokens)] * config["embedding"]["scale"]
+    streams, cached = [], {}
+    for i, L in enumerate(config["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        mp = p + "mix."
+        h = offset_norm(x, w[p + "norm1"], eps)
+        if L["type"] == "delta":
+            y = delta(w, mp, m, eps, h)
+        elif L["type"] == "attention":
+            if "kv_from" not in m:
+                cached[i] = attention_entries(w, mp, m, h)
+            y = differential_attention(w, mp, m, eps, h, cached[m.get("kv_from", i)])
+        else:
+            raise ValueError(L["type"])
+        x = x + offset_norm(y, w[p + "norm1b"], eps)
+        if L.get("mlp") is not None:
+            x = x + offset_norm(feed_forward(w, p + "mlp.", offset_norm(x, w[p + "norm2"], eps)), w[p + "norm2b"], eps)
+        streams.append(x)
+    return linear(w["head"], offset_norm(x, w["final.norm"], eps)), np.stack(streams)
+
+
+def forward_vifivik(config, w, tokens):
     eps = config["norm"]["eps"]
     x = np.asarray(w["embed"], F)[np.asarray(tokens)]
     streams, cached = [], {}
@@ -160,3 +291,11 @@ def forward(config, w, tokens):
     logits = linear(w["head"], rms_norm(x, w["final.norm"], eps))
     cap = config["logit_softcap"]
     return cap * np.tanh(logits / cap), np.stack(streams)
+
+
+FORWARD = {"Vifivik": forward_vifivik, "Lanedra": forward_lanedra}
+
+
+def forward(config, w, tokens):
+    """(logits [T, vocab], residual streams [layers, T, width])"""
+    return FORWARD[config["architecture"]](config, w, tokens)

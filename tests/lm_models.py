@@ -33,14 +33,80 @@ def latent(heads, dim, rot, rank, vdim, scale, base=10000.0, kv_from=None):
     return "latent_attention", m
 
 
+def delta(heads, kv_heads, dim, vdim, conv):
+    return "delta", dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, conv=conv)
+
+
+def yarn(factor, original, fast=32.0, slow=1.0):
+    return dict(factor=factor, original=original, fast=fast, slow=slow)
+
+
+def diff_attention(heads, kv_heads, dim, vdim, window, rot_dims=None, base=10000.0, scaling=None, diff=0.4, scale=None, kv_from=None):
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, mask=dict(size=window), diff=diff,
+             scale=1.3 * dim ** -0.5 if scale is None else scale, rot=dict(base=base, dims=dim // 2 * 2 if rot_dims is None else rot_dims))
+    if scaling is not None:
+        m["rot"]["scaling"] = scaling
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return "attention", m
+
+
+def _layers(layers, ff):
+    return [{"type": t, "mixer": copy.deepcopy(m), "mlp": None if f is None else {"kind": "dense", "ff": f}}
+            for (t, m), f in zip(layers, ff)]
+
+
 def config(width, vocab, layers, ff, eps=1e-5, softcap=20.0):
     """layers: list of (type, mixer); ff: one size per layer, None for no feed-forward."""
     return {"architecture": "Vifivik", "width": width, "vocab": vocab, "norm": {"eps": eps}, "logit_softcap": softcap,
-            "layers": [{"type": t, "mixer": copy.deepcopy(m), "mlp": None if f is None else {"kind": "dense", "ff": f}}
-                       for (t, m), f in zip(layers, ff)]}
+            "layers": _layers(layers, ff)}
+
+
+def lanedra(width, vocab, layers, ff, eps=1e-5, scale=1.7):
+    return {"architecture": "Lanedra", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": scale},
+            "layers": _layers(layers, ff)}
+
+
+def lanedra_tensors(cfg, seed):
+    rng = np.random.default_rng(seed)
+    W, V = cfg["width"], cfg["vocab"]
+
+    def mat(n, k, gain=1.0):
+        return rng.standard_normal((n, k)) * gain / np.sqrt(k)
+
+    def offsets(n, mean=0.0):
+        return mean + rng.uniform(-0.3, 0.3, n)
+
+    w = {"embed": rng.standard_normal((V, W)), "head": mat(V, W, 3.0), "final.norm": offsets(W)}
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        q = p + "mix."
+        H, G, D, Vd = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        w[p + "norm1"], w[p + "norm1b"] = offsets(W), offsets(W, -0.2)
+        if L["type"] == "delta":
+            for n, rows in (("q", G * D), ("k", G * D), ("v", H * Vd)):
+                w[q + n] = mat(rows, W)
+                w[q + n + ".conv"] = rng.standard_normal((rows, m["conv"])) * 0.6
+            w[q + "b"], w[q + "a"], w[q + "g"] = mat(H, W, 2.0), mat(H, W), mat(H * Vd, W)
+            w[q + "A_log"], w[q + "dt_bias"] = np.log(rng.uniform(0.5, 8.0, H)), rng.uniform(-5.0, 0.0, H)
+            w[q + "norm"] = rng.uniform(0.6, 1.4, Vd)
+        else:
+            w[q + "q"] = mat(H * 2 * D, W, 1.5)
+            if "kv_from" not in m:
+                w[q + "k"], w[q + "v"] = mat(G * 2 * D, W, 1.5), mat(G * Vd, W)
+            for n in ("lq1", "lk1", "lq2", "lk2"):
+                w[q + n] = rng.standard_normal(D) * 0.6 * D ** -0.25
+        w[q + "o"] = mat(W, H * Vd)
+        if L["mlp"] is not None:
+            w[p + "norm2"], w[p + "norm2b"] = offsets(W), offsets(W, -0.2)
+            w[p + "mlp.gate"], w[p + "mlp.up"] = mat(L["mlp"]["ff"], W), mat(L["mlp"]["ff"], W)
+            w[p + "mlp.down"] = mat(W, L["mlp"]["ff"])
+    return w
 
 
 def tensors(cfg, seed):
+    if cfg["architecture"] == "Lanedra":
+        return lanedra_tensors(cfg, seed)
     rng = np.random.default_rng(seed)
     W, V = cfg["width"], cfg["vocab"]
 
@@ -198,3 +264,71 @@ def needle_tokens(length, key_at, query_at, seed=0):
     tok[list(np.atleast_1d(key_at))] = KEY
     tok[list(np.atleast_1d(query_at))] = QUERY
     return tok
+
+
+# ------------------------------------------------------------------------------------------- Lanedra
+LANEDRA = {   # one mixer each
+    "delta": lambda: lanedra(60, 83, [delta(6, 3, 20, 28, 4)], [None]),
+    "delta_no_window": lambda: lanedra(52, 64, [delta(5, 1, 33, 12, 1)], [36], eps=1e-3, scale=0.4),
+    "delta_own_keys": lambda: lanedra(40, 50, [delta(4, 4, 72, 40, 2)], [None]),
+    "delta_wide_state": lambda: lanedra(64, 70, [delta(4, 2, 200, 72, 3)], [None]),
+    "delta_very_wide_state": lambda: lanedra(64, 70, [delta(2, 1, 300, 33, 3)], [None]),
+    "delta_many_heads": lambda: lanedra(48, 64, [delta(80, 16, 24, 40, 7)], [None]),
+    "delta_many_wide_heads": lambda: lanedra(48, 64, [delta(78, 39, 136, 36, 2)], [None]),
+    "diff": lambda: lanedra(56, 79, [diff_attention(6, 3, 12, 20, 9)], [None]),
+    "diff_itself_only": lambda: lanedra(44, 60, [diff_attention(3, 1, 16, 24, 1, rot_dims=8)], [28]),
+    "diff_whole_context": lambda: lanedra(48, 64, [diff_attention(4, 4, 20, 36, 100000, rot_dims=0, diff=0.0)], [None]),
+    "diff_scaled_rotation": lambda: lanedra(72, 90, [diff_attention(4, 2, 24, 32, 64, base=700.0, scaling=yarn(6.0, 48, 5.0, 0.4))], [40], scale=1.0),
+    "diff_partly_rotated": lambda: lanedra(72, 90, [diff_attention(4, 2, 40, 24, 33, rot_dims=16, base=50.0, scaling=yarn(3.0, 64))], [None], eps=1e-2),
+    "diff_two_head_tiles": lambda: lanedra(64, 64, [diff_attention(20, 2, 9, 13, 50, rot_dims=6, diff=0.8)], [None]),
+    "diff_mid": lambda: lanedra(48, 64, [diff_attention(3, 1, 100, 92, 70)], [None]),
+    "diff_wide": lambda: lanedra(48, 64, [diff_attention(2, 1, 72, 150, 40, rot_dims=32)], [None]),
+    "diff_very_wide": lambda: lanedra(48, 64, [diff_attention(2, 2, 40, 264, 45)], [None]),
+    "diff_huge_keys": lambda: lanedra(48, 64, [diff_attention(2, 1, 520, 24, 45, rot_dims=100)], [None]),
+}
+
+
+def lanedra_mixed():
+    """Every branch together: order of layers, shared caches under other windows and constants, layers without feed-forward."""
+    s = yarn(4.0, 96, 8.0, 0.7)
+    return lanedra(88, 131, [
+        diff_attention(6, 2, 20, 28, 24, base=5000.0, scaling=s),
+        delta(4, 2, 24, 20, 4),
+        diff_attention(6, 2, 20, 28, 57, base=5000.0, scaling=s, kv_from=0, diff=0.2, scale=0.35),
+        delta(3, 3, 36, 44, 2),
+        diff_attention(3, 3, 28, 12, 31, rot_dims=20, base=777.0, diff=0.7),
+        diff_attention(6, 2, 20, 28, 11, base=5000.0, scaling=s, kv_from=0),
+        delta(5, 1, 12, 60, 5)],
+        [52, None, None, 68, 33, 40, 24], eps=2e-6, scale=2.5)
+
+
+def window_needle(root, window, second=False, group=1, dim=24):
+    """One attention layer in which token QUERY finds token KEY, through dimensions that are not rotated, with a score far above
+    all others in one of the maps, wherever KEY stands inside the window."""
+    kv, rot = 2, 8
+    cfg = lanedra(64, 60, [diff_attention(kv * group, kv, dim, 40, window, rot_dims=rot, base=100.0, diff=0.3)], [None])
+    w = lanedra_tensors(cfg, 78)
+    w["l0.norm1b"] = w["l0.norm1b"] + 2.0
+    m = cfg["layers"][0]["mixer"]
+    h = plain.offset_norm(w["embed"] * cfg["embedding"]["scale"], w["l0.norm1"], cfg["norm"]["eps"])
+    key = (w["l0.mix.k"] @ h[KEY]).reshape(kv, 2, dim)[..., rot:]
+    q = w["l0.mix.q"].reshape(kv * group, 2, dim, -1)
+    for head in range(kv * group):
+        k = key[head // group, int(second)]
+        q[head, int(second), rot:] += np.outer(k * (30.0 / m["scale"] / (k @ k)), h[QUERY] / (h[QUERY] @ h[QUERY]))
+    return Model(root, cfg, weights=w)
+
+
+def memory_model(root, conv=3, dim=20):
+    """One delta layer without noticeable decay that writes at token KEY and next to nothing elsewhere: what stands in its state
+    shows at every later token."""
+    cfg = lanedra(64, 60, [delta(4, 2, dim, 24, conv)], [None])
+    w = lanedra_tensors(cfg, 79)
+    u = np.full(64, 64 ** -0.5)
+    w["embed"] = w["embed"] - np.outer(w["embed"] @ u, u) + 10.0 * u
+    w["embed"][KEY] -= 20.0 * u
+    w["l0.norm1"] = np.zeros(64)
+    w["l0.mix.b"] = np.tile(-1.3 * u, (4, 1))
+    w["l0.mix.A_log"], w["l0.mix.dt_bias"] = np.full(4, -6.0), np.full(4, -4.0)
+    w["l0.mix.a"] = w["l0.mix.a"] * 0.1
+    return Model(root, cfg, weights=w)
