@@ -897,7 +897,8 @@ def run_attention_only(args):
 
 def run_layered(spec):
     """Prefill and decode throughput of the config.json model, the roofline fraction of each of its kernels, and the same for
-    the INT4 decode model of that width (which takes prompts token by token: its decode step is its prefill)."""
+    another model of that width: the INT4 decode model (which takes prompts token by token: its decode step is its prefill)
+    beside Vifivik, Vifivik beside Lanedra."""
     import torch
 
     from blackwell_b200 import bench_layered as bl
@@ -909,16 +910,24 @@ def run_layered(spec):
     bf16 = int8_tensor_peak_tops()[0] / 2
     sampler = ClockSampler(0)
     sampler.start()
+    lanedra = size.startswith("lanedra-")
+    sizes = shapes.VIFIVIK_BENCH[size.removeprefix("lanedra-")]
+    cfg = shapes.LANEDRA_BENCH[size.removeprefix("lanedra-")] if lanedra else sizes[0]
     out = {"option": "layered", "size": size, "hbm_gbs": peak, "bf16_tflops": bf16, "peak_kind": kind, "data": "random weights",
            "l2": "every timed pass reads more than L2 holds, or rotates over buffers larger than L2"}
     if part in ("", "model"):
-        out["model"] = bl.model_records(peak, size)
-    if part in ("", "int4"):
-        shape = shapes.VIFIVIK_BENCH[size][1]
-        out["int4"] = [run_decode(shape, b, 2048, 20, dev) for b in (1, 8, 32, 64)]
+        out["model"] = bl.model_records(peak, cfg)
+        if lanedra:
+            out["vifivik"] = bl.model_records(peak, sizes[0])
+    if part in ("", "int4") and not lanedra:
+        out["int4"] = [run_decode(sizes[1], b, 2048, 20, dev) for b in (1, 8, 32, 64)]
     if part in ("", "kernels"):
-        out["kernels"] = bl.linear_records(peak, bf16, size) + bl.recurrence_records(peak, bf16, size) + bl.latent_records(peak, bf16, size)
-    if part in ("", "int4kernels"):
+        out["kernels"] = bl.recurrence_records(peak, bf16, cfg) + (bl.diff_records if lanedra else bl.latent_records)(peak, bf16, cfg)
+        if lanedra:
+            out["vifivik_kernels"] = bl.recurrence_records(peak, bf16, sizes[0]) + bl.latent_records(peak, bf16, sizes[0])
+    if part in ("", "kernels", "linear"):
+        out["linear"] = bl.linear_records(peak, bf16, cfg)
+    if part in ("", "int4kernels") and not lanedra:
         out["int4_kernels"] = {"M%d" % m: per_matrix_times(dev, m) for m in (1, 8, 64)}
         out["int4_attention"] = attention_records(dev)
     out["clocks"] = sampler.stop()
@@ -1002,8 +1011,9 @@ def main():
                     "step is timed as the mean of as many passes as that needs); 0 for profiling runs")
     ap.add_argument("--timeline", default=None, help="diagnostic: per-phase timeline of the small-batch kernel on one "
                     "matrix of the set, NAME[:f16|i8]; needs a library built with -DBW_GEMV_TIMELINE")
-    ap.add_argument("--layered", default=None, help="config.json models (Vifivik layers, random weights) beside the INT4 decode "
-                    "model of the same width: SIZE[:model|kernels|int4|int4kernels], SIZE = 2k or 4k; prints its own JSON line")
+    ap.add_argument("--layered", default=None, help="config.json models (random weights): Vifivik beside the INT4 decode model of "
+                    "the same width, SIZE[:model|kernels|linear|int4|int4kernels], SIZE = 2k or 4k, or Lanedra beside Vifivik, "
+                    "lanedra-SIZE[:model|kernels|linear]; prints its own JSON line")
     ap.add_argument("--tune", default=None, help="profiling aid: comma list of key=value for bw_set_tuning")
     args = ap.parse_args()
     global _ONLY

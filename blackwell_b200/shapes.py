@@ -77,8 +77,23 @@ def vifivik_config(width: int, ff: int, vocab: int, layers: int, head_scale: int
     return {"architecture": "Vifivik", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "logit_softcap": 25.0, "layers": out}
 
 
+def lanedra_config(width: int, ff: int, vocab: int, layers: int, head_scale: int, window: int = 1024) -> dict:
+    """A Lanedra configuration of the same width, depth, feed-forward and vocabulary: the pattern delta, attention, attention on
+    that cache, delta."""
+    delta = {"heads": 32 * head_scale, "kv_heads": 16 * head_scale, "dim": 128, "vdim": 128, "conv": 4}
+    attn = {"heads": 16 * head_scale, "kv_heads": 4 * head_scale, "dim": 64, "vdim": 128, "diff": 0.5, "scale": 64 ** -0.5, "mask": {"size": window},
+            "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    out = []
+    for i in range(layers):
+        kind, mixer = [("delta", delta), ("attention", attn), ("attention", {**attn, "kv_from": i - 1}), ("delta", delta)][i % 4]
+        out.append({"type": kind, "mixer": dict(mixer), "mlp": {"kind": "dense", "ff": ff}})
+    return {"architecture": "Lanedra", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "layers": out}
+
+
 # name -> (config.json model, the INT4 decode model of the same width, feed-forward size, layer count and vocabulary)
 VIFIVIK_BENCH = {
     "2k": (vifivik_config(2048, 5632, 32768, 8, 1), ModelShape("int4-2k", 8, 2048, 5632, 16, 4, 128, 32768)),
     "4k": (vifivik_config(4096, 12288, 65536, 8, 2), ModelShape("int4-4k", 8, 4096, 12288, 32, 8, 128, 65536)),
 }
+# the same sizes as Lanedra models
+LANEDRA_BENCH = {"2k": lanedra_config(2048, 5632, 32768, 8, 1), "4k": lanedra_config(4096, 12288, 65536, 8, 2)}

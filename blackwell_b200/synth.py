@@ -90,7 +90,22 @@ def write_random_model(directory: str, cfg: dict, seed: int = 0, device="cuda") 
         p, m = f"l{i}.", L["mixer"]
         q, H, vd = p + "mix.", m["heads"], m["vdim"]
         shapes[p + "norm1"] = (W,)
-        if L["type"] == "mamba2":
+        if cfg["architecture"] == "Lanedra":
+            shapes[p + "norm1b"] = (W,)
+            if L["mlp"]:
+                shapes[p + "norm2b"] = (W,)
+        if L["type"] == "delta":
+            D, G = m["dim"], m["kv_heads"]
+            for n, rows in (("q", G * D), ("k", G * D), ("v", H * vd)):
+                shapes.update({q + n: (rows, W), q + n + ".conv": (rows, m["conv"])})
+            shapes.update({q + "a": (H, W), q + "b": (H, W), q + "g": (H * vd, W), q + "A_log": (H,), q + "dt_bias": (H,), q + "norm": (vd,)})
+        elif L["type"] == "attention":
+            D, G = m["dim"], m["kv_heads"]
+            shapes[q + "q"] = (H * 2 * D, W)
+            if "kv_from" not in m:
+                shapes.update({q + "k": (G * 2 * D, W), q + "v": (G * vd, W)})
+            shapes.update({q + n: (D,) for n in ("lq1", "lk1", "lq2", "lk2")})
+        elif L["type"] == "mamba2":
             inner, gn = H * vd, m["groups"] * m["state"]
             shapes.update({q + "in": (2 * inner + 2 * gn + H, W), q + "conv": (inner + 2 * gn, m["conv"]), q + "conv.b": (inner + 2 * gn,),
                            q + "dt_bias": (H,), q + "A_log": (H,), q + "D": (H,), q + "norm": (inner,)})
@@ -125,8 +140,11 @@ def write_random_model(directory: str, cfg: dict, seed: int = 0, device="cuda") 
             t = torch.randn(shape, generator=gen, device=device)
             if len(shape) == 2 and name != "embed":
                 t *= shape[1] ** -0.5
-            elif name.endswith(("norm", "norm1", "norm2")):
-                t = 1.0 + 0.1 * t
+            elif name.endswith(("norm", "norm1", "norm2", "norm1b", "norm2b")):
+                around_zero = cfg["architecture"] == "Lanedra" and not name.endswith("mix.norm")
+                t = (0.0 if around_zero else 1.0) + 0.1 * t
+            elif name.endswith((".lq1", ".lk1", ".lq2", ".lk2")):
+                t *= 0.1
             elif name.endswith("dt_bias"):
                 t = t - 4.0
             f.write(t.to(torch.bfloat16).view(torch.int16).cpu().numpy().tobytes())

@@ -280,7 +280,7 @@ LANEDRA = {   # one mixer each
     "diff_whole_context": lambda: lanedra(48, 64, [diff_attention(4, 4, 20, 36, 100000, rot_dims=0, diff=0.0)], [None]),
     "diff_scaled_rotation": lambda: lanedra(72, 90, [diff_attention(4, 2, 24, 32, 64, base=700.0, scaling=yarn(6.0, 48, 5.0, 0.4))], [40], scale=1.0),
     "diff_partly_rotated": lambda: lanedra(72, 90, [diff_attention(4, 2, 40, 24, 33, rot_dims=16, base=50.0, scaling=yarn(3.0, 64))], [None], eps=1e-2),
-    "diff_two_head_tiles": lambda: lanedra(64, 64, [diff_attention(20, 2, 9, 13, 50, rot_dims=6, diff=0.8)], [None]),
+    "diff_two_head_tiles": lambda: lanedra(64, 64, [diff_attention(20, 2, 9, 13, 50, rot_dims=6, diff=0.6)], [None]),
     "diff_mid": lambda: lanedra(48, 64, [diff_attention(3, 1, 100, 92, 70)], [None]),
     "diff_wide": lambda: lanedra(48, 64, [diff_attention(2, 1, 72, 150, 40, rot_dims=32)], [None]),
     "diff_very_wide": lambda: lanedra(48, 64, [diff_attention(2, 2, 40, 264, 45)], [None]),
