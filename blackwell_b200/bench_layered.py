@@ -27,7 +27,7 @@ class RecurrenceArgs(C.Structure):
 
 class DiffArgs(C.Structure):
     _fields_ = ([(n, C.c_int) for n in ("heads", "kv_heads", "dim", "V", "window", "rot_dims")] + [("cs", C.c_void_p), ("max_seq", C.c_int)] +
-                [(n, C.c_float) for n in ("scale", "lam", "out_scale", "eps")] + [("cache", C.c_void_p), ("cap", C.c_int), ("q", C.c_void_p),
+                [(n, C.c_float) for n in ("scale", "lam", "out_scale", "eps")] + [("cache", C.c_void_p), ("cap", C.c_int), ("slots", C.c_int), ("q", C.c_void_p),
                 ("k", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_long), ("out", C.c_void_p), ("ldout", C.c_long), ("splits", C.c_int)])
 
 
@@ -176,7 +176,7 @@ def diff_records(peak, bf16_peak, cfg):
         ids = torch.arange(slots, device="cuda", dtype=torch.int32)
         pos = torch.full((slots,), ctx - 1, device="cuda", dtype=torch.int32)
         pp = proj.data_ptr()
-        a = DiffArgs(H, G, D, V, window, rot, cs.data_ptr(), ctx, m["scale"], 0.5, 0.5, 1e-5, cache.data_ptr(), cap, pp, pp + 2 * H * 2 * D,
+        a = DiffArgs(H, G, D, V, window, rot, cs.data_ptr(), ctx, m["scale"], 0.5, 0.5, 1e-5, cache.data_ptr(), cap, slots, pp, pp + 2 * H * 2 * D,
                      pp + 2 * (H + G) * 2 * D, proj.stride(0), o.data_ptr(), H * V, 0)
 
         def run(j):

@@ -5,12 +5,15 @@
 //   diff_prep_kernel     portions and 32-bit mode: rotates the queries in place, writes the new cache rows.
 //   diff_decode_kernel   one token per sequence (bf16): rotation, cache row, attention and combination in one launch.  An MMA
 //                        row tile is eight heads of one key / value head, map 1 in rows 0-7 and map 2 in rows 8-15, so that
-//                        both maps of a head meet in the registers of one thread; each warp streams its own 16-key tiles,
-//                        the context is split over a cluster whose blocks merge through distributed shared memory.
+//                        both maps of a head meet in the registers of one thread; each warp streams its own 16-key tiles
+//                        by TMA, the context is split over a cluster whose blocks merge through distributed shared memory.
 //   diff_flash_kernel    portions (bf16): flash attention with one half of the warps per map, combined through shared memory.
 //   diff_scalar_kernel   32-bit mode and sizes the others do not take.
 // Scores, softmax and sums are fp32; the softmax weights enter the MMA as a bf16 high part plus a bf16 remainder.
 #pragma once
+#include <cuda.h>
+
+#include "gemm_w4a8_tc.cuh"
 #include "lm_device.cuh"
 #include "lm_ops.h"
 
@@ -175,145 +178,155 @@ __global__ void __launch_bounds__(256) diff_scalar_kernel(const DiffAttnArgs a, 
 }
 
 // ------------------------------------------------------------------------------------------ decode
-constexpr int kDiffWarps = 4;
-constexpr int kDiffTile = 16;    // keys per tile of a warp
-struct DiffDecodeSmem {          // queries, new cache entry, stats of the warps and of the block, tiles (later partial outputs)
-    int qrow, row, q_off, new_off, st_off, tile_off, tile, total;
-    __host__ __device__ DiffDecodeSmem(int dim, int V, int VT, int stages) {
-        const int n16 = diff_row(dim, V) / 8;
-        row = (n16 | 1) * 16;    // odd multiple of 16 bytes: conflict-free ldmatrix
+constexpr int kDiffTile = 16;    // positions per tile of a warp, from a multiple of 16 on
+struct DiffDecodeSmem {          // queries, new cache entry, stats, barriers, then the warps' tiles (later their partial outputs)
+    int qrow, boxes, tile, new_off, st_off, bar_off, ring_off, total;   // a tile: boxes of 16 rows x 64 columns, swizzled
+    __host__ __device__ DiffDecodeSmem(int dim, int V, int VT, int warps, int stages) {
+        boxes = (diff_row(dim, V) + 63) / 64;
+        tile = boxes * kDiffTile * 128;
         qrow = pad16(dim) * 2 + 16;
-        q_off = 0;
         new_off = 16 * qrow;
-        st_off = new_off + n16 * 16;
-        tile_off = st_off + (kDiffWarps + 1) * 16 * 8;
-        tile = kDiffTile * row;
-        const int ring = kDiffWarps * stages * tile + 32, part = kDiffWarps * 16 * VT * 8 * 4;   // a value fragment may read 16 bytes past a row
-        total = tile_off + (ring > part ? ring : part);
+        st_off = new_off + boxes * 128;                // [warps][16] maximum, sum; [warps][16] weights; the block's [16] maximum, sum
+        bar_off = st_off + warps * 16 * 12 + 16 * 8;
+        ring_off = (bar_off + warps * stages * 8 + 1023) & ~1023;
+        const int ring = warps * stages * tile + 2048, part = warps * 16 * VT * 8 * 4;   // a value fragment may start one box past the tile
+        total = 1024 + ring_off + (ring > part ? ring : part);   // 1024: alignment of the base
     }
 };
 
-// Block (split, key / value head and eight of its query heads, row).  KS: 16-wide query steps per map; VT: value columns / 8.
-template <int KS, int VT>
-__global__ void __launch_bounds__(kDiffWarps * 32) diff_decode_kernel(const DiffAttnArgs a, const Rows r, int stages) {
-    extern __shared__ __align__(16) unsigned char smem[];
-    const DiffDecodeSmem L(a.dim, a.V, VT, stages);
+// Block (split, key / value head and eight of its query heads, row); WARPS warps, each with tiles and softmax state of its own.
+// KS: 16-wide query steps per map; VT: value columns / 8.
+template <int KS, int VT, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32) diff_decode_kernel(const __grid_constant__ CUtensorMap map, const DiffAttnArgs a, const Rows r,
+                                                                 int stages, int* status) {
+    extern __shared__ unsigned char smem_raw[];
+    unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+    const DiffDecodeSmem L(a.dim, a.V, VT, WARPS, stages);
     const int D8 = pad8(a.dim), D16 = pad16(a.dim), V8 = pad8(a.V), seg = diff_row(a.dim, a.V), group = a.heads / a.kv_heads;
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, q4 = lane & 3;
     const int htiles = (group + 7) / 8, kvh = blockIdx.y / htiles, h0 = (blockIdx.y - kvh * htiles) * 8, nh = min(8, group - h0);
     const int split = blockIdx.x, row = blockIdx.z, half = a.rot_dims / 2;
-    const uint32_t sb = smem_u32(smem);
-    float2* stats = reinterpret_cast<float2*>(smem + L.st_off);   // [warp][16], then the block's [16]: maximum, sum
+    const uint32_t sb = smem_u32(smem), bars = sb + L.bar_off + warp * stages * 8, ring = sb + L.ring_off + warp * stages * L.tile;
+    float2* stats = reinterpret_cast<float2*>(smem + L.st_off);
+    float* weights = reinterpret_cast<float*>(stats + WARPS * 16);
+    float2* block_stats = reinterpret_cast<float2*>(weights + WARPS * 16);
+    if (lane == 0) {
+        for (int i = 0; i < stages; ++i) mbar_init(bars + 8 * i, 1);
+        mbar_fence_init();
+    }
+    __syncwarp();
     pdl_trigger();
     pdl_wait();
     const int slot = r.slot_of(row), pos = min(r.pos_of(row), a.max_seq - 1);
     if (slot < 0) return;                                         // the whole cluster
-    const int k0 = first_key(a, pos), n = pos + 1 - k0, ring0 = k0 % a.cap;
-    const int tiles = (n + kDiffTile - 1) / kDiffTile, per = (tiles + a.splits - 1) / a.splits;
-    const int t0 = split * per, t1 = min(tiles, t0 + per);
-    const long ldc = (long)a.kv_heads * seg;
-    bf16* cache = static_cast<bf16*>(a.cache) + (long)slot * a.cap * ldc + kvh * seg;
-    const int fresh = a.k ? n - 1 : n;                            // this position comes from the projection, not from the cache
-    const RowWalk walk(lane, 32, seg / 8);
-    const uint32_t ring = sb + L.tile_off + warp * stages * L.tile;
-    auto issue = [&](int tile, int buf) {
-        if (tile < t1) {
-            for (RowWalk w = walk; w.row < kDiffTile; w.next()) {
-                const int j = tile * kDiffTile + w.row;
-                int i = ring0 + j;
-                if (i >= a.cap) i -= a.cap;
-                cp_async16z(ring + buf * L.tile + w.row * L.row + w.col * 16, j < fresh ? cache + i * ldc + w.col * 8 : cache, j < fresh);
-            }
-        }
-        cp_async_commit();
+    const int k0 = first_key(a, pos), tile0 = k0 / kDiffTile, tiles = pos / kDiffTile - tile0 + 1, per = (tiles + a.splits - 1) / a.splits;
+    const int t0 = tile0 + split * per, t1 = min(tile0 + tiles, t0 + per);
+    const int fresh = a.k ? pos - 1 : pos;                        // last position that comes from the cache
+    int waited = 0, issued = 0;
+    auto issue = [&](int tile) {   // lane 0
+        const int s = issued % stages, y = slot * a.cap + (int)((long)tile * kDiffTile % a.cap);
+        mbar_expect_tx(bars + 8 * s, L.tile);
+        for (int b = 0; b < L.boxes; ++b) tc::tma_load_2d(ring + s * L.tile + b * kDiffTile * 128, &map, kvh * seg + b * 64, y, bars + 8 * s);
     };
-    for (int s = 0; s < stages - 1; ++s) issue(t0 + warp + kDiffWarps * s, s);
+    int next = t0 + warp;
+    for (; issued < stages && next < t1; next += WARPS, ++issued)
+        if (lane == 0) issue(next);
     // rotated queries: row = map * 8 + head
     const float2* cs = a.cs + (long)pos * half;
-    for (int i = t; i < 16 * D16; i += kDiffWarps * 32) {
+#pragma unroll 4
+    for (int i = t; i < 16 * D16; i += WARPS * 32) {
         const int qr = i / D16, d = i - qr * D16, hh = qr & 7;
         float v = 0.f;
         if (hh < nh && d < D8) {
             const bf16* q = static_cast<const bf16*>(a.q) + (long)row * a.ld + (2L * (kvh * group + h0 + hh) + (qr >> 3)) * D8;
             v = rot_half_elem(q, d, a.rot_dims, cs);
         }
-        *reinterpret_cast<bf16*>(smem + L.q_off + qr * L.qrow + d * 2) = __float2bfloat16_rn(v);
+        *reinterpret_cast<bf16*>(smem + qr * L.qrow + d * 2) = __float2bfloat16_rn(v);
     }
-    if (a.k && t1 == tiles && t0 < t1) {   // the newest position's entry
+    if (a.k && t1 == tile0 + tiles && t0 < t1) {   // the newest position's entry
         const bf16* k = static_cast<const bf16*>(a.k) + (long)row * a.ld + 2L * kvh * D8;
         const bf16* v = static_cast<const bf16*>(a.v) + (long)row * a.ld + kvh * V8;
-        bf16* entry = cache + (long)(pos % a.cap) * ldc;
-        for (int i = t; i < seg; i += kDiffWarps * 32) {
-            const bf16 x = i < 2 * D8 ? __float2bfloat16_rn(rot_half_elem(k + (i < D8 ? 0 : D8), i < D8 ? i : i - D8, a.rot_dims, cs)) : v[i - 2 * D8];
+        bf16* entry = static_cast<bf16*>(a.cache) + (((long)slot * a.cap + pos % a.cap) * a.kv_heads + kvh) * seg;
+        for (int i = t; i < L.boxes * 64; i += WARPS * 32) {
+            bf16 x = __float2bfloat16_rn(0.f);
+            if (i < 2 * D8) x = __float2bfloat16_rn(rot_half_elem(k + (i < D8 ? 0 : D8), i < D8 ? i : i - D8, a.rot_dims, cs));
+            else if (i < seg) x = v[i - 2 * D8];
             *reinterpret_cast<bf16*>(smem + L.new_off + i * 2) = x;
-            if (h0 == 0) entry[i] = x;
+            if (h0 == 0 && i < seg) entry[i] = x;
         }
     }
     __syncthreads();
-    uint32_t qa[KS][2], qb[KS][2];         // map 1: rows 0-7 of the tile, map 2: rows 8-15
+    uint32_t qa[KS][2], qb[KS][2];         // map 1: rows 0-7 of the MMA tile, map 2: rows 8-15
 #pragma unroll
     for (int i = 0; i < KS; ++i)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             const int off = g * L.qrow + (i * 16 + e * 8 + 2 * q4) * 2;
-            qa[i][e] = i * 16 < D16 ? *reinterpret_cast<const uint32_t*>(smem + L.q_off + off) : 0u;
-            qb[i][e] = i * 16 < D16 ? *reinterpret_cast<const uint32_t*>(smem + L.q_off + 8 * L.qrow + off) : 0u;
+            qa[i][e] = i * 16 < D16 ? *reinterpret_cast<const uint32_t*>(smem + off) : 0u;
+            qb[i][e] = i * 16 < D16 ? *reinterpret_cast<const uint32_t*>(smem + 8 * L.qrow + off) : 0u;
         }
     float O[VT][4] = {};
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {};
     const float sl2 = a.scale * 1.4426950408889634f;   // softmax in base 2
-    int buf = 0;
-    for (int tile = t0 + warp; tile < t1; tile += kDiffWarps) {
-        if (stages == 3) cp_async_wait<1>();
-        else cp_async_wait<0>();
-        __syncwarp();
-        const uint32_t kb = ring + buf * L.tile;
-        const int j0 = tile * kDiffTile;
-        if (fresh < n && tile == tiles - 1) {
-            unsigned char* dst = smem + (kb - sb) + (n - 1 - j0) * L.row;
-            for (int i = lane; i < seg / 8; i += 32) *reinterpret_cast<uint4*>(dst + i * 16) = *reinterpret_cast<const uint4*>(smem + L.new_off + i * 16);
+    CopyWait copied{status};
+    const int krow = (lane & 7) + (lane >> 4) * 8, kc = (lane >> 3) & 1, vrow = lane & 15, vc = lane >> 4;
+    for (int tile = t0 + warp; tile < t1; tile += WARPS) {
+        const int s_ = waited % stages, j0 = tile * kDiffTile;
+        const uint32_t kb = ring + s_ * L.tile;
+        copied(bars + 8 * s_, (waited / stages) & 1);
+        ++waited;
+        if (j0 < k0 || j0 + kDiffTile - 1 > fresh) {   // rows that are not visible become zeros, the newest one its entry
+            unsigned char* dst = smem + (kb - sb);
+            for (int i = lane; i < L.boxes * kDiffTile * 8; i += 32) {
+                const int c = i & 7, rr = (i >> 3) & 15, b = i >> 7, p = j0 + rr;
+                if (p < k0 || p > fresh)
+                    *reinterpret_cast<uint4*>(dst + b * kDiffTile * 128 + rr * 128 + ((c ^ (rr & 7)) << 4)) =
+                        p == pos ? *reinterpret_cast<const uint4*>(smem + L.new_off + b * 128 + c * 16) : make_uint4(0, 0, 0, 0);
+            }
+            fence_proxy_async();   // before the next copy into this buffer
             __syncwarp();
         }
-        issue(tile + kDiffWarps * (stages - 1), buf == 0 ? stages - 1 : buf - 1);
-        float s[2][4] = {};
-        const uint32_t ka = kb + ((lane & 7) + (lane >> 4) * 8) * L.row + ((lane >> 3) & 1) * 16;
+        // 16-byte column chunk `chunk` of tile row `rr`
+        auto at = [&](int rr, int chunk) { return kb + (chunk >> 3) * (kDiffTile * 128) + rr * 128 + (((chunk ^ rr) & 7) << 4); };
+        float s[4][4] = {};            // two accumulators per eight keys: one per map
 #pragma unroll
         for (int i = 0; i < KS; ++i)
             if (i * 16 < D16) {
-                uint32_t b[4];
-                ldsm4(ka + i * 32, b);
+                uint32_t b[4], c[4];
+                ldsm4(at(krow, 2 * i + kc), b);
+                ldsm4(at(krow, D8 / 8 + 2 * i + kc), c);
                 mma_bf16(s[0], qa[i][0], 0u, qa[i][1], 0u, b[0], b[1]);
                 mma_bf16(s[1], qa[i][0], 0u, qa[i][1], 0u, b[2], b[3]);
-                ldsm4(ka + D8 * 2 + i * 32, b);
-                mma_bf16(s[0], 0u, qb[i][0], 0u, qb[i][1], b[0], b[1]);
-                mma_bf16(s[1], 0u, qb[i][0], 0u, qb[i][1], b[2], b[3]);
+                mma_bf16(s[2], 0u, qb[i][0], 0u, qb[i][1], c[0], c[1]);
+                mma_bf16(s[3], 0u, qb[i][0], 0u, qb[i][1], c[2], c[3]);
             }
         float alpha[2];
 #pragma unroll
         for (int p = 0; p < 2; ++p) {
-            float mx = m[p];
+            float mx = m[p], x[4];
 #pragma unroll
             for (int c = 0; c < 2; ++c)
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
-                    float& x = s[c][2 * p + e];
-                    x = j0 + 8 * c + 2 * q4 + e < n ? x * sl2 : -INFINITY;
-                    mx = fmaxf(mx, x);
+                    const int key = j0 + 8 * c + 2 * q4 + e;
+                    x[2 * c + e] = key >= k0 && key <= pos ? s[2 * p + c][2 * p + e] * sl2 : -INFINITY;
+                    mx = fmaxf(mx, x[2 * c + e]);
                 }
             mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));   // finite: the first key of a tile is always visible
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));   // finite: every tile holds a visible position
             alpha[p] = exp2_fast(m[p] - mx);
             m[p] = mx;
             float sum = 0.f;
 #pragma unroll
-            for (int c = 0; c < 2; ++c)
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    float& x = s[c][2 * p + e];
-                    x = exp2_fast(x - mx);
-                    sum += x;
-                }
+            for (int e = 0; e < 4; ++e) {
+                x[e] = exp2_fast(x[e] - mx);
+                sum += x[e];
+            }
             l[p] = l[p] * alpha[p] + sum;
+            s[0][2 * p] = x[0];
+            s[0][2 * p + 1] = x[1];
+            s[1][2 * p] = x[2];
+            s[1][2 * p + 1] = x[3];
         }
         if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
 #pragma unroll
@@ -324,19 +337,25 @@ __global__ void __launch_bounds__(kDiffWarps * 32) diff_decode_kernel(const Diff
         split_bf16(s[0][2], s[0][3], ph[1], pl[1]);
         split_bf16(s[1][0], s[1][1], ph[2], pl[2]);
         split_bf16(s[1][2], s[1][3], ph[3], pl[3]);
-        const uint32_t va = kb + (lane & 15) * L.row + (2 * D8 + (lane >> 4) * 8) * 2;
 #pragma unroll
         for (int j = 0; j < VT; j += 2)
             if (8 * j < V8) {
                 uint32_t v[4];
-                ldsm4t(va + j * 16, v);
+                ldsm4t(at(vrow, D8 / 4 + j + vc), v);
                 mma_bf16(O[j], ph[0], ph[1], ph[2], ph[3], v[0], v[1]);
                 mma_bf16(O[j + 1], ph[0], ph[1], ph[2], ph[3], v[2], v[3]);
                 mma_bf16(O[j], pl[0], pl[1], pl[2], pl[3], v[0], v[1]);
                 mma_bf16(O[j + 1], pl[0], pl[1], pl[2], pl[3], v[2], v[3]);
             }
-        buf = buf + 1 == stages ? 0 : buf + 1;
+        __syncwarp();                  // everybody is done with the buffer
+        if (next < t1) {
+            if (lane == 0) issue(next);
+            ++issued;
+            next += WARPS;
+        }
     }
+    if (copied.dead)                   // gave up: copies still in flight land before the buffers are used for something else
+        for (; waited < issued; ++waited) mbar_wait(bars + 8 * (waited % stages), (waited / stages) & 1);
     // merge: the warps of the block, then the blocks of the cluster
 #pragma unroll
     for (int p = 0; p < 2; ++p) {
@@ -344,65 +363,82 @@ __global__ void __launch_bounds__(kDiffWarps * 32) diff_decode_kernel(const Diff
         l[p] += __shfl_xor_sync(0xffffffffu, l[p], 2);
         if (q4 == 0) stats[warp * 16 + g + 8 * p] = make_float2(m[p], l[p]);
     }
-    cp_async_wait<0>();
     __syncthreads();   // everybody is done with the tiles
-    float* part = reinterpret_cast<float*>(smem + L.tile_off);   // [warp][16][VT * 8]
+    constexpr int kRow = VT * 8;
+    float* part = reinterpret_cast<float*>(smem + L.ring_off);   // [warp][16][kRow]
 #pragma unroll
     for (int j = 0; j < VT; ++j) {
-        float* o = part + (warp * 16 + g) * VT * 8 + 8 * j + 2 * q4;
+        float* o = part + (warp * 16 + g) * kRow + 8 * j + 2 * q4;
         *reinterpret_cast<float2*>(o) = make_float2(O[j][0], O[j][1]);
-        *reinterpret_cast<float2*>(o + 8 * VT * 8) = make_float2(O[j][2], O[j][3]);
+        *reinterpret_cast<float2*>(o + 8 * kRow) = make_float2(O[j][2], O[j][3]);
+    }
+    if (t < 16) {
+        float mx = -INFINITY, sum = 0.f;
+#pragma unroll
+        for (int w = 0; w < WARPS; ++w) mx = fmaxf(mx, stats[w * 16 + t].x);
+#pragma unroll
+        for (int w = 0; w < WARPS; ++w) {
+            const float2 st = stats[w * 16 + t];
+            const float f = st.y > 0.f ? exp2_fast(st.x - mx) : 0.f;   // a warp without tiles has neither
+            weights[w * 16 + t] = f;
+            sum = fmaf(f, st.y, sum);
+        }
+        block_stats[t] = make_float2(mx, sum);
     }
     __syncthreads();
-    for (int i = t; i < 16 * V8; i += kDiffWarps * 32) {
-        const int rr = i / V8, c = i - rr * V8;
-        float mx = -INFINITY;
+    for (int rr = warp; rr < 16; rr += WARPS) {
+        if ((rr & 7) >= nh) continue;
+        for (int c = lane * 4; c < V8; c += 128) {   // these four columns are read and written by this thread alone
+            float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-        for (int w = 0; w < kDiffWarps; ++w) mx = fmaxf(mx, stats[w * 16 + rr].x);
-        float o = 0.f, sum = 0.f;
-#pragma unroll
-        for (int w = 0; w < kDiffWarps; ++w) {
-            const float2 st = stats[w * 16 + rr];
-            const float f = st.y > 0.f ? exp2_fast(st.x - mx) : 0.f;   // a warp without keys has neither
-            sum = fmaf(f, st.y, sum);
-            o = fmaf(f, part[(w * 16 + rr) * VT * 8 + c], o);
+            for (int w = 0; w < WARPS; ++w) {
+                const float f = weights[w * 16 + rr];
+                const float4 x = *reinterpret_cast<const float4*>(part + (w * 16 + rr) * kRow + c);
+                o.x = fmaf(f, x.x, o.x);
+                o.y = fmaf(f, x.y, o.y);
+                o.z = fmaf(f, x.z, o.z);
+                o.w = fmaf(f, x.w, o.w);
+            }
+            *reinterpret_cast<float4*>(part + rr * kRow + c) = o;
         }
-        part[rr * VT * 8 + c] = o;   // this thread alone reads and writes the element
-        if (c == 0) stats[kDiffWarps * 16 + rr] = make_float2(mx, sum);
     }
     cluster_sync_all();
-    const uint32_t st = sb + L.st_off + kDiffWarps * 16 * 8, pb = sb + L.tile_off;
-    for (int hh = split + a.splits * warp; hh < nh; hh += a.splits * kDiffWarps) {
-        float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {};
-        float o[2][(VT + 3) / 4] = {};
-        for (int s = 0; s < a.splits; ++s)
+    constexpr int kCols = (VT + 3) / 4;
+    const uint32_t st = smem_u32(block_stats), pb = sb + L.ring_off;
+    for (int hh = split + a.splits * warp; hh < nh; hh += a.splits * WARPS) {
+        // lane = 4 * block + 2 * map + (maximum, sum)
+        const int src = lane >> 2, p = (lane >> 1) & 1;
+        const float v = src < a.splits ? ld_dsmem(st + (hh + 8 * p) * 8 + (lane & 1) * 4, src) : 0.f;
+        const float lm = __shfl_sync(0xffffffffu, v, lane & ~1), ls = __shfl_sync(0xffffffffu, v, lane | 1);
+        float mx = ls > 0.f ? lm : -INFINITY;   // a block without tiles has neither
 #pragma unroll
-            for (int p = 0; p < 2; ++p) {
-                const int rr = hh + 8 * p;
-                const float ls = ld_dsmem(st + rr * 8 + 4, s);
-                if (ls > 0.f) {
-                    const float ms = ld_dsmem(st + rr * 8, s), mn = fmaxf(mx[p], ms), fo = exp2_fast(mx[p] - mn), fn = exp2_fast(ms - mn);
-                    mx[p] = mn;
-                    sum[p] = sum[p] * fo + ls * fn;
+        for (int o = 4; o < 32; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        float f = ls > 0.f ? exp2_fast(lm - mx) : 0.f, sum = f * ls;
 #pragma unroll
-                    for (int j = 0; j < (VT + 3) / 4; ++j) {
-                        const int c = 32 * j + lane;
-                        if (c < V8) o[p][j] = o[p][j] * fo + ld_dsmem(pb + (rr * VT * 8 + c) * 4, s) * fn;
-                    }
-                }
+        for (int o = 4; o < 32; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        f *= (p ? -a.lambda : 1.0f) / sum;
+        float o[kCols] = {}, ss = 0.f;
+        for (int s = 0; s < a.splits; ++s) {
+            const float f0 = __shfl_sync(0xffffffffu, f, 4 * s), f1 = __shfl_sync(0xffffffffu, f, 4 * s + 2);
+            if (f0 == 0.f && f1 == 0.f) continue;
+            float x[2][kCols];
+#pragma unroll
+            for (int j = 0; j < kCols; ++j) {
+                const int c = min(32 * j + lane, V8 - 1);
+                x[0][j] = ld_dsmem(pb + (hh * kRow + c) * 4, s);
+                x[1][j] = ld_dsmem(pb + ((hh + 8) * kRow + c) * 4, s);
             }
-        const float f0 = 1.0f / sum[0], f1 = a.lambda / sum[1];
-        float ss = 0.f;
 #pragma unroll
-        for (int j = 0; j < (VT + 3) / 4; ++j) {
-            o[0][j] = o[0][j] * f0 - o[1][j] * f1;
-            ss = fmaf(o[0][j], o[0][j], ss);
+            for (int j = 0; j < kCols; ++j) o[j] = fmaf(f0, x[0][j], fmaf(f1, x[1][j], o[j]));
         }
-        const float f = a.out_scale / sqrtf(warp_sum(ss) / (float)a.V + a.eps);
+#pragma unroll
+        for (int j = 0; j < kCols; ++j)
+            if (32 * j + lane < V8) ss = fmaf(o[j], o[j], ss);
+        const float scale = a.out_scale / sqrtf(warp_sum(ss) / (float)a.V + a.eps);
         bf16* out = static_cast<bf16*>(a.out) + (long)row * a.ldout + (kvh * group + h0 + hh) * V8;
 #pragma unroll
-        for (int j = 0; j < (VT + 3) / 4; ++j)
-            if (32 * j + lane < V8) out[32 * j + lane] = __float2bfloat16_rn(o[0][j] * f);
+        for (int j = 0; j < kCols; ++j)
+            if (32 * j + lane < V8) out[32 * j + lane] = __float2bfloat16_rn(o[j] * scale);
     }
     cluster_sync_all();   // nobody leaves while its partial result may still be read
 }

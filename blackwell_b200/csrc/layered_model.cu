@@ -385,7 +385,7 @@ public:
         w->proj = std::max(w->proj, (long)in_.N);
         w->mixed = std::max(w->mixed, (long)mixed_ld());
         if (owner_) return 0;
-        cap_ = reach_ > 0 ? (int)std::min<long>(e.max_seq, (long)reach_ - 1 + e.max_rows) : e.max_seq;
+        cap_ = reach_ > 0 ? (int)std::min<long>(e.max_seq, ((long)reach_ - 1 + e.max_rows + 15) / 16 * 16) : e.max_seq;
         char* c = nullptr;
         BW_TRY(ctx.alloc(&c, (size_t)e.slots * cap_ * s_.kv_heads * lm::diff_row(s_.dim, s_.vdim) * e.elem()));
         cache_ = c;
@@ -395,7 +395,7 @@ public:
         BW_TRY(project(e, w, in_, w.xb, w.ldx, r.T, w.proj_b, in_.N, nullptr, 0, in_.N, st));
         lm::DiffAttnArgs a = base(e);
         const DiffAttention* own = owner_ ? owner_ : this;
-        a.cache = own->cache_; a.cap = own->cap_;
+        a.cache = own->cache_; a.cap = own->cap_; a.slots = e.slots;
         a.q = w.proj_b; a.ld = in_.N;
         if (!owner_) {
             a.k = e.at(w.proj_b, k_);

@@ -1,5 +1,4 @@
 // Host side of the bfloat16 linear kernels: routing by row count, tensor maps, launch shapes.
-#include <cuda.h>
 #include <cuda_runtime.h>
 
 #include <atomic>
@@ -8,36 +7,13 @@
 #include "../../include/blackwell_b200.h"
 #include "host_util.h"
 #include "linear_bf16.cuh"
+#include "tensor_map.h"
 
 namespace bw {
 namespace lm {
 namespace {
 
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-EncodeTiledFn encode_fn() {
-    static EncodeTiledFn fn = nullptr;
-    static std::once_flag once;
-    std::call_once(once, [] {
-        void* p = nullptr;
-        cudaDriverEntryPointQueryResult q;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) == cudaSuccess &&
-            q == cudaDriverEntryPointSuccess)
-            fn = reinterpret_cast<EncodeTiledFn>(p);
-    });
-    return fn;
-}
-
-// Row-major bf16 matrix [rows][cols], boxes of box_rows x 64 columns in the 128-byte swizzle.
-bool make_map(CUtensorMap* m, const void* base, int cols, int rows, long ld, int box_rows) {
-    const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-    const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
-    const cuuint32_t box[2] = {(cuuint32_t)kTcK, (cuuint32_t)box_rows}, es[2] = {1, 1};
-    return encode_fn()(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, es,
-                       CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                       CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
+static_assert(kTcK == kMapCols, "a K block is one box");
 
 template <typename F>
 cudaError_t allow_smem(F kern, std::once_flag (&once)[kMaxDevices], int bytes) {

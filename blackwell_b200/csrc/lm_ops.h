@@ -158,7 +158,7 @@ struct DiffAttnArgs {
     int max_seq;
     float scale, lambda, out_scale, eps;
     void* cache;                      // [slot][cap] rows of kv_heads * diff_row: position p at row p % cap
-    int cap;                          // max_seq, or at least window - 1 + the rows of a call
+    int cap, slots;                   // cap: max_seq, or a multiple of 16 of at least window - 1 + the rows of a call
     void* q;                          // [T][ld], head h's map i at (2 h + i) * pad8(dim), not rotated yet; portions rotate in place
     const void *k, *v;                // [T][ld], laid out the same way / head g at g * pad8(V); NULL: already in the cache
     long ld;

@@ -469,7 +469,7 @@ int bw_latent_attention(const bw_latent_args* a, const bw_rows* rows, int expand
  * (2 h + i) * P8(dim); k likewise over the key / value heads, v: head g at g * P8(V); all before rotation (portions and the 32-bit
  * form rotate q in place); k, v NULL: the positions are in the cache already.  Pairs (i, i + rot_dims / 2) are rotated by
  * cs [max_seq][rot_dims / 2] cos / sin.  cache [slot][cap][kv_heads * (2 * P8(dim) + P8(V))], position p in row p % cap; cap is
- * max_seq or at least window - 1 + rows of one sequence.  dim <= 4096, V <= 2048.  splits: blocks (1, 2, 4, 8) that share the
+ * max_seq, or a multiple of 16 of at least window - 1 + rows of one sequence.  dim <= 4096, V <= 2048.  splits: blocks (1, 2, 4, 8) that share the
  * context of a token step, 0 = automatic. */
 typedef struct bw_diff_attention_args {
     int heads, kv_heads, dim, V, window, rot_dims;
@@ -477,7 +477,7 @@ typedef struct bw_diff_attention_args {
     int max_seq;
     float scale, lambda, out_scale, eps;
     void* cache;
-    int cap;
+    int cap, slots;
     void* q;
     const void *k, *v;
     long ld;

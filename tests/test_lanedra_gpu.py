@@ -254,12 +254,12 @@ class Rows(C.Structure):
 
 class DiffArgs(C.Structure):
     _fields_ = ([(n, C.c_int) for n in ("heads", "kv_heads", "dim", "V", "window", "rot_dims")] + [("cs", C.c_void_p), ("max_seq", C.c_int)] +
-                [(n, C.c_float) for n in ("scale", "lam", "out_scale", "eps")] + [("cache", C.c_void_p), ("cap", C.c_int), ("q", C.c_void_p),
+                [(n, C.c_float) for n in ("scale", "lam", "out_scale", "eps")] + [("cache", C.c_void_p), ("cap", C.c_int), ("slots", C.c_int), ("q", C.c_void_p),
                 ("k", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_long), ("out", C.c_void_p), ("ldout", C.c_long), ("splits", C.c_int)])
 
 
 @pytest.mark.parametrize("splits", [1, 2, 4, 8])
-@pytest.mark.parametrize("window, cap, positions", [(0, 600, [0, 15, 16, 511, 599]), (200, 200, [1, 198, 199, 200, 598]), (37, 61, [36, 37, 60, 61, 597])])
+@pytest.mark.parametrize("window, cap, positions", [(0, 600, [0, 15, 16, 511, 599]), (200, 208, [1, 199, 200, 207, 208, 598]), (37, 48, [36, 37, 47, 48, 49, 597])])
 def test_decode_attention_splits(cuda, window, cap, positions, splits):
     """One token per sequence against the plain formulas for every number of context splits, full and ring caches."""
     import torch
@@ -291,7 +291,7 @@ def test_decode_attention_splits(cuda, window, cap, positions, splits):
                                         slot=torch.arange(B, dtype=torch.int32), pos=torch.tensor(positions, dtype=torch.int32)).items()}
     out = torch.zeros((B, H * V), dtype=torch.bfloat16, device="cuda")
     pp = dev["proj"].data_ptr()
-    a = DiffArgs(H, G, D, V, window, rot, dev["cs"].data_ptr(), max_seq, 0.2, lam, 0.6, 1e-5, dev["cache"].data_ptr(), cap, pp, pp + 2 * H * 2 * D,
+    a = DiffArgs(H, G, D, V, window, rot, dev["cs"].data_ptr(), max_seq, 0.2, lam, 0.6, 1e-5, dev["cache"].data_ptr(), cap, B, pp, pp + 2 * H * 2 * D,
                  pp + 2 * (H + G) * 2 * D, proj.shape[1], out.data_ptr(), H * V, splits)
     r = Rows(B, dev["slot"].data_ptr(), dev["pos"].data_ptr(), 0, 0)
     assert _lib.load().bw_diff_attention(C.byref(a), C.byref(r), 0, None) == 0
@@ -310,8 +310,8 @@ def test_rejected_calls(cuda, tmp_path):
     L = _lib.load()
     one = C.c_void_p(16)
     good = dict(heads=4, kv_heads=2, dim=16, V=16, window=8, rot_dims=8, cs=one, max_seq=64, scale=1.0, lam=0.1, out_scale=1.0, eps=1e-5, cache=one,
-                cap=64, q=one, k=one, v=one, ld=64, out=one, ldout=64, splits=1)
-    for change in (dict(kv_heads=3), dict(rot_dims=18), dict(rot_dims=7), dict(cap=6), dict(ld=63), dict(V=4000), dict(v=None), dict(window=-1)):
+                cap=64, slots=1, q=one, k=one, v=one, ld=64, out=one, ldout=64, splits=1)
+    for change in (dict(kv_heads=3), dict(rot_dims=18), dict(rot_dims=7), dict(cap=6), dict(cap=40), dict(slots=0), dict(ld=63), dict(V=4000), dict(v=None), dict(window=-1)):
         assert L.bw_diff_attention(C.byref(DiffArgs(**{**good, **change})), C.byref(Rows(2, None, None, 0, 0)), 0, None) != 0, change
     m = lm.Model(tmp_path, lm.lanedra_mixed(), 16)
     cfg = json.loads(json.dumps(m.cfg))
