@@ -19,7 +19,12 @@ constexpr int kDeltaMat = kChunk * kChunk * 2;
 constexpr int kDeltaUnit = 4 * kDeltaMat + 4 * kChunk * 4;
 constexpr int kInvRow = kChunk + 4;   // floats of a row of A^T in shared memory
 
-inline __host__ __device__ int delta_prepare_smem(int N) { return 2 * kChunk * (pad16(N) * 2 + 16) + kChunk * kInvRow * 4 + 4 * kChunk * 4; }
+// q and k, whose place T and a factor take over; A^T; the four vectors
+inline __host__ __device__ int delta_prepare_front(int N) {
+    const int qk = 2 * kChunk * (pad16(N) * 2 + 16), inv = kChunk * kInvRow * 4 + 32 * 36 * 4;
+    return qk > inv ? qk : inv;
+}
+inline __host__ __device__ int delta_prepare_smem(int N) { return delta_prepare_front(N) + kChunk * kInvRow * 4 + 4 * kChunk * 4; }
 
 // Block (head, chunk).
 __global__ void __launch_bounds__(256) delta_prepare_kernel(const RecurrenceArgs a, const Rows r) {
@@ -27,7 +32,7 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const RecurrenceArgs
     const int NP = pad16(a.N), N8 = pad8(a.N), qrow = NP * 2 + 16;
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, q4 = lane & 3;
     const int h = blockIdx.x, ch = blockIdx.y, grp = h / (a.heads / a.groups);
-    float* At = reinterpret_cast<float*>(smem + 2 * kChunk * qrow);   // [column of A][row of A]
+    float* At = reinterpret_cast<float*>(smem + delta_prepare_front(a.N));   // [column of A][row of A]
     float *cum = At + kChunk * kInvRow, *beta = cum + kChunk, *rk = beta + kChunk, *rq = rk + kChunk;
     unsigned char* unit = static_cast<unsigned char*>(a.chunk_scratch) + ((long)ch * a.heads + h) * kDeltaUnit;
     const uint32_t qb = smem_u32(smem), kb = qb + kChunk * qrow;
@@ -123,28 +128,81 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const RecurrenceArgs
     }
     for (int i = t; i < 4 * kChunk; i += 256) reinterpret_cast<float*>(unit + 4 * kDeltaMat)[i] = cum[i];
     __syncthreads();
-    // column t of (I + A)^-1 by forward substitution: once x_l is known, its multiples leave the rows below
+    // T = (I + A)^-1: the 16 x 16 blocks on the diagonal by forward substitution, a thread per column, then twice the block
+    // below two inverted ones, T_21 = -T_22 A_21 T_11
+    float *T = reinterpret_cast<float*>(smem), *M = T + kChunk * kInvRow;
+    for (int i = t; i < kChunk * kInvRow / 4; i += 256) reinterpret_cast<float4*>(T)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    __syncthreads();
     if (t < kChunk) {
-        float x[kChunk];
+        const int b0 = t & ~15, j = t & 15;
+        float x[16];
 #pragma unroll
-        for (int i = 0; i < kChunk; ++i) x[i] = i == t ? 1.f : 0.f;
+        for (int i = 0; i < 16; ++i) x[i] = i == j ? 1.f : 0.f;
 #pragma unroll
-        for (int l = 0; l < kChunk; ++l)
+        for (int l = 0; l < 16; ++l)
 #pragma unroll
-            for (int i = (l + 1) / 4 * 4; i < kChunk; i += 4) {   // A is zero on and above the diagonal
-                const float4 v = *reinterpret_cast<const float4*>(At + l * kInvRow + i);
+            for (int i = (l + 1) / 4 * 4; i < 16; i += 4) {   // A is zero on and above the diagonal
+                const float4 v = *reinterpret_cast<const float4*>(At + (b0 + l) * kInvRow + b0 + i);
                 x[i] = fmaf(-v.x, x[l], x[i]);
                 x[i + 1] = fmaf(-v.y, x[l], x[i + 1]);
                 x[i + 2] = fmaf(-v.z, x[l], x[i + 2]);
                 x[i + 3] = fmaf(-v.w, x[l], x[i + 3]);
             }
-        bf16* o = reinterpret_cast<bf16*>(unit) + t;
 #pragma unroll
-        for (int i = 0; i < kChunk; ++i) {
-            const bf16 hi = __float2bfloat16_rn(x[i]);
-            o[i * kChunk] = hi;
-            o[i * kChunk + kDeltaMat / 2] = __float2bfloat16_rn(x[i] - __bfloat162float(hi));
+        for (int i = 0; i < 16; ++i) T[(b0 + i) * kInvRow + t] = x[i];
+    }
+    __syncthreads();
+    {
+        const int b0 = t >> 7 << 5, i = (t >> 3) & 15, j = (t & 7) * 2;
+        float* Mp = M + (t >> 7) * 16 * 20;
+        float2 s = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int l = 0; l < 16; ++l) {
+            const float x = At[(b0 + l) * kInvRow + b0 + 16 + i];
+            const float2 y = *reinterpret_cast<const float2*>(T + (b0 + l) * kInvRow + b0 + j);
+            s.x = fmaf(x, y.x, s.x);
+            s.y = fmaf(x, y.y, s.y);
         }
+        *reinterpret_cast<float2*>(Mp + i * 20 + j) = s;
+        __syncthreads();
+        s = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int l = 0; l < 16; ++l) {
+            const float x = -T[(b0 + 16 + i) * kInvRow + b0 + 16 + l];
+            const float2 y = *reinterpret_cast<const float2*>(Mp + l * 20 + j);
+            s.x = fmaf(x, y.x, s.x);
+            s.y = fmaf(x, y.y, s.y);
+        }
+        *reinterpret_cast<float2*>(T + (b0 + 16 + i) * kInvRow + b0 + j) = s;
+    }
+    __syncthreads();
+    {
+        const int i = t >> 3, j = (t & 7) * 4;
+        auto product = [&](auto left, const float* right, int ld) {
+            float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+            for (int l = 0; l < 32; ++l) {
+                const float x = left(l);
+                const float4 y = *reinterpret_cast<const float4*>(right + l * ld + j);
+                s.x = fmaf(x, y.x, s.x);
+                s.y = fmaf(x, y.y, s.y);
+                s.z = fmaf(x, y.z, s.z);
+                s.w = fmaf(x, y.w, s.w);
+            }
+            return s;
+        };
+        const float4 mt = product([&](int l) { return At[l * kInvRow + 32 + i]; }, T, kInvRow);
+        *reinterpret_cast<float4*>(M + i * 36 + j) = mt;
+        __syncthreads();
+        *reinterpret_cast<float4*>(T + (32 + i) * kInvRow + j) = product([&](int l) { return -T[(32 + i) * kInvRow + 32 + l]; }, M, 36);
+    }
+    __syncthreads();
+    for (int i = t; i < kChunk * kChunk / 2; i += 256) {
+        const float2 x = *reinterpret_cast<const float2*>(T + (i >> 5) * kInvRow + (i & 31) * 2);
+        uint32_t hi, lo;
+        split_bf16(x.x, x.y, hi, lo);
+        reinterpret_cast<uint32_t*>(unit)[i] = hi;
+        reinterpret_cast<uint32_t*>(unit + kDeltaMat)[i] = lo;
     }
 }
 

@@ -122,6 +122,44 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(A* out, long ldout, con
     }
 }
 
+// The same with one group per head and the gate last: a warp per head.
+template <typename A>
+__global__ void __launch_bounds__(256) gated_norm_heads_kernel(A* out, long ldout, const float* o, long ldo, const A* gate, long ldg,
+                                                               const float* w, int heads, int V, float eps) {
+    pdl_trigger();
+    pdl_wait();
+    const int h = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, V8 = pad8(V);
+    if (h >= heads) return;
+    const long r = blockIdx.y;
+    const float* orow = o + r * ldo + h * V8;
+    const A* grow = gate + r * ldg + h * V8;
+    A* dst = out + r * ldout + h * V8;
+    constexpr int kVec = 4;   // first 512 columns in registers
+    float4 x[kVec];
+    float ss = 0.f;
+    auto add = [&](const float4& v) { ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss)))); };
+#pragma unroll
+    for (int j = 0; j < kVec; ++j) {   // columns V .. V8 are zero
+        const int c = j * 128 + lane * 4;
+        x[j] = c < V8 ? *reinterpret_cast<const float4*>(orow + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        add(x[j]);
+    }
+    for (int c = kVec * 128 + lane * 4; c < V8; c += 128) add(*reinterpret_cast<const float4*>(orow + c));
+    const float rms = 1.0f / sqrtf(warp_sum(ss) / (float)V + eps);
+    auto emit = [&](int c, const float4& v) {
+        const float y[4] = {v.x, v.y, v.z, v.w};
+        float z[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) z[e] = c + e < V ? y[e] * silu_f(to_f(grow[c + e])) * rms * (w ? w[(long)h * V + c + e] : 1.f) : 0.f;
+        if constexpr (sizeof(A) == 2) *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack_bf16(z[0], z[1]), pack_bf16(z[2], z[3]));
+        else *reinterpret_cast<float4*>(dst + c) = make_float4(z[0], z[1], z[2], z[3]);
+    };
+#pragma unroll
+    for (int j = 0; j < kVec; ++j)
+        if (j * 128 + lane * 4 < V8) emit(j * 128 + lane * 4, x[j]);
+    for (int c = kVec * 128 + lane * 4; c < V8; c += 128) emit(c, *reinterpret_cast<const float4*>(orow + c));
+}
+
 // Conv channel of a padded column (counted from the start of the convolved part), -1 for padding.
 __device__ __forceinline__ int conv_channel(const ConvArgs& c, int col) {
     const int V8 = pad8(c.V), N8 = pad8(c.N), x_cols = c.heads * V8;
@@ -130,6 +168,16 @@ __device__ __forceinline__ int conv_channel(const ConvArgs& c, int col) {
     return b % N8 < c.N ? c.heads * c.V + (b / N8) * c.N + b % N8 : -1;
 }
 __host__ __device__ __forceinline__ int conv_cols(const ConvArgs& c) { return c.heads * pad8(c.V) + 2 * c.groups * pad8(c.N); }
+
+// Step size (or strength) and log decay of rows [t0, t1) of head h.
+__device__ __forceinline__ void step_sizes(const ConvArgs& c, int h, int t0, int t1) {
+    const float a = -expf(c.A_log[h]), b = c.dt_bias[h];
+    for (int t = t0; t < t1; ++t) {
+        const float dt = softplus_f(c.dt_raw[(long)t * c.ld_dt + h] + b);
+        c.log_decay[(long)t * c.heads + h] = a * dt;
+        c.weight[(long)t * c.heads + h] = c.beta_raw ? sigmoid_f(c.beta_raw[(long)t * c.ld_dt + h]) : dt;
+    }
+}
 
 constexpr int kConvRows = 8;   // rows per block
 
@@ -159,14 +207,68 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const ConvArgs c, const 
             static_cast<A*>(c.out)[(long)t * c.ldo + col] = from_f<A>(silu_f(y));
         }
     } else if (col < cols + c.heads) {
-        const int h = col - cols;
-        const float a = -expf(c.A_log[h]), b = c.dt_bias[h];
-        for (int t = t0; t < t1; ++t) {
-            const float dt = softplus_f(c.dt_raw[(long)t * c.ld_dt + h] + b);
-            c.log_decay[(long)t * c.heads + h] = a * dt;
-            c.weight[(long)t * c.heads + h] = c.beta_raw ? sigmoid_f(c.beta_raw[(long)t * c.ld_dt + h]) : dt;
+        step_sizes(c, col - cols, t0, t1);
+    }
+}
+
+// bf16 prompts and few taps: a thread walks down 16 rows of eight columns (always of one head block) with the last inputs in
+// registers.
+constexpr int kConvWalk = 16;
+template <int TAPS>
+__global__ void __launch_bounds__(128) conv_walk_kernel(const ConvArgs c, const Rows r) {
+    pdl_wait();
+    const int channels = c.heads * c.V + 2 * c.groups * c.N, vecs = conv_cols(c) / 8;
+    const int vec = blockIdx.x * 128 + threadIdx.x, t0 = blockIdx.y * kConvWalk, t1 = min(r.T, t0 + kConvWalk);
+    if (vec >= vecs) {
+        if (vec < vecs + c.heads) step_sizes(c, vec - vecs, t0, t1);
+        return;
+    }
+    const bf16* u = static_cast<const bf16*>(c.u) + c.off + vec * 8;
+    bf16* out = static_cast<bf16*>(c.out) + vec * 8;
+    auto unpack = [](const uint4& v, float (&x)[8]) {
+        const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            x[2 * i] = __uint_as_float(w[i] << 16);
+            x[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
+        }
+    };
+    float w[TAPS][8], bias[8], win[TAPS][8];   // win[i]: the input TAPS - 1 - i rows back
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+        const int ch = conv_channel(c, vec * 8 + e);   // padding columns: zero weights, zero output
+        bias[e] = ch >= 0 && c.bias ? c.bias[ch] : 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j][e] = ch >= 0 ? c.w[ch * TAPS + j] : 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) {
+            const int s = t0 - (TAPS - 1) + j, p = r.pos0 + s;
+            float v = 0.f;
+            if (s >= 0) v = to_f(u[(long)s * c.ldu + e]);
+            else if (p >= 0 && ch >= 0) v = c.ring[((long)r.slot * TAPS + p % TAPS) * channels + ch];
+            win[j][e] = v;
         }
     }
+#pragma unroll 4
+    for (int t = t0; t < t1; ++t) {
+        unpack(*reinterpret_cast<const uint4*>(u + (long)t * c.ldu), win[TAPS - 1]);
+        float y[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            y[e] = bias[e];
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) y[e] = fmaf(w[j][e], win[j][e], y[e]);
+            y[e] = __fdividef(y[e], 1.0f + __expf(-y[e]));
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) win[j][e] = win[j + 1][e];
+        }
+        *reinterpret_cast<uint4*>(out + (long)t * c.ldo) =
+            make_uint4(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]), pack_bf16(y[4], y[5]), pack_bf16(y[6], y[7]));
+    }
+}
+template <int TAPS>
+cudaError_t conv_walk(const ConvArgs& c, const Rows& r, cudaStream_t st) {
+    return launch_pdl(conv_walk_kernel<TAPS>, dim3((conv_cols(c) / 8 + c.heads + 127) / 128, (r.T + kConvWalk - 1) / kConvWalk), dim3(128), 0, st, c, r);
 }
 
 template <typename A>
@@ -218,6 +320,13 @@ cudaError_t gated_norm(void* out, long ldout, const float* o, long ldo, const vo
     if (groups < 1 || (heads * V) % groups != 0) return cudaErrorInvalidValue;
     const dim3 grid(groups, T), block(256);
     count_launch(1);
+    if (groups == heads && !gate_first) {
+        const dim3 by_heads((heads + 7) / 8, T);
+        return f32 ? launch_pdl(gated_norm_heads_kernel<float>, by_heads, block, 0, st, static_cast<float*>(out), ldout, o, ldo,
+                                static_cast<const float*>(gate), ldg, w, heads, V, eps)
+                   : launch_pdl(gated_norm_heads_kernel<bf16>, by_heads, block, 0, st, static_cast<bf16*>(out), ldout, o, ldo,
+                                static_cast<const bf16*>(gate), ldg, w, heads, V, eps);
+    }
     return f32 ? launch_pdl(gated_norm_kernel<float>, grid, block, 0, st, static_cast<float*>(out), ldout, o, ldo,
                             static_cast<const float*>(gate), ldg, w, heads, V, groups, gate_first, eps)
                : launch_pdl(gated_norm_kernel<bf16>, grid, block, 0, st, static_cast<bf16*>(out), ldout, o, ldo,
@@ -228,6 +337,11 @@ cudaError_t conv_silu(const ConvArgs& c, const Rows& r, int f32, cudaStream_t st
     const int n = conv_cols(c) + c.heads;
     const dim3 grid((n + 127) / 128, (r.T + kConvRows - 1) / kConvRows), block(128);
     count_launch(1);
+    if (!f32 && r.T >= kConvWalk) {
+        if (c.taps == 2) return conv_walk<2>(c, r, st);
+        if (c.taps == 3) return conv_walk<3>(c, r, st);
+        if (c.taps == 4) return conv_walk<4>(c, r, st);
+    }
     return f32 ? launch_pdl(conv_silu_kernel<float>, grid, block, 0, st, c, r) : launch_pdl(conv_silu_kernel<bf16>, grid, block, 0, st, c, r);
 }
 
