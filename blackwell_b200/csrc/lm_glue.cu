@@ -3,6 +3,8 @@
 // are read and written as bf16 (serving) or fp32 (32-bit mode).
 #include <cuda_runtime.h>
 
+#include <algorithm>
+
 #include "host_util.h"
 #include "lm_device.cuh"
 #include "lm_ops.h"
@@ -11,86 +13,136 @@ namespace bw {
 namespace lm {
 namespace {
 
-constexpr int kKeep = 8;   // values of a row that a thread of a norm kernel keeps in registers
+// Row kernels: a block per row, VEC neighbouring columns per access (4, or 1 for widths that are not a multiple of 4), the
+// first KEEP vectors of a thread in registers.  Weights are fetched before the kernel waits for its predecessor.
+template <int VEC, int KEEP>
+struct RowVecs {
+    static constexpr int kKeep = KEEP;
+    float v[kKeep][VEC];
+    static __device__ __forceinline__ int col(int j) { return (j * blockDim.x + threadIdx.x) * VEC; }
+    static __device__ __forceinline__ void get(const float* p, float (&x)[VEC]) {
+        if constexpr (VEC == 4) *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(p);
+        else x[0] = p[0];
+    }
+    static __device__ __forceinline__ void put(float* p, const float (&x)[VEC]) {
+        if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = *reinterpret_cast<const float4*>(x);
+        else p[0] = x[0];
+    }
+    static __device__ __forceinline__ void put(bf16* p, const float (&x)[VEC]) {
+        if constexpr (VEC == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]));
+        else p[0] = __float2bfloat16_rn(x[0]);
+    }
+    // p NULL, or beyond the row: `other`
+    __device__ __forceinline__ void load(const float* p, int width, float other) {
+#pragma unroll
+        for (int j = 0; j < kKeep; ++j) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[j][e] = other;
+            if (p && col(j) < width) get(p + col(j), v[j]);
+        }
+    }
+    __device__ __forceinline__ float squares() const {
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < kKeep; ++j)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) s = fmaf(v[j][e], v[j][e], s);
+        return s;
+    }
+    // f(column) for the columns that are not kept
+    template <typename F>
+    static __device__ __forceinline__ void beyond(int width, F f) {
+        for (int i = kKeep * blockDim.x * VEC + threadIdx.x; i < width; i += blockDim.x) f(i);
+    }
+};
 
-// xb = x / rms(x) * next (next NULL: x) for the block's row x, of which keep[] holds the first values.
-template <typename A>
-__device__ __forceinline__ void next_input(A* xb, const float* x, const float* next, const float (&keep)[kKeep], int width, float eps,
-                                           float* buf) {
+// xb = x / rms(x) * next (next NULL: x) for the block's row x, of which `keep` holds the first values, `gain` those of next.
+template <typename A, int VEC, int KEEP>
+__device__ __forceinline__ void next_input(A* xb, const float* x, const float* next, const RowVecs<VEC, KEEP>& keep,
+                                           const RowVecs<VEC, KEEP>& gain, int width, float eps, float* buf) {
+    typedef RowVecs<VEC, KEEP> R;
     float f = 1.f;
     if (next) {
-        float ss = 0.f;
-#pragma unroll
-        for (int j = 0; j < kKeep; ++j) ss = fmaf(keep[j], keep[j], ss);
-        for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
+        float ss = keep.squares();
+        R::beyond(width, [&](int i) { ss = fmaf(x[i], x[i], ss); });
         f = 1.0f / sqrtf(block_sum(ss, buf) / (float)width + eps);
     }
 #pragma unroll
-    for (int j = 0; j < kKeep; ++j) {
-        const int i = j * blockDim.x + threadIdx.x;
-        if (i < width) xb[i] = from_f<A>(next ? keep[j] * f * next[i] : keep[j]);
-    }
-    for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) xb[i] = from_f<A>(next ? x[i] * f * next[i] : x[i]);
+    for (int j = 0; j < R::kKeep; ++j)
+        if (R::col(j) < width) {
+            float v[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[e] = keep.v[j][e] * f * gain.v[j][e];
+            R::put(xb + R::col(j), v);
+        }
+    R::beyond(width, [&](int i) { xb[i] = from_f<A>(x[i] * f * (next ? next[i] : 1.f)); });
 }
 
-template <typename A>
+template <typename A, int VEC, int KEEP>
 __global__ void __launch_bounds__(512) embed_kernel(float* x, A* xb, long ldxb, const bf16* table, long ldt, const int* tokens,
                                                     int width, int vocab, float scale, const float* next, float eps) {
     __shared__ float buf[32];
+    typedef RowVecs<VEC, KEEP> R;
+    R gain, keep;
+    gain.load(next, width, 1.f);
     pdl_trigger();
     pdl_wait();
     const long r = blockIdx.x;
     int tok = tokens[r];
     tok = tok < 0 ? 0 : tok >= vocab ? vocab - 1 : tok;
     const bf16* row = table + (long)tok * ldt;
-    float keep[kKeep];
+    float* xr = x + r * width;
 #pragma unroll
-    for (int j = 0; j < kKeep; ++j) {
-        const int i = j * blockDim.x + threadIdx.x;
-        keep[j] = i < width ? to_f(row[i]) * scale : 0.f;
-        if (i < width) x[r * width + i] = keep[j];
+    for (int j = 0; j < R::kKeep; ++j) {
+        const int c = R::col(j);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) keep.v[j][e] = c < width ? to_f(row[c + e]) * scale : 0.f;
+        if (c < width) R::put(xr + c, keep.v[j]);
     }
-    for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) x[r * width + i] = to_f(row[i]) * scale;
-    next_input<A>(xb + r * ldxb, x + r * width, next, keep, width, eps, buf);
+    R::beyond(width, [&](int i) { xr[i] = to_f(row[i]) * scale; });   // read again by this thread alone
+    next_input<A, VEC, KEEP>(xb + r * ldxb, xr, next, keep, gain, width, eps, buf);
 }
 
 // ADD: x += y / rms(y) * w and xb = the next sublayer's input; otherwise xb = x / rms(x) * w for a listed row.
-template <typename A, bool ADD>
+template <typename A, int VEC, int KEEP, bool ADD>
 __global__ void __launch_bounds__(512) norm_kernel(float* x, A* xb, long ldxb, const float* y, const float* w, const float* next,
                                                    const int* rows, int width, float eps) {
     __shared__ float buf[32];
+    typedef RowVecs<VEC, KEEP> R;
+    R weight, gain, keep, sum;
+    weight.load(w, width, 0.f);
+    if (ADD) gain.load(next, width, 1.f);
     pdl_trigger();
     pdl_wait();
     const int out_row = blockIdx.x;
     const long r = rows ? rows[out_row] : out_row;
-    const float* src = (ADD ? y : x) + r * width;
-    float ss = 0.f;
-    float keep[kKeep];
-#pragma unroll
-    for (int j = 0; j < kKeep; ++j) {
-        const int i = j * blockDim.x + threadIdx.x;
-        keep[j] = i < width ? src[i] : 0.f;
-        ss = fmaf(keep[j], keep[j], ss);
-    }
-    for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) ss = fmaf(src[i], src[i], ss);
+    float* xr = x + r * width;
+    const float* src = ADD ? y + r * width : xr;
+    keep.load(src, width, 0.f);
+    if (ADD) sum.load(xr, width, 0.f);
+    float ss = keep.squares();
+    R::beyond(width, [&](int i) { ss = fmaf(src[i], src[i], ss); });
     const float rms = 1.0f / sqrtf(block_sum(ss, buf) / (float)width + eps);
-    auto emit = [&](int i, float v) {
-        v = v * rms * w[i];
-        if (ADD) {
-            v += x[r * width + i];
-            x[r * width + i] = v;
-        } else {
-            xb[(long)out_row * ldxb + i] = from_f<A>(v);
-        }
-        return v;
-    };
+    A* xo = xb + out_row * ldxb;
 #pragma unroll
-    for (int j = 0; j < kKeep; ++j) {
-        const int i = j * blockDim.x + threadIdx.x;
-        if (i < width) keep[j] = emit(i, keep[j]);
+    for (int j = 0; j < R::kKeep; ++j) {
+        const int c = R::col(j);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            const float v = keep.v[j][e] * rms * weight.v[j][e];
+            keep.v[j][e] = ADD ? sum.v[j][e] + v : v;
+        }
+        if (c < width) {
+            if (ADD) R::put(xr + c, keep.v[j]);
+            else R::put(xo + c, keep.v[j]);
+        }
     }
-    for (int i = kKeep * blockDim.x + threadIdx.x; i < width; i += blockDim.x) emit(i, src[i]);
-    if (ADD) next_input<A>(xb + r * ldxb, x + r * width, next, keep, width, eps, buf);
+    R::beyond(width, [&](int i) {
+        const float v = src[i] * rms * w[i];
+        if (ADD) xr[i] += v;
+        else xo[i] = from_f<A>(v);
+    });
+    if (ADD) next_input<A, VEC, KEEP>(xo, xr, next, keep, gain, width, eps, buf);
 }
 
 template <typename A>
@@ -284,35 +336,59 @@ __global__ void __launch_bounds__(128) conv_ring_kernel(const ConvArgs c, const 
 
 }  // namespace
 
-static int norm_threads(int width) { return width <= 256 ? 64 : width <= 1024 ? 128 : width <= 2048 ? 256 : 512; }
+namespace {
+
+// threads of a row kernel: one access per thread, up to 512
+int row_threads(int width, int vec) { return std::min(512, std::max(64, (width / vec + 31) / 32 * 32)); }
+
+// Calls f<VEC, KEEP>() with the instance for this width.
+template <typename F>
+cudaError_t by_width(int width, F f) {
+    if (width % 4 != 0) return f.template operator()<1, 4>();
+    return width <= 2048 ? f.template operator()<4, 1>() : width <= 4096 ? f.template operator()<4, 2>() : f.template operator()<4, 4>();
+}
+template <typename A>
+struct Embed {
+    float* x; void* xb; long ldxb; const bf16* table; long ldt; const int* tokens; int T, width, vocab; float scale; const float* next;
+    float eps; cudaStream_t st;
+    template <int VEC, int KEEP>
+    cudaError_t operator()() const {
+        return launch_pdl(embed_kernel<A, VEC, KEEP>, dim3(T), dim3(row_threads(width, VEC)), 0, st, x, static_cast<A*>(xb), ldxb, table, ldt,
+                          tokens, width, vocab, scale, next, eps);
+    }
+};
+template <typename A, bool ADD>
+struct Norm {
+    float* x; void* xb; long ldxb; const float *y, *w, *next; const int* rows; int T, width; float eps; cudaStream_t st;
+    template <int VEC, int KEEP>
+    cudaError_t operator()() const {
+        return launch_pdl(norm_kernel<A, VEC, KEEP, ADD>, dim3(T), dim3(row_threads(width, VEC)), 0, st, x, static_cast<A*>(xb), ldxb, y, w, next,
+                          rows, width, eps);
+    }
+};
+
+}  // namespace
 
 cudaError_t embed(float* x, void* xb, long ldxb, const bf16* table, long ldt, const int* tokens, int T, int width, int vocab,
                   float scale, const float* next, float eps, int f32, cudaStream_t st) {
-    const dim3 grid(T), block(norm_threads(width));
     count_launch(1);
-    return f32 ? launch_pdl(embed_kernel<float>, grid, block, 0, st, x, static_cast<float*>(xb), ldxb, table, ldt, tokens, width, vocab,
-                            scale, next, eps)
-               : launch_pdl(embed_kernel<bf16>, grid, block, 0, st, x, static_cast<bf16*>(xb), ldxb, table, ldt, tokens, width, vocab,
-                            scale, next, eps);
+    return f32 ? by_width(width, Embed<float>{x, xb, ldxb, table, ldt, tokens, T, width, vocab, scale, next, eps, st})
+               : by_width(width, Embed<bf16>{x, xb, ldxb, table, ldt, tokens, T, width, vocab, scale, next, eps, st});
 }
 
 cudaError_t norm_add(float* x, void* xb, long ldxb, const float* y, const float* w, const float* next, int T, int width, float eps,
                      int f32, cudaStream_t st) {
-    const dim3 grid(T), block(norm_threads(width));
-    const int* none = nullptr;
     count_launch(1);
-    return f32 ? launch_pdl(norm_kernel<float, true>, grid, block, 0, st, x, static_cast<float*>(xb), ldxb, y, w, next, none, width, eps)
-               : launch_pdl(norm_kernel<bf16, true>, grid, block, 0, st, x, static_cast<bf16*>(xb), ldxb, y, w, next, none, width, eps);
+    return f32 ? by_width(width, Norm<float, true>{x, xb, ldxb, y, w, next, nullptr, T, width, eps, st})
+               : by_width(width, Norm<bf16, true>{x, xb, ldxb, y, w, next, nullptr, T, width, eps, st});
 }
 
 cudaError_t norm_rows(void* xb, long ldxb, const float* x, const float* w, const int* rows, int T, int width, float eps, int f32,
                       cudaStream_t st) {
-    const dim3 grid(T), block(norm_threads(width));
-    float* xm = const_cast<float*>(x);
-    const float* none = nullptr;
     count_launch(1);
-    return f32 ? launch_pdl(norm_kernel<float, false>, grid, block, 0, st, xm, static_cast<float*>(xb), ldxb, none, w, none, rows, width, eps)
-               : launch_pdl(norm_kernel<bf16, false>, grid, block, 0, st, xm, static_cast<bf16*>(xb), ldxb, none, w, none, rows, width, eps);
+    float* xm = const_cast<float*>(x);
+    return f32 ? by_width(width, Norm<float, false>{xm, xb, ldxb, nullptr, w, nullptr, rows, T, width, eps, st})
+               : by_width(width, Norm<bf16, false>{xm, xb, ldxb, nullptr, w, nullptr, rows, T, width, eps, st});
 }
 
 cudaError_t gated_norm(void* out, long ldout, const float* o, long ldo, const void* gate, long ldg, const float* w, int T,

@@ -177,7 +177,7 @@ class Model:
     def bar(self, tokens, f32):
         """Largest error a test accepts: a few times what rounding the inputs and outputs of every product and the outputs of
         silu to bfloat16 does to the logits of these tokens; for the 32-bit mode the same amplification applied to fp32
-        roundings."""
+        roundings, whose sum over a row grows with the row's length."""
         def rounded(x):
             return to_bf16(x)[1].reshape(np.shape(x))
 
@@ -192,7 +192,7 @@ class Model:
             noise = rel_error(self.plain(tokens)[0], exact).max()
         finally:
             plain.linear, plain.silu = linear, silu
-        return 4 * noise * (2.0 ** -13 if f32 else 1.0)
+        return 4 * noise * (2.0 ** -13 * max(1.0, self.cfg["width"] / 512) ** 0.5 if f32 else 1.0)
 
     def greedy(self, prompt, n):
         seq = list(prompt)
@@ -284,6 +284,9 @@ LANEDRA = {   # one mixer each
     "diff_mid": lambda: lanedra(48, 64, [diff_attention(3, 1, 100, 92, 70)], [None]),
     "diff_wide": lambda: lanedra(48, 64, [diff_attention(2, 1, 72, 150, 40, rot_dims=32)], [None]),
     "diff_very_wide": lambda: lanedra(48, 64, [diff_attention(2, 2, 40, 264, 45)], [None]),
+    "odd_width": lambda: lanedra(46, 51, [delta(3, 1, 10, 14, 3)], [27]),
+    "odd_wide_width": lambda: lanedra(2101, 40, [diff_attention(2, 1, 16, 20, 30)], [24]),
+    "wide_width": lambda: lanedra(8452, 40, [delta(2, 1, 16, 20, 3)], [24]),
     "diff_huge_keys": lambda: lanedra(48, 64, [diff_attention(2, 1, 520, 24, 45, rot_dims=100)], [None]),
 }
 
